@@ -199,8 +199,8 @@ class TwinOps:
         w = scores.gather(1, best.indices)
         weights.copy_(w / w.sum(-1, keepdim=True) if renormalize else w)
 
-    def moe_align(self, idx, E, with_tiles=None):
-        flat = idx.reshape(-1).long()
+    def moe_align(self, idx, E, with_tiles=None, table=None):
+        flat = (idx if table is None else table[idx.long()]).reshape(-1).long()
         order = torch.sort(flat, stable=True).indices.to(torch.int32)
         place = torch.empty_like(order)
         place[order.long()] = torch.arange(order.numel(), dtype=torch.int32)
@@ -436,7 +436,7 @@ def _rope_headnorm_write(self, proj, k_off, v_off, positions, freq, rot_dims, no
 
 
 def _attention_biased(self, out, q, k_cache, v_cache, block_tables, step, KVH, page_size, scale, softcap, slopes, window,
-                      chunk=None, sinks=None):
+                      chunk=None, sinks=None, keep=0, out_freq=None, gate=None):
     T, H, Dk = q.shape
     Dv = out.shape[2]
     G = H // KVH
@@ -458,7 +458,7 @@ def _attention_biased(self, out, q, k_cache, v_cache, block_tables, step, KVH, p
         j = torch.arange(seq_len)[None, :]
         ok = j <= i
         if window:
-            ok = ok & (j > i - window)
+            ok = ok & ((j > i - window) | (j < keep))
         if chunk:
             ok = ok & (j >= i // chunk * chunk)
         vv = torch.where(ok.any(0)[:, None, None], vv, torch.zeros_like(vv))      # pages a window gave back
@@ -473,7 +473,15 @@ def _attention_biased(self, out, q, k_cache, v_cache, block_tables, step, KVH, p
             if sinks is not None:
                 s = torch.cat([s, sinks[h].float().expand(Tq, 1)], -1)
             p = torch.softmax(s, -1)[:, :seq_len]
-            out[qs:qe, h] = (p @ vv[:, h // G]).to(out.dtype)
+            o = p @ vv[:, h // G]
+            if out_freq is not None:
+                a = -i.float() * out_freq.float()[None, :]
+                c, sn = torch.cos(a), torch.sin(a)
+                u, v = o[:, :Dv // 2], o[:, Dv // 2:]
+                o = torch.cat([u * c - v * sn, v * c + u * sn], -1)
+            if gate is not None:
+                o = o * torch.sigmoid(gate[qs:qe, h].float())[:, None]
+            out[qs:qe, h] = o.to(out.dtype)
 
 
 # -- a residual stream in several copies, the state-space mixer, gates -----------------------------------------------
@@ -591,6 +599,126 @@ def _rope_pairs_write(self, proj, k_off, v_off, positions, freq, magnitude, rot_
             k_cache[slot // page_size, :, slot % page_size] = k[t]
             v_cache[slot // page_size, :, slot % page_size] = v[t]
 
+
+# -- norms on outputs, normed and turned heads, the real-gated linear recurrent unit, clamped gated units ---------------
+def _post_norm(self, out, stream, y, weight, eps, base=None, rows=None, place=None, pair_weights=None, top=1, scale=1.0,
+               next_weight=None, next_eps=0.0):
+    T, h = stream.shape
+    v = torch.zeros(T, h)
+    if rows is not None:
+        r = rows[place.long()].view(T, top, h)
+        if pair_weights is not None:
+            r = r * pair_weights.view(T, top, 1)
+        v = scale * r.sum(1)
+    if y is not None:
+        v = v + self.materialize(y).float()
+    n = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+    stream.copy_((stream if base is None else base.float()) + n)
+    if out is None:
+        return
+    x = stream
+    if next_weight is not None:
+        x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + next_eps) * next_weight.float()
+    out.copy_(x.to(out.dtype))
+
+
+def _turn_halves(x, positions, freq, magnitude=1.0):
+    """x [T, heads, D]: dimension i < len(freq) turned with dimension i + len(freq) by position * freq[i]."""
+    n = freq.shape[0]
+    a = positions.float()[:, None] * freq.float()[None, :]
+    c, s = (torch.cos(a) * magnitude)[:, None, :], (torch.sin(a) * magnitude)[:, None, :]
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
+def _qkv_heads_write(self, proj, k_off, v_off, positions, q_w, k_w, eps, freq, magnitude, rot_dims, v_norm, v_freq, k_cache,
+                     v_cache, slots, H, G, D, V, page_size):
+    T = proj.shape[0]
+    unit = lambda x: x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+    q = proj[:, :H * D].float().reshape(T, H, D)
+    k = proj[:, k_off:k_off + G * D].float().reshape(T, G, D)
+    v = proj[:, v_off:v_off + G * V].float().reshape(T, G, V)
+    if q_w is not None:
+        q, k = unit(q) * q_w.float(), unit(k) * k_w.float()
+    if rot_dims:
+        q, k = _turn_halves(q, positions, freq, magnitude), _turn_halves(k, positions, freq, magnitude)
+    if v_norm:
+        v = unit(v)
+    if v_freq is not None:
+        v = _turn_halves(v, positions, v_freq)
+    proj[:, :H * D] = q.reshape(T, H * D).to(proj.dtype)
+    if slots is not None:
+        k, v = k.to(proj.dtype), v.to(proj.dtype)
+        for t, slot in enumerate(slots.tolist()):
+            if slot >= 0:
+                k_cache[slot // page_size, :, slot % page_size] = k[t]
+                v_cache[slot // page_size, :, slot % page_size] = v[t]
+    return proj
+
+
+def _glu(g, u, glu):
+    limit, slope, offset = glu
+    g, u = torch.clamp(g.float(), max=limit), torch.clamp(u.float(), -limit, limit)
+    return g * torch.sigmoid(slope * g) * (u + offset)
+
+
+def _glu_pairs(self, out, gu, glu):
+    out.copy_(_glu(gu[:, 0::2], gu[:, 1::2], glu).to(out.dtype))
+
+
+def _grouped_glu(self, out, x, w, order, row_scale, offsets, tiles, top, glu):
+    gu = torch.empty((out.shape[0], w.shape[1]), dtype=torch.float32)
+    self.grouped_linear(gu, x, w, order, row_scale, offsets, tiles, top)
+    out.copy_(_glu(gu[:, 0::2], gu[:, 1::2], glu).to(out.dtype))
+
+
+def _short_filter(self, out, x, x_off, conv_w, conv_b, state, tail_off, step, taps):
+    W = out.shape[1]
+    qs, slots = step.q_start.tolist(), step.state_slots.tolist()
+    for b in range(step.num_requests):
+        lo, hi = qs[b], qs[b + 1]
+        tail = state[slots[b]][tail_off:tail_off + (taps - 1) * W].view(taps - 1, W)
+        rows = torch.cat([tail, x[lo:hi, x_off:x_off + W].float()], 0)
+        acc = conv_b.float().expand(hi - lo, W).clone() if conv_b is not None else torch.zeros(hi - lo, W)
+        for u in range(taps):
+            acc = acc + rows[u:u + hi - lo] * conv_w.float()[:, u]
+        out[lo:hi] = acc.to(out.dtype)
+
+
+def _rglru_gates(self, ab, u, ra, ri, ra_b, ri_b, rate):
+    T, W = u.shape
+    n = ra.shape[0]
+    parts = u.float().view(T, n, W // n)
+    gate = lambda w, b: torch.sigmoid(torch.einsum("tnk,nok->tno", parts, w.float()).reshape(T, W) + b.float())
+    la = -rate.float() * gate(ra, ra_b)
+    ab[..., 0] = torch.exp(la)
+    ab[..., 1] = torch.sqrt(-torch.expm1(2.0 * la)) * gate(ri, ri_b) * u.float()
+
+
+def _rglru_scan(self, out, ab, proj, y_off, x_off, state, step, taps):
+    W = out.shape[1]
+    qs, slots = step.q_start.tolist(), step.state_slots.tolist()
+    for b in range(step.num_requests):
+        lo, hi = qs[b], qs[b + 1]
+        row = state[slots[b]]
+        S = row[:W].clone()
+        for t in range(lo, hi):
+            S = ab[t, :, 0] * S + ab[t, :, 1]
+            out[t] = (S * F.gelu(proj[t, y_off:y_off + W].float(), approximate="tanh")).to(out.dtype)
+        row[:W] = S
+        if taps > 1:
+            tail = row[W:].view(taps - 1, W)
+            tail.copy_(torch.cat([tail, proj[lo:hi, x_off:x_off + W].float()], 0)[-(taps - 1):].clone())
+
+
+def _rglru_step(self, *args):
+    return False                        # (the chain of the three above serves every step here)
+
+
+for _name, _fn in (("post_norm", _post_norm), ("qkv_heads_write", _qkv_heads_write), ("glu_pairs", _glu_pairs),
+                   ("grouped_glu", _grouped_glu), ("short_filter", _short_filter), ("rglru_gates", _rglru_gates),
+                   ("rglru_scan", _rglru_scan), ("rglru_step", _rglru_step)):
+    setattr(TwinOps, _name, _fn)
 
 for _name, _fn in (("hyper_norm", _hyper_norm), ("ssm_prepare", _ssm_prepare), ("ssm_scan", _ssm_scan),
                    ("gated_group_rmsnorm", _gated_group_rmsnorm), ("gate_mul", _gate_mul), ("act_mul", _act_mul),

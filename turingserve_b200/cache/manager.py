@@ -7,8 +7,8 @@ window and block size) form a GROUP.  A group has its own pool ``[runs, 2, pages
 ``[runs, pages, kv_heads, page, head_dim]`` and ``[runs, pages, kv_heads, page, value_dim]``)
 (the reference's single ``[L, 2, NB, KVH, 16, D]`` tensor, turingserve/engine/builder.py:76-80,
 is the one-group case), its own allocator and, per request, its own block table.  Pages go back
-to the group's free list when a request is released, and, in a group with a window or with blocks
-of positions, as soon as no later position can see them; freed pages are re-issued first-in first-out.
+to the group's free list when a request is released, and, in a group with a window (but for first tokens that
+stay visible) or with blocks of positions, as soon as no later position can see them; freed pages are re-issued first-in first-out.
 
 Slot arithmetic as turingserve/kv/kv_manager.py:17-40:
 slot(pos) = table[pos // page] * page + pos % page; pages needed = ceil(tokens / page) - held.
@@ -89,7 +89,7 @@ class CacheManager:
         for r, n in enumerate(needs):
             if n.cache is None or n.cache_from is not None:
                 continue
-            key = (n.cache.num_kv_heads, n.cache.head_dim, n.cache.window, n.cache.v_dim, n.cache.chunk)
+            key = (n.cache.num_kv_heads, n.cache.head_dim, n.cache.window, n.cache.v_dim, n.cache.chunk, n.cache.keep_first)
             if key not in keys:
                 keys[key] = len(self.groups)
                 self.groups.append(CacheGroup(n.cache, [], num_pages))
@@ -209,7 +209,9 @@ class CacheManager:
                 first_needed = max(first_needed, rc.num_tokens // c * c)
             keep_from = first_needed // self.page_size
             table = rc.tables[gi]
-            for p in range(rc.first_live_page[gi], min(keep_from, len(table))):
+            # (pages that hold a first token which stays visible are never given back)
+            stay = -(-g.need.keep_first // self.page_size) if w is not None else 0
+            for p in range(max(rc.first_live_page[gi], stay), min(keep_from, len(table))):
                 if table[p] != 0:
                     g.allocator.free(table[p])
                     table[p] = 0

@@ -91,6 +91,17 @@ class StreamLayerNormSpec:
 
 
 @dataclass(frozen=True)
+class PostRMSNormSpec:
+    """RMS norm of what a sublayer RETURNS, over a residual stream in 32-bit: x <- x + y / sqrt(mean(y^2) + eps) *
+    (weight_offset + weight), the sublayers reading x itself.  ``weight_offset`` 1: the weight is stored around zero."""
+
+    eps: float
+    weight_offset: float = 0.0
+    weight_name: str = "weight"         # local tensor name of the scale ('' = the norm's prefix itself)
+    kind: str = "rmsnorm_post"
+
+
+@dataclass(frozen=True)
 class BranchJoinSpec:
     """How the outputs of a layer's branches enter the residual stream: x <- x + scale * (their sum)."""
 
@@ -134,6 +145,48 @@ class SinkAttentionSpec:
     qkv_bias: bool = False
     out_gate: bool = False
     kind: str = "sink_attention"
+
+
+@dataclass(frozen=True)
+class NormedAttentionSpec:
+    """Grouped-query softmax attention over keys ``key_dim`` and values ``value_dim`` wide, no biases.  ``qk_norm``: every
+    head of q and k is RMS-normed over its dimensions with a learned weight common to the heads, before the rotation
+    (``position``, pairs of halves).  ``value_norm``: every head's value is divided by its root mean square (no weight).
+    ``value_base`` b: values are turned by their positions over all their dimensions, pair (m, m + value_dim / 2) by
+    j b^(-2m / value_dim), cached so, and a head's output at position i is turned back by -i b^(-2m / value_dim).
+    score = cap tanh(q.k scale / cap) (``softcap`` None: no cap).  ``window`` w: position i sees i - w < j <= i, and the
+    first ``keep_first`` positions of the sequence whatever the distance.  ``head_gate``: head h's output times
+    sigmoid(W_g h)_h, one number per head ('g'), before the output projection.  eps of all norms: ``norm_eps``."""
+
+    num_heads: int
+    num_kv_heads: int
+    key_dim: int
+    value_dim: int
+    scale: float
+    norm_eps: float
+    position: Any = None
+    softcap: float | None = None
+    window: int | None = None
+    keep_first: int = 0
+    qk_norm: bool = True
+    value_norm: bool = True
+    value_base: float | None = None
+    head_gate: bool = True
+    kind: str = "normed_attention"
+
+
+@dataclass(frozen=True)
+class RGLRUSpec:
+    """Recurrent block of a real-gated linear recurrent unit (Griffin): two branches ``width`` wide, y = gelu_tanh(W_y h
+    + b) and u = filter(W_x h + b) (``conv_taps`` taps per channel, with bias); r and i are sigmoids of block-diagonal
+    products of u in ``num_blocks`` equal parts (with bias); log a = -decay_scale r softplus(lam), S <- a S + sqrt(1 - a^2) i u;
+    output W_o (S y)."""
+
+    width: int
+    num_blocks: int
+    conv_taps: int
+    decay_scale: float = 8.0
+    kind: str = "rglru"
 
 
 @dataclass(frozen=True)
@@ -255,7 +308,7 @@ class YarnRotarySpec:
     index at which a pair turns r times is idx(r) = dims * log(original / (2 * pi * r)) / (2 * log(base)); the
     blend starts at first = max(floor(idx(fast)), 0) and is complete at last = min(ceil(idx(slow)), dims - 1):
     share_i = min(max((i - first) / max(last - first, 0.001), 0), 1).  Cosine and sine are both scaled by
-    1 + 0.1 * log(factor)."""
+    1 + 0.1 * log(factor).  ``pairing`` "halves": dimension i is paired with dimension i + dims/2 instead."""
 
     base: float
     dims: int
@@ -263,6 +316,7 @@ class YarnRotarySpec:
     original: float = 0.0
     fast: float = 32.0
     slow: float = 1.0
+    pairing: str = "neighbours"
     kind: str = "yarn_pairs"
 
 
@@ -345,7 +399,10 @@ class RoutedMLPSpec:
     down(act(gate(.)) * up(.)).  ``correction``: a learned vector added to the scores for the choice only (the
     weights stay the scores).  ``identity``: so many more router outputs, behind the ``num_experts`` with
     tensors, are experts that return their input.  ``shared_intermediate_size``: one more feed-forward of the same
-    form ('shared.up', 'shared.down') that every token uses, added unweighted."""
+    form ('shared.up', 'shared.down') that every token uses, added unweighted.  ``table_rows`` not None: no router; an integer
+    table ('table' [table_rows, top_k]) gives every token id its experts, each with weight 1 / top_k.  ``activation``
+    "clamped_glu" (gated only): g sigmoid(glu_slope g) (u + glu_offset) with g = min(gate, glu_limit), u = clamp(up, +-glu_limit);
+    the shared expert has a limit of its own (``shared_glu_limit``)."""
 
     num_experts: int
     top_k: int
@@ -358,6 +415,11 @@ class RoutedMLPSpec:
     correction: bool = False
     identity: int = 0
     shared_intermediate_size: int | None = None
+    table_rows: int | None = None
+    glu_limit: float = float("inf")
+    shared_glu_limit: float = float("inf")
+    glu_slope: float = 1.702
+    glu_offset: float = 1.0
     kind: str = "routed_mlp"
 
 

@@ -26,3 +26,18 @@ template <> __device__ __forceinline__ float ts_activate_for<bf16>(float z, int 
   if (kind == TS_ACT_SILU) return __fdividef(z, 1.f + __expf(-z));
   return ts_activate(z, kind);
 }
+
+// A gated unit whose inputs are clamped: g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(slope g) (u + offset).
+struct TsGlu {
+  float limit, slope, offset;
+};
+template <typename T> __device__ __forceinline__ float ts_glu_for(float g, float u, const TsGlu& a) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return g / (1.f + expf(-a.slope * g)) * (u + a.offset);
+}
+template <> __device__ __forceinline__ float ts_glu_for<bf16>(float g, float u, const TsGlu& a) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return __fdividef(g, 1.f + __expf(-a.slope * g)) * (u + a.offset);
+}

@@ -1,5 +1,5 @@
 // The attention of attention_biased.cu (capped scores, distance bias per head, window, blocks of positions, a sink in
-// the softmax's denominator, values of their own width or inside the key rows) on the tensor cores, bfloat16 storage, for key rows that are a multiple of 64 wide.
+// the softmax's denominator, kept first tokens, outputs turned back and gated, values of their own width or inside the key rows) on the tensor cores, bfloat16 storage, for key rows that are a multiple of 64 wide.
 //
 // Work split as in the prompt-portion kernel: one block per (tile of 64 query ROWS, kv head, request), a row being
 // one (token, head-in-group) pair, four warps of 16 rows (m16n8k16), keys 64 at a time through a cp.async pipeline
@@ -44,7 +44,7 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
                             const int* __restrict__ seq_lens, int table_width, int H, int KVH, int page, float scale,
                             float softcap, const float* __restrict__ slopes, int window, int v_chunks, int splits,
                             float* __restrict__ scratch, int* __restrict__ counters, int block_of,
-                            const float* __restrict__ sinks) {
+                            const float* __restrict__ sinks, int keep, AttnFinish fin) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int CHK = DK / 8, KS = DK / 16, NT = DV / 8, CHV = DV / 8;
@@ -112,24 +112,30 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
   int j_hi = prefix + last_row / G;
   int j_lo = window > 0 ? max(0, prefix + row0 / G - window + 1) : 0;
   if (block_of > 0) j_lo = max(j_lo, (prefix + row0 / G) / block_of * block_of);
+  // the kept first tokens that lie before what the window shows any row: `kept` tiles of their own, ahead of the window's
+  const int keep_end = keep > 0 ? min(keep, j_lo) : 0;
+  int kept = (keep_end + BM_TILE - 1) / BM_TILE, kept_first = 0;
+  int n_tiles = seq_len > 0 ? kept + (j_hi - j_lo) / BM_TILE + 1 : 0;
   if (my_splits > 1) {
-    const int all = (j_hi - j_lo) / BM_TILE + 1;
-    const int per = (all + my_splits - 1) / my_splits;
-    const int first = j_lo + split * per * BM_TILE;
-    j_hi = min(j_hi, first + per * BM_TILE - 1);
-    j_lo = first;
+    const int per = (n_tiles + my_splits - 1) / my_splits;
+    const int t0 = split * per, t1 = min(n_tiles, t0 + per);
+    n_tiles = max(0, t1 - t0);
+    j_lo += max(0, t0 - kept) * BM_TILE;
+    kept_first = min(t0, kept);
+    kept = max(0, min(t1, kept) - kept_first);                       // (of this block)
+    if (n_tiles > kept) j_hi = min(j_hi, j_lo + (n_tiles - kept) * BM_TILE - 1);
   }
-  const int n_tiles = (seq_len > 0 && j_hi >= j_lo) ? (j_hi - j_lo) / BM_TILE + 1 : 0;
   const int w_first = row0 + wrow, w_last = min(w_first + 15, n_rows - 1);
   const int w_pos_lo = prefix + w_first / G, w_pos_hi = (w_first < n_rows) ? prefix + w_last / G : -1;
 
   const int page_shift = (page & (page - 1)) == 0 ? 31 - __clz(page) : -1;
   const int page_first = j_lo / page;
-  const int n_pages = n_tiles > 0 ? j_hi / page - page_first + 1 : 0;
-  const bool pages_staged = n_pages <= BM_PAGES_S;
+  const int n_pages = n_tiles > kept ? j_hi / page - page_first + 1 : 0;
+  const int kept_pages = kept > 0 ? (keep_end - 1) / page + 1 : 0;   // (staged ahead of the others)
+  const bool pages_staged = kept_pages + n_pages <= BM_PAGES_S;
   if (pages_staged) {
-    for (int i = threadIdx.x; i < n_pages; i += BM_WARPS * 32)
-      pages_s[i] = block_tables[(size_t)b * table_width + page_first + i];
+    for (int i = threadIdx.x; i < kept_pages + n_pages; i += BM_WARPS * 32)
+      pages_s[i] = block_tables[(size_t)b * table_width + (i < kept_pages ? i : page_first + i - kept_pages)];
     __syncthreads();
   }
   const int v_width = DV * v_chunks;                                 // a value row's width in its own tensor
@@ -139,18 +145,21 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
   constexpr int LPK = CHK >= 32 ? 32 : (CHK >= 16 ? 16 : 8);         // lanes a key
   constexpr int KPI = BM_WARPS * (32 / LPK);                         // keys the block brings in one round
   auto load_tile = [&](int t, int stage) {
-    const int j0 = j_lo + t * BM_TILE;
+    const bool early = t < kept;                                     // a tile of kept first tokens
+    const int j0 = early ? (kept_first + t) * BM_TILE : j_lo + (t - kept) * BM_TILE;
+    const int j_end = early ? keep_end - 1 : j_hi;
+    const int page_at = early ? 0 : kept_pages - page_first;         // a logical page's place among the staged ones, less the page
     unsigned char* ks_ = k_s + (size_t)stage * BM_TILE * DK * 2;
     unsigned char* vs_ = v_s + (size_t)stage * BM_TILE * DV * 2;
     const int c0 = lane % LPK;
 #pragma unroll 2
     for (int key = warp * (32 / LPK) + lane / LPK; key < BM_TILE; key += KPI) {
       const int j = j0 + key;
-      const bool ok = j <= j_hi;
+      const bool ok = j <= j_end;
       size_t tok = 0;
       if (ok) {
         const int lp = page_shift >= 0 ? (j >> page_shift) : (j / page);
-        const int pg = pages_staged ? pages_s[lp - page_first] : block_tables[(size_t)b * table_width + lp];
+        const int pg = pages_staged ? pages_s[lp + page_at] : block_tables[(size_t)b * table_width + lp];
         tok = ((size_t)pg * KVH + kvh) * page + (size_t)(j - lp * page);
       }
       const bf16* krow = k_cache + tok * DK;
@@ -182,9 +191,11 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
     __syncthreads();
     const unsigned char* ks_ = k_s + (size_t)(t % STAGES) * BM_TILE * DK * 2;
     const unsigned char* vs_ = V_IN_K ? ks_ : v_s + (size_t)(t % STAGES) * BM_TILE * DV * 2;
-    const int j0 = j_lo + t * BM_TILE;
+    const bool early = t < kept;
+    const int j0 = early ? (kept_first + t) * BM_TILE : j_lo + (t - kept) * BM_TILE;
+    const int j_end = early ? keep_end - 1 : j_hi;
     const bool in_future = j0 > w_pos_hi;                                          // warp-uniform
-    const bool in_past = (window > 0 && (j0 + BM_TILE - 1) < (w_pos_lo - window + 1)) ||
+    const bool in_past = (window > 0 && j0 >= keep && (j0 + BM_TILE - 1) < (w_pos_lo - window + 1)) ||
                          (block_of > 0 && w_pos_lo >= 0 && (j0 + BM_TILE - 1) < w_pos_lo / block_of * block_of);
     if (!in_future && !in_past) {
       float s_acc[NTW][4];
@@ -216,7 +227,7 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
           float v = s_acc[nt][e] * scale;
           if (softcap > 0.f) v = capped(v, softcap, inv_cap);
           v = (v - slope[e >> 1] * (float)(p - j)) * BM_LOG2E;
-          const bool ok = (j <= p) && (j >= lo[e >> 1]) && (j <= j_hi);
+          const bool ok = (j <= p) && (j >= lo[e >> 1] || j < keep) && (j <= j_end);
           v = ok ? v : -INFINITY;
           s_acc[nt][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -294,6 +305,23 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
         const float down = exp2f(m_run[r] - top);
         inv = down / (l_run[r] * down + exp2f(sink2[r] - top));
       }
+      if (fin.gate != nullptr) {
+        const int row = row0 + wrow + (lane >> 2) + 8 * r;
+        const bf16* gate = (const bf16*)fin.gate + (size_t)(qs + row / G) * fin.gate_ts + kvh * G + row % G;
+        inv *= 1.f / (1.f + expf(-to_f(*gate)));
+      }
+      if (fin.out_freq != nullptr) {                                 // (whole value rows only: both columns of a pair are this thread's)
+#pragma unroll
+        for (int i = 0; i < NT / 2; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            float sn, cs;
+            sincosf((float)pos[r] * fin.out_freq[i * 8 + (lane & 3) * 2 + e], &sn, &cs);
+            const float a = o[i][2 * r + e], c = o[i + NT / 2][2 * r + e];
+            o[i][2 * r + e] = a * cs + c * sn;
+            o[i + NT / 2][2 * r + e] = c * cs - a * sn;
+          }
+      }
 #pragma unroll
       for (int i = 0; i < NT; ++i) {
         const int d = i * 8 + (lane & 3) * 2;
@@ -369,29 +397,51 @@ attention_biased_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, cons
       const float down = exp2f(mm - top);
       inv = down / (ll * down + exp2f(sk - top));
     }
+    if (fin.gate != nullptr) inv *= 1.f / (1.f + expf(-to_f(((const bf16*)fin.gate)[(size_t)qs * fin.gate_ts + kvh * G + row])));
     for (int k = 0; k < n_rec; ++k) m_m[row * BM_MAX_RECORDS + k] *= inv;
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < n_rows * (DV / 4); idx += BM_WARPS * 32) {
-    const int row = idx / (DV / 4), d = (idx % (DV / 4)) * 4;
-    float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-    for (int k0 = 0; k0 < n_rec; k0 += 16) {                         // sixteen loads in flight, then their sum, in record order
-      float4 v[16];
+  // (four columns and, so that pairs can be turned, the four half a row further)
+  constexpr int HALF = DV / 2;
+  for (int idx = threadIdx.x; idx < n_rows * (HALF / 4); idx += BM_WARPS * 32) {
+    const int row = idx / (HALF / 4), d = (idx % (HALF / 4)) * 4;
+    float a[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    for (int k0 = 0; k0 < n_rec; k0 += 8) {                          // sixteen loads in flight, then their sums, in record order
+      float4 v[2][8];
 #pragma unroll
-      for (int u = 0; u < 16; ++u)
-        v[u] = k0 + u < n_rec ? __ldcg(reinterpret_cast<const float4*>(rec_of(k0 + u, row) + 4 + d)) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int u = 0; u < 8; ++u)
 #pragma unroll
-      for (int u = 0; u < 16; ++u) {
+        for (int h = 0; h < 2; ++h)
+          v[h][u] = k0 + u < n_rec ? __ldcg(reinterpret_cast<const float4*>(rec_of(k0 + u, row) + 4 + d + h * HALF))
+                                   : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
         const float w = k0 + u < n_rec ? m_m[row * BM_MAX_RECORDS + k0 + u] : 0.f;
-        a0 = fmaf(v[u].x, w, a0);
-        a1 = fmaf(v[u].y, w, a1);
-        a2 = fmaf(v[u].z, w, a2);
-        a3 = fmaf(v[u].w, w, a3);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          a[h][0] = fmaf(v[h][u].x, w, a[h][0]);
+          a[h][1] = fmaf(v[h][u].y, w, a[h][1]);
+          a[h][2] = fmaf(v[h][u].z, w, a[h][2]);
+          a[h][3] = fmaf(v[h][u].w, w, a[h][3]);
+        }
       }
     }
-    bf16* dst = out + (size_t)qs * out_ts + (size_t)(kvh * G + row) * out_hs + chunk * DV + d;
-    *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a0, a1);
-    *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(a2, a3);
+    if (fin.out_freq != nullptr) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float sn, cs;
+        sincosf((float)prefix * fin.out_freq[d + e], &sn, &cs);      // (the single token's position)
+        const float x = a[0][e], y = a[1][e];
+        a[0][e] = x * cs + y * sn;
+        a[1][e] = y * cs - x * sn;
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      bf16* dst = out + (size_t)qs * out_ts + (size_t)(kvh * G + row) * out_hs + chunk * DV + h * HALF + d;
+      *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a[h][0], a[h][1]);
+      *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(a[h][2], a[h][3]);
+    }
   }
 }
 
@@ -399,7 +449,7 @@ template <int DK, int DV, bool V_IN_K, int STAGES, int SPREAD>
 int launch(bf16* out, int out_ts, int out_hs, const bf16* q, int q_ts, int q_hs, const bf16* k_cache, const bf16* v_cache,
            const int* block_tables, const int* q_start, const int* seq_lens, int B, int table_width, int max_q_len, int H,
            int KVH, int page, float scale, float softcap, const float* slopes, int window, int v_chunks, int splits,
-           float* scratch, int* counters, int block_of, const float* sinks, cudaStream_t s) {
+           float* scratch, int* counters, int block_of, const float* sinks, int keep, AttnFinish fin, cudaStream_t s) {
   const size_t smem = (size_t)BM_ROWS * DK * 2 + (size_t)STAGES * BM_TILE * DK * 2 + (V_IN_K ? 0 : (size_t)STAGES * BM_TILE * DV * 2);
   static bool configured = false;
   if (!configured) {
@@ -412,7 +462,7 @@ int launch(bf16* out, int out_ts, int out_hs, const bf16* q, int q_ts, int q_hs,
   dim3 grid(ceil_div(max_q_len * G, BM_ROWS) * v_chunks * splits, KVH, B);
   ts_launch(attention_biased_mma_kernel<DK, DV, V_IN_K, STAGES, SPREAD>, dim3(grid), dim3(BM_WARPS * 32), smem, s, out, out_ts, out_hs, q,
             q_ts, q_hs, k_cache, v_cache, block_tables, q_start, seq_lens, table_width, H, KVH, page, scale, softcap, slopes,
-            window, v_chunks, splits, scratch, counters, block_of, sinks);
+            window, v_chunks, splits, scratch, counters, block_of, sinks, keep, fin);
   TS_LAUNCH_CHECK();
 }
 
@@ -451,7 +501,8 @@ TS_API int ts_attention_biased_mma(void* out, int out_ts, int out_hs, const void
                                    const void* v_cache, const int* block_tables, const int* q_start, const int* seq_lens,
                                    int B, int table_width, int max_q_len, int H, int KVH, int Dk, int Dv, int page,
                                    float scale, float softcap, const float* slopes, int window, int splits, float* scratch,
-                                   int* counters, int spread, int block_of, const float* sinks, void* stream) {
+                                   int* counters, int spread, int block_of, const float* sinks, int keep, const float* out_freq,
+                                   const void* gate, int gate_ts, void* stream) {
   if (B <= 0 || max_q_len <= 0) return 0;
   const int v_in_k = v_cache == nullptr;
   const int inst = (KVH > 0 && H % KVH == 0) ? instance_of(Dk, Dv, v_in_k) : 0;
@@ -459,6 +510,13 @@ TS_API int ts_attention_biased_mma(void* out, int out_ts, int out_hs, const void
   if ((q_ts % 8) || (q_hs % 8) || ((uintptr_t)q & 15) || (out_ts % 2) || (out_hs % 2) || ((uintptr_t)out & 3))
     TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_attention_biased_mma: query rows must start on 16-byte boundaries");
   if (B > 65535 || KVH > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_attention_biased_mma: %d requests / %d kv heads", B, KVH);
+  if (keep < 0 || (keep > 0 && block_of > 0)) TS_REFUSE(TS_ERR_SHAPE, "ts_attention_biased_mma: %d kept tokens (with blocks of %d)", keep, block_of);
+  if (out_freq != nullptr && ts_attention_biased_mma_chunk(Dk, Dv, v_in_k) != Dv)
+    TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_attention_biased_mma: values of %d are cut over blocks, their pairs cannot be turned", Dv);
+  AttnFinish fin;
+  fin.out_freq = out_freq;
+  fin.gate = gate;
+  fin.gate_ts = gate_ts;
   if (splits < 1) splits = 1;
   if (splits > 1 && (splits > BM_MAX_SPLITS || H / KVH > BM_ROWS || scratch == nullptr || counters == nullptr))
     TS_REFUSE(TS_ERR_LIMIT, "ts_attention_biased_mma: %d splits", splits);
@@ -471,14 +529,14 @@ TS_API int ts_attention_biased_mma(void* out, int out_ts, int out_hs, const void
     if (spread && groups == 1)                                                                                                \
       return launch<DKK, DVV, VK, ST, 1>((bf16*)out, out_ts, out_hs, (const bf16*)q, q_ts, q_hs, (const bf16*)k_cache,        \
                                          (const bf16*)v_cache, block_tables, q_start, seq_lens, B, table_width, max_q_len,    \
-                                         H, KVH, page, scale, softcap, slopes, window, CHUNKS, splits, scratch, counters, block_of, sinks, s); \
+                                         H, KVH, page, scale, softcap, slopes, window, CHUNKS, splits, scratch, counters, block_of, sinks, keep, fin, s); \
     if (spread)                                                                                                               \
       return launch<DKK, DVV, VK, ST, 2>((bf16*)out, out_ts, out_hs, (const bf16*)q, q_ts, q_hs, (const bf16*)k_cache,        \
                                          (const bf16*)v_cache, block_tables, q_start, seq_lens, B, table_width, max_q_len,    \
-                                         H, KVH, page, scale, softcap, slopes, window, CHUNKS, splits, scratch, counters, block_of, sinks, s); \
+                                         H, KVH, page, scale, softcap, slopes, window, CHUNKS, splits, scratch, counters, block_of, sinks, keep, fin, s); \
     return launch<DKK, DVV, VK, ST, 0>((bf16*)out, out_ts, out_hs, (const bf16*)q, q_ts, q_hs, (const bf16*)k_cache,      \
                                            (const bf16*)v_cache, block_tables, q_start, seq_lens, B, table_width, max_q_len,  \
-                                           H, KVH, page, scale, softcap, slopes, window, CHUNKS, splits, scratch, counters, block_of, sinks, s); \
+                                           H, KVH, page, scale, softcap, slopes, window, CHUNKS, splits, scratch, counters, block_of, sinks, keep, fin, s); \
   } while (0)
   if (inst == 1) TS_BM(64, 64, false, 3, 1);
   if (inst == 2) TS_BM(128, 128, false, 2, 1);                        // (two stages: 80 KB a block, so two blocks share an SM)

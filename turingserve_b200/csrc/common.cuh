@@ -81,6 +81,14 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 
+// What an attention kernel does to a head's output on its way to memory: the pairs (m, m + Dv/2) turned by -position *
+// out_freq[m] (null: not), then the head times sigmoid(gate[token * gate_ts + head]) (null: not).
+struct AttnFinish {
+  const float* out_freq;
+  const void* gate;
+  int gate_ts;
+};
+
 // Programmatic dependent launch: a kernel launched with ts_launch may start while its predecessor
 // in the stream is still running.  Every kernel calls pdl_launch_dependents() first (its successor
 // may be scheduled) and pdl_wait() before it reads or writes anything a predecessor may touch;

@@ -10,12 +10,16 @@
 //   ts_moe_align       pairs p = t * top + r sorted by expert: offsets[E + 1], order[P] (sorted place -> pair),
 //                      place[P] (pair -> sorted place), and the list of row tiles (expert, first row) the
 //                      grouped products walk; experts from `with_tiles` on get a group but no tiles (experts
-//                      without weights, whose output is their input).
+//                      without weights, whose output is their input).  With a table [rows, top] the choices are
+//                      the rows of the token ids (no router): pair p's expert is table[id[p / top], p % top].
 //   ts_grouped_linear  out[i, :] = act(a_i . W[e(i)]^T) for the sorted places i; a_i is row i of `x`, or, when
 //                      `order` is given, row order[i] / top of `x` times row_scale[order[i]] (rounded to the
 //                      storage type: the weighted input of an expert).  32-bit accumulation in ascending k
 //                      (FFMA; tensor cores for bfloat16 with K a multiple of 8): a row's result does not
 //                      depend on its tile-mates.
+//   ts_grouped_glu     the same with gate and up rows taking turns in W (gate 0, up 0, gate 1, ...): neighbouring
+//                      columns of the product are a gate and its up, and what leaves the kernel is the clamped
+//                      gated unit of the two, half as wide
 //   ts_moe_combine     out[t, :] = sum over r (ascending) of (w[t, r] *) y[place[t * top + r], :], in 32-bit; a pair
 //                      whose sorted place is *pass_from or later contributes the token's own input row instead.
 #include "activations.cuh"
@@ -124,9 +128,22 @@ router_topk_kernel(int* __restrict__ idx_out, float* __restrict__ w_out, const T
 
 // ---------------------------------------------------------------------------------------------------
 // One block.  tiles: [0] = number of row tiles, then (expert, first sorted row) pairs.
+// the expert of pair p: its entry of idx, or, with a table, of the row its token's id names
+__device__ __forceinline__ int expert_of(const int* idx, int p, int E, const int* table, int top, int table_rows) {
+  int e;
+  if (table == nullptr) {
+    e = idx[p];
+  } else {
+    const int id = min(max(idx[p / top], 0), table_rows - 1);
+    e = table[(size_t)id * top + p % top];
+  }
+  return min(max(e, 0), E - 1);
+}
+
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(const int* __restrict__ idx, int P, int E, int* __restrict__ offsets, int* __restrict__ order,
-                 int* __restrict__ place, int* __restrict__ tiles, int tile_rows, int with_tiles) {
+                 int* __restrict__ place, int* __restrict__ tiles, int tile_rows, int with_tiles,
+                 const int* __restrict__ table, int top, int table_rows) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ int sm_i[];
@@ -134,7 +151,7 @@ moe_align_kernel(const int* __restrict__ idx, int P, int E, int* __restrict__ of
   int* cursor = sm_i + E;     // [E]
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&count[min(max(idx[p], 0), E - 1)], 1);
+  for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&count[expert_of(idx, p, E, table, top, table_rows)], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0, n = 0;
@@ -155,18 +172,18 @@ moe_align_kernel(const int* __restrict__ idx, int P, int E, int* __restrict__ of
   // a pair's place inside its expert's group is whatever the cursor gives: a row's result does not depend
   // on where in a tile it sits
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
-    const int at = atomicAdd(&cursor[min(max(idx[p], 0), E - 1)], 1);
+    const int at = atomicAdd(&cursor[expert_of(idx, p, E, table, top, table_rows)], 1);
     order[at] = p;
     place[p] = at;
   }
 }
 
 // ---------------------------------------------------------------------------------------------------
-template <typename TI, typename TO>
+template <typename TI, typename TO, bool GLU>
 __global__ void __launch_bounds__(256)
 grouped_linear_kernel(TO* __restrict__ out, const TI* __restrict__ x, const TI* __restrict__ w,
                       const int* __restrict__ order, const float* __restrict__ row_scale,
-                      const int* __restrict__ offsets, const int* __restrict__ tiles, int top, int N, int K, int act) {
+                      const int* __restrict__ offsets, const int* __restrict__ tiles, int top, int N, int K, int act, TsGlu glu) {
   pdl_launch_dependents();
   pdl_wait();
   if ((int)blockIdx.y >= tiles[0]) return;
@@ -225,11 +242,19 @@ grouped_linear_kernel(TO* __restrict__ out, const TI* __restrict__ x, const TI* 
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= m_end) continue;
+    if constexpr (GLU) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int n = n0 + tx * 4 + j;
-      if (n >= N) continue;
-      out[(size_t)m * N + n] = from_f<TO>(ts_activate(acc[i][j], act));
+      for (int j = 0; j < 4; j += 2) {
+        const int n = n0 + tx * 4 + j;
+        if (n < N) out[(size_t)m * (N / 2) + n / 2] = from_f<TO>(ts_glu_for<TO>(acc[i][j], acc[i][j + 1], glu));
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int n = n0 + tx * 4 + j;
+        if (n >= N) continue;
+        out[(size_t)m * N + n] = from_f<TO>(ts_activate(acc[i][j], act));
+      }
     }
   }
 }
@@ -242,11 +267,11 @@ grouped_linear_kernel(TO* __restrict__ out, const TI* __restrict__ x, const TI* 
 constexpr int GM_BM = 64, GM_BN = 64, GM_BK = 64, GM_STAGES = 4, GM_WARPS = 4;
 static_assert(GM_BM == GL_BM, "both grouped kernels walk the same row tiles");
 
-template <typename TO>
+template <typename TO, bool GLU>
 __global__ void __launch_bounds__(GM_WARPS * 32)
 grouped_linear_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ x, const bf16* __restrict__ w,
                           const int* __restrict__ order, const float* __restrict__ row_scale,
-                          const int* __restrict__ offsets, const int* __restrict__ tiles, int top, int N, int K, int act) {
+                          const int* __restrict__ offsets, const int* __restrict__ tiles, int top, int N, int K, int act, TsGlu glu) {
   pdl_launch_dependents();
   pdl_wait();
   if ((int)blockIdx.y >= tiles[0]) return;
@@ -338,14 +363,24 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ x, cons
     __syncthreads();
   }
   cp_async_wait<0>();
+  if constexpr (GLU) {
 #pragma unroll
-  for (int nt = 0; nt < GM_BN / 8; ++nt)
+    for (int nt = 0; nt < GM_BN / 8; ++nt)
 #pragma unroll
-    for (int e_ = 0; e_ < 4; ++e_) {
-      const int m = m0 + warp * 16 + (lane >> 2) + 8 * (e_ >> 1);
-      const int n = n0 + nt * 8 + (lane & 3) * 2 + (e_ & 1);
-      if (m < m_end && n < N) out[(size_t)m * N + n] = from_f<TO>(ts_activate(acc[nt][e_], act));
-    }
+      for (int h = 0; h < 2; ++h) {
+        const int m = m0 + warp * 16 + (lane >> 2) + 8 * h, n = n0 + nt * 8 + (lane & 3) * 2;
+        if (m < m_end && n < N) out[(size_t)m * (N / 2) + n / 2] = from_f<TO>(ts_glu_for<TO>(acc[nt][2 * h], acc[nt][2 * h + 1], glu));
+      }
+  } else {
+#pragma unroll
+    for (int nt = 0; nt < GM_BN / 8; ++nt)
+#pragma unroll
+      for (int e_ = 0; e_ < 4; ++e_) {
+        const int m = m0 + warp * 16 + (lane >> 2) + 8 * (e_ >> 1);
+        const int n = n0 + nt * 8 + (lane & 3) * 2 + (e_ & 1);
+        if (m < m_end && n < N) out[(size_t)m * N + n] = from_f<TO>(ts_activate(acc[nt][e_], act));
+      }
+  }
 }
 
 // The same product for steps of a few tokens, where an expert has a handful of rows and the time is the experts'
@@ -359,11 +394,11 @@ grouped_linear_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ x, cons
 constexpr int GV_ROWS = 8, GV_WARPS = 8, GV_UNROLL = 8;
 constexpr int GV_STREAM_ROWS = 64;      // steps with at most this many (token, choice) pairs take this kernel
 
-template <typename TO>
+template <typename TO, bool GLU>
 __global__ void __launch_bounds__(GV_WARPS * 32)
 grouped_linear_stream_kernel(TO* __restrict__ out, const bf16* __restrict__ x, const bf16* __restrict__ w,
                              const int* __restrict__ order, const float* __restrict__ row_scale,
-                             const int* __restrict__ offsets, const int* __restrict__ tiles, int top, int N, int K, int act) {
+                             const int* __restrict__ offsets, const int* __restrict__ tiles, int top, int N, int K, int act, TsGlu glu) {
   pdl_launch_dependents();
   // (the tile list is written by the kernel before this one: nothing can be fetched ahead of the wait)
   pdl_wait();
@@ -417,7 +452,10 @@ grouped_linear_stream_kernel(TO* __restrict__ out, const bf16* __restrict__ x, c
         mma_bf16(acc, a2, wv[u].z, wv[u].w);
       }
     }
-    if (row_ok) {
+    if (row_ok && GLU) {
+      const int n = n0 + 2 * t;
+      if (n < N) out[(size_t)row * (N / 2) + n / 2] = from_f<TO>(ts_glu_for<TO>(acc[0], acc[1], glu));
+    } else if (row_ok) {
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         const int n = n0 + 2 * t + i;
@@ -466,7 +504,81 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
   }
 }
 
+// out[t, i] = the clamped gated unit of columns 2 i (gate) and 2 i + 1 (up) of a row; the row may be the partial sums of a
+// product cut along K (summed in split order, rounded as the product's own last pass would have).
+template <typename T, bool PARTS>
+__global__ void __launch_bounds__(256)
+glu_pairs_kernel(T* __restrict__ out, const T* __restrict__ gu, const float* __restrict__ part, int splits, size_t split_stride,
+                 size_t total, TsGlu glu) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    float g = 0.f, u = 0.f;
+    if (PARTS) {
+      for (int sp = 0; sp < splits; ++sp) {
+        const float2 p = __ldcg(reinterpret_cast<const float2*>(part + sp * split_stride + 2 * i));
+        g += p.x;
+        u += p.y;
+      }
+      g = round_to<T>(g);
+      u = round_to<T>(u);
+    } else {
+      g = to_f(gu[2 * i]);
+      u = to_f(gu[2 * i + 1]);
+    }
+    out[i] = from_f<T>(ts_glu_for<T>(g, u, glu));
+  }
+}
+
+// the same for bfloat16 rows, 8 outputs (32 bytes in, 16 bytes out) a thread
+__global__ void __launch_bounds__(256)
+glu_pairs_vec_kernel(bf16* __restrict__ out, const bf16* __restrict__ gu, size_t total8, TsGlu glu) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total8; i += (size_t)gridDim.x * blockDim.x) {
+    const uint4 a = reinterpret_cast<const uint4*>(gu)[2 * i], b = reinterpret_cast<const uint4*>(gu)[2 * i + 1];
+    const __nv_bfloat162* ah = reinterpret_cast<const __nv_bfloat162*>(&a);
+    const __nv_bfloat162* bh = reinterpret_cast<const __nv_bfloat162*>(&b);
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 p = __bfloat1622float2(ah[j]), q = __bfloat1622float2(bh[j]);
+      v[j] = ts_glu_for<bf16>(p.x, p.y, glu);
+      v[4 + j] = ts_glu_for<bf16>(q.x, q.y, glu);
+    }
+    uint4 o;
+    __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) oh[j] = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+    reinterpret_cast<uint4*>(out)[i] = o;
+  }
+}
+
 }  // namespace
+
+// out [rows, inter]; gu [rows, 2 inter] in `dtype`, or part [splits, rows, 2 inter] 32-bit on 8-byte boundaries.
+TS_API int ts_glu_pairs(void* out, const void* gu, const float* part, int splits, int rows, int inter, float limit, float slope,
+                        float offset, int dtype, void* stream) {
+  const size_t total = (size_t)rows * inter;
+  if (total == 0) return 0;
+  if (part != nullptr && ((uintptr_t)part & 7)) TS_REFUSE(TS_ERR_ALIGN, "ts_glu_pairs: partial sums on 8-byte boundaries");
+  cudaStream_t s = (cudaStream_t)stream;
+  const TsGlu glu = {limit, slope, offset};
+  if (dtype == TS_BF16 && part == nullptr && total % 8 == 0 && !(((uintptr_t)out | (uintptr_t)gu) & 15)) {
+    const size_t total8 = total / 8;
+    const int vb = (int)((total8 + 255) / 256 < 148 * 32 ? (total8 + 255) / 256 : 148 * 32);
+    ts_launch(glu_pairs_vec_kernel, dim3(vb), dim3(256), 0, s, (bf16*)out, (const bf16*)gu, total8, glu);
+    TS_LAUNCH_CHECK();
+  }
+  const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+#define TS_GP(TT, P)                                                                                                    \
+  ts_launch(glu_pairs_kernel<TT, P>, dim3(blocks), dim3(256), 0, s, (TT*)out, (const TT*)gu, part, splits, 2 * total, total, glu)
+  if (dtype == TS_F32) { if (part != nullptr) TS_GP(float, true); else TS_GP(float, false); }
+  else if (dtype == TS_BF16) { if (part != nullptr) TS_GP(bf16, true); else TS_GP(bf16, false); }
+  else TS_REFUSE(TS_ERR_DTYPE, "ts_glu_pairs: dtype %d", dtype);
+#undef TS_GP
+  TS_LAUNCH_CHECK();
+}
 
 TS_API int ts_moe_tile_rows() { return GL_BM; }
 
@@ -492,12 +604,15 @@ TS_API int ts_router_topk(int* idx_out, float* w_out, const void* x, const float
 
 // tiles needs 1 + 2 * (ceil(P / tile_rows) + E) ints.
 // with_tiles: the experts [0, with_tiles) get row tiles (E: all of them).
+// table [table_rows, top] not null: idx holds the P / top token ids and the choices are the table's rows.
 TS_API int ts_moe_align(const int* idx, int P, int E, int* offsets, int* order, int* place, int* tiles, int with_tiles,
-                        void* stream) {
+                        const int* table, int top, int table_rows, void* stream) {
   if (P <= 0) return 0;
+  if (table != nullptr && (top < 1 || table_rows < 1 || P % top))
+    TS_REFUSE(TS_ERR_SHAPE, "ts_moe_align: %d pairs from a table of %d x %d", P, table_rows, top);
   if (E > 4096) TS_REFUSE(TS_ERR_LIMIT, "ts_moe_align: %d experts (limit 4096)", E);
   ts_launch(moe_align_kernel, dim3(1), dim3(1024), sizeof(int) * 2 * E, (cudaStream_t)stream, idx, P, E, offsets, order,
-            place, tiles, GL_BM, with_tiles);
+            place, tiles, GL_BM, with_tiles, table, top, table_rows);
   TS_LAUNCH_CHECK();
 }
 
@@ -515,23 +630,22 @@ TS_API int ts_moe_gather(void* xs, const void* x, const int* order, const float*
   TS_LAUNCH_CHECK();
 }
 
-// w: [E, N, K].  out: [P, N].  act: 0 none, 1 tanh-form GELU, 2 squared ReLU, 3 SiLU.
-TS_API int ts_grouped_linear(void* out, const void* x, const void* w, const int* order, const float* row_scale,
-                             const int* offsets, const int* tiles, int P, int E, int top, int N, int K, int act,
-                             int dtype, int out_dtype, void* stream) {
-  if (P <= 0 || N <= 0) return 0;
-  if (K <= 0) TS_REFUSE(TS_ERR_SHAPE, "ts_grouped_linear: K = %d", K);
-  cudaStream_t s = (cudaStream_t)stream;
+namespace {
+
+template <bool GLU>
+int launch_grouped(void* out, const void* x, const void* w, const int* order, const float* row_scale, const int* offsets,
+                   const int* tiles, int P, int E, int top, int N, int K, int act, TsGlu glu, int dtype, int out_dtype,
+                   cudaStream_t s) {
   dim3 grid(ceil_div(N, GL_BN), ceil_div(P, GL_BM) + E);
   if (grid.y > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_grouped_linear: %d rows too many for one launch", P);
   if (dtype == TS_BF16 && K % 8 == 0 && !(((uintptr_t)x | (uintptr_t)w) & 15) && P <= GV_STREAM_ROWS) {
     dim3 sgrid(ceil_div(N, GV_WARPS * 8), ceil_div(P, GL_BM) + E);
     if (out_dtype == TS_BF16)
-      ts_launch(grouped_linear_stream_kernel<bf16>, dim3(sgrid), dim3(GV_WARPS * 32), 0, s, (bf16*)out, (const bf16*)x,
-                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act);
+      ts_launch(grouped_linear_stream_kernel<bf16, GLU>, dim3(sgrid), dim3(GV_WARPS * 32), 0, s, (bf16*)out, (const bf16*)x,
+                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act, glu);
     else if (out_dtype == TS_F32)
-      ts_launch(grouped_linear_stream_kernel<float>, dim3(sgrid), dim3(GV_WARPS * 32), 0, s, (float*)out, (const bf16*)x,
-                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act);
+      ts_launch(grouped_linear_stream_kernel<float, GLU>, dim3(sgrid), dim3(GV_WARPS * 32), 0, s, (float*)out, (const bf16*)x,
+                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act, glu);
     else
       TS_REFUSE(TS_ERR_DTYPE, "ts_grouped_linear: dtype %d -> %d", dtype, out_dtype);
     TS_LAUNCH_CHECK();
@@ -540,30 +654,52 @@ TS_API int ts_grouped_linear(void* out, const void* x, const void* w, const int*
     const size_t smem = (size_t)GM_STAGES * (GM_BM + GM_BN) * GM_BK * 2;
     static bool configured = false;
     if (!configured) {
-      cudaError_t e1 = cudaFuncSetAttribute(grouped_linear_mma_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      cudaError_t e2 = cudaFuncSetAttribute(grouped_linear_mma_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      cudaError_t e1 = cudaFuncSetAttribute(grouped_linear_mma_kernel<bf16, GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      cudaError_t e2 = cudaFuncSetAttribute(grouped_linear_mma_kernel<float, GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e1 != cudaSuccess || e2 != cudaSuccess) TS_REFUSE((int)(e1 != cudaSuccess ? e1 : e2), "ts_grouped_linear: shared memory %zu", smem);
       configured = true;
     }
     if (out_dtype == TS_BF16)
-      ts_launch(grouped_linear_mma_kernel<bf16>, dim3(grid), dim3(GM_WARPS * 32), smem, s, (bf16*)out, (const bf16*)x,
-                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act);
+      ts_launch(grouped_linear_mma_kernel<bf16, GLU>, dim3(grid), dim3(GM_WARPS * 32), smem, s, (bf16*)out, (const bf16*)x,
+                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act, glu);
     else if (out_dtype == TS_F32)
-      ts_launch(grouped_linear_mma_kernel<float>, dim3(grid), dim3(GM_WARPS * 32), smem, s, (float*)out, (const bf16*)x,
-                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act);
+      ts_launch(grouped_linear_mma_kernel<float, GLU>, dim3(grid), dim3(GM_WARPS * 32), smem, s, (float*)out, (const bf16*)x,
+                (const bf16*)w, order, row_scale, offsets, tiles, top, N, K, act, glu);
     else
       TS_REFUSE(TS_ERR_DTYPE, "ts_grouped_linear: dtype %d -> %d", dtype, out_dtype);
     TS_LAUNCH_CHECK();
   }
 #define TS_GLK(TI, TO)                                                                                           \
-  ts_launch(grouped_linear_kernel<TI, TO>, dim3(grid), dim3(256), 0, s, (TO*)out, (const TI*)x, (const TI*)w, order, \
-            row_scale, offsets, tiles, top, N, K, act)
+  ts_launch(grouped_linear_kernel<TI, TO, GLU>, dim3(grid), dim3(256), 0, s, (TO*)out, (const TI*)x, (const TI*)w, order, \
+            row_scale, offsets, tiles, top, N, K, act, glu)
   if (dtype == TS_F32 && out_dtype == TS_F32) TS_GLK(float, float);
   else if (dtype == TS_BF16 && out_dtype == TS_BF16) TS_GLK(bf16, bf16);
   else if (dtype == TS_BF16 && out_dtype == TS_F32) TS_GLK(bf16, float);
   else TS_REFUSE(TS_ERR_DTYPE, "ts_grouped_linear: dtype %d -> %d", dtype, out_dtype);
 #undef TS_GLK
   TS_LAUNCH_CHECK();
+}
+
+}  // namespace
+
+// w: [E, N, K].  out: [P, N].  act: 0 none, 1 tanh-form GELU, 2 squared ReLU, 3 SiLU.
+TS_API int ts_grouped_linear(void* out, const void* x, const void* w, const int* order, const float* row_scale,
+                             const int* offsets, const int* tiles, int P, int E, int top, int N, int K, int act,
+                             int dtype, int out_dtype, void* stream) {
+  if (P <= 0 || N <= 0) return 0;
+  if (K <= 0) TS_REFUSE(TS_ERR_SHAPE, "ts_grouped_linear: K = %d", K);
+  return launch_grouped<false>(out, x, w, order, row_scale, offsets, tiles, P, E, top, N, K, act, TsGlu{0.f, 0.f, 0.f}, dtype,
+                               out_dtype, (cudaStream_t)stream);
+}
+
+// w: [E, N, K], its rows in turns a gate and its up; out: [P, N / 2].
+TS_API int ts_grouped_glu(void* out, const void* x, const void* w, const int* order, const float* row_scale,
+                          const int* offsets, const int* tiles, int P, int E, int top, int N, int K, float limit, float slope,
+                          float offset, int dtype, int out_dtype, void* stream) {
+  if (P <= 0 || N <= 0) return 0;
+  if (K <= 0 || N % 2) TS_REFUSE(TS_ERR_SHAPE, "ts_grouped_glu: N = %d, K = %d", N, K);
+  return launch_grouped<true>(out, x, w, order, row_scale, offsets, tiles, P, E, top, N, K, 0, TsGlu{limit, slope, offset}, dtype,
+                              out_dtype, (cudaStream_t)stream);
 }
 
 // x (out's type, [T, N]) and pass_from (one int on the device): pairs sorted to place *pass_from or later add the

@@ -68,7 +68,7 @@ class LazyProduct:
 class CudaOps:
     """ctypes front of ``libturingserve_b200.so``."""
 
-    ABI = 14
+    ABI = 15
     UNSUPPORTED = -4            # a kernel's refusal of a shape or layout another kernel takes
 
     def __init__(self, lib_path: str) -> None:
@@ -117,7 +117,7 @@ class CudaOps:
             "ts_attention_diff": [P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, F, F, I, P],
             "ts_attention_diff_mma": [P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, F, F, P, P, I, I, P],
             "ts_router_topk": [P, P, P, P, I, I, I, I, I, I, I, P, P],
-            "ts_moe_align": [P, I, I, P, P, P, P, I, P],
+            "ts_moe_align": [P, I, I, P, P, P, P, I, P, I, I, P],
             "ts_grouped_linear": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
             "ts_moe_combine": [P, P, P, P, I, I, I, I, P, P, P, P],
             "ts_hyper_norm": [P, P, P, P, I, P, P, P, P, P, F, I, I, I, I, F, I, P],
@@ -132,14 +132,25 @@ class CudaOps:
             "ts_delta_prepare": [P, P, I, P, P, P, P, ctypes.c_longlong, P, P, P, I, I, I, I, I, I, F, I, P],
             "ts_delta_scan": [P, P, P, I, P, ctypes.c_longlong, P, P, I, I, I, I, I, I, I, I, P],
             "ts_head_gated_rmsnorm": [P, P, P, I, P, F, I, I, I, I, P],
-            "ts_attention_biased": [P, I, I, P, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, I, I, P, P, I, I, P, P],
-            "ts_attention_biased_mma": [P, I, I, P, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, I, I, P, P, I, I, P, P],
+            "ts_attention_biased": [P, I, I, P, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, I, I, P, P, I, I, P, I, P, P, I, P],
+            "ts_attention_biased_mma": [P, I, I, P, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, I, I, P, P, I, I, P, I, P, P, I, P],
             "ts_rope_headnorm_write": [P, I, I, I, P, P, I, I, F, P, P, P, I, I, I, I, I, I, I, P, I, P],
             "ts_rope_headnorm_write_supports_parts": [I, I, I, I],
             "ts_rms_rows": [P, P, I, I, I, P, F, I, I, P],
             "ts_qk_rownorm_write": [P, I, P, P, F, P, F, I, P, P, P, I, I, I, I, I, I, P],
             "ts_latent_kv_write": [P, I, I, P, F, P, P, F, I, P, P, I, I, I, I, I, P],
             "ts_rotate_pairs": [P, I, I, P, I, I, P, P, F, I, I, I, I, I, P],
+            "ts_grouped_glu": [P, P, P, P, P, P, P, I, I, I, I, I, F, F, F, I, I, P],
+            "ts_glu_pairs": [P, P, P, I, I, I, F, F, F, I, P],
+            "ts_post_norm": [P, P, P, P, P, I, P, P, P, P, I, F, P, F, P, F, I, I, I, P],
+            "ts_qkv_heads_write": [P, I, I, I, P, P, P, F, P, F, I, I, P, P, P, P, I, I, I, I, I, I, I, P, I, I, I, P],
+            "ts_qkv_heads_supports_parts": [I, I, I, I, I, I, I, I],
+            "ts_short_filter": [P, I, P, I, I, P, P, P, ctypes.c_longlong, ctypes.c_longlong, P, P, P, I, I, I, I, P],
+            "ts_rglru_gates": [P, P, P, P, P, P, P, I, I, I, I, P],
+            "ts_rglru_scan": [P, P, P, I, I, I, P, ctypes.c_longlong, P, P, I, I, I, I, I, P],
+            "ts_rglru_step": [P, P, I, I, I, P, P, P, P, P, P, P, P, ctypes.c_longlong, P, I, I, I, I, P, I, P],
+            "ts_rglru_step_supported": [I, I, I, I],
+            "ts_rglru_step_counters": [I, I],
             "ts_batched_linear": [P, I, I, P, I, I, P, I, I, I, I, I, P],
         }
         for name, args in sigs.items():
@@ -783,19 +794,26 @@ class CudaOps:
     biased_decode_splits = int(os.environ.get("TURINGSERVE_B200_BIASED_DECODE_SPLITS", "0"))
 
     def attention_biased(self, out, q, k_cache, v_cache, block_tables, step, KVH: int, page_size: int, scale: float,
-                         softcap: float, slopes, window, chunk=None, sinks=None) -> None:
+                         softcap: float, slopes, window, chunk=None, sinks=None, keep: int = 0, out_freq=None,
+                         gate=None) -> None:
         """out [T, H, Dv] = softmax over the visible keys of cap tanh(q.k scale / cap) - slope_h (i - j), times the
         values; q [T, H, Dk] (views with unit last stride).  ``v_cache`` None: the values are the first Dv columns
         of the key rows.  ``softcap`` 0: none; ``slopes`` (float32 [H]) None: none; ``window`` None: none; ``chunk`` c:
-        position i sees only j >= floor(i / c) c; ``sinks`` (float32 [H]): exp(sink_h) joins the softmax's denominator.  The keys
-        of requests that bring one token are cut over several blocks when the step's longest context is long."""
+        position i sees only j >= floor(i / c) c; ``sinks`` (float32 [H]): exp(sink_h) joins the softmax's denominator;
+        ``keep``: with a window, the first ``keep`` positions stay visible.  On its way out a head's pairs (m, m + Dv/2) are
+        turned by -position * out_freq[m] (float32 [Dv / 2]) and the head is multiplied by sigmoid(gate[t, h]) (``gate`` [T, H] in
+        q's type, unit last stride).  The keys of requests that bring one token are cut over several blocks when the step's longest context is long."""
         T, H, Dk = q.shape
         Dv = out.shape[2]
         if out.stride(2) != 1 or q.stride(2) != 1:
             raise ValueError("attention_biased: rows must be contiguous")
         B = step.num_requests
         w = 0 if window is None else int(window)
-        reach = min(step.max_seq_len, w) if w else step.max_seq_len
+        keep = int(keep) if w else 0
+        reach = min(step.max_seq_len, w + keep) if w else step.max_seq_len
+        if gate is not None and (gate.stride(1) != 1 or gate.dtype != q.dtype):
+            raise ValueError("attention_biased: gates in the heads' type, rows contiguous")
+        gate_ts = 0 if gate is None else gate.stride(0)
         c = 0 if chunk is None else int(chunk)
         if c:
             reach = min(reach, c)
@@ -829,7 +847,7 @@ class CudaOps:
                     block_tables.data_ptr() + 4 * first * width, step.q_start.data_ptr() + 4 * first,
                     step.seq_lens.data_ptr() + 4 * first, count, width, max_q, H, KVH, Dk, Dv, page_size, float(scale),
                     float(softcap), _ptr(slopes), w, n_splits, _ptr(scratch), _ptr(counters), spread_flag, c, _ptr(sinks),
-                    self._stream())
+                    keep, _ptr(out_freq), _ptr(gate), gate_ts, self._stream())
 
             if spread:
                 rc = launch(0, nd, 1, ms, 1)
@@ -856,7 +874,7 @@ class CudaOps:
             _ptr(out), out.stride(0), out.stride(1), _ptr(q), q.stride(0), q.stride(1), _ptr(k_cache), _ptr(v_cache),
             _ptr(block_tables), _ptr(step.q_start), _ptr(step.seq_lens), B, block_tables.shape[1], step.max_q_len, H, KVH,
             Dk, Dv, page_size, float(scale), float(softcap), _ptr(slopes), w, splits, _ptr(scratch), _ptr(counters),
-            _code(q.dtype), c, _ptr(sinks), self._stream()), "attention_biased")
+            _code(q.dtype), c, _ptr(sinks), keep, _ptr(out_freq), _ptr(gate), gate_ts, self._stream()), "attention_biased")
 
     # -- a residual stream in several copies -------------------------------------------------------------------
     def hyper_norm(self, out, streams, y, mix, out_w, in_w, weight, eps: float, first: bool = False,
@@ -954,11 +972,12 @@ class CudaOps:
                                             1 if softmax else 0, 1 if renormalize else 0, _code(x.dtype), _ptr(correction),
                                             self._stream()), "router_topk")
 
-    def moe_align(self, idx, E: int, with_tiles: int | None = None):
-        """Sorts the (token, choice) pairs of ``idx`` by expert on the device.  Returns (offsets [E + 1],
+    def moe_align(self, idx, E: int, with_tiles: int | None = None, table=None):
+        """Sorts the (token, choice) pairs of ``idx`` by expert on the device; with ``table`` (int32 [rows, top]) ``idx`` holds
+        token ids and a token's choices are the table's row of its id.  Returns (offsets [E + 1],
         order [P], place [P], tiles): work buffers of this object, valid until the next call.  ``with_tiles``:
         only the experts below it get row tiles for the grouped products (the others have no weights)."""
-        P = idx.numel()
+        P = idx.numel() if table is None else idx.numel() * table.shape[1]
         dev = idx.device
         rows = self.lib.ts_moe_tile_rows()
         offsets = self._buffer("moe_offsets", E + 1, torch.int32, dev, floor=1024)
@@ -966,7 +985,9 @@ class CudaOps:
         place = self._buffer("moe_place", P, torch.int32, dev, floor=1 << 14)
         tiles = self._buffer("moe_tiles", 1 + 2 * (-(-P // rows) + E), torch.int32, dev, floor=1 << 12)
         self._check(self.lib.ts_moe_align(_ptr(idx), P, E, _ptr(offsets), _ptr(order), _ptr(place), _ptr(tiles),
-                                          E if with_tiles is None else int(with_tiles), self._stream()), "moe_align")
+                                          E if with_tiles is None else int(with_tiles), _ptr(table),
+                                          1 if table is None else table.shape[1], 0 if table is None else table.shape[0],
+                                          self._stream()), "moe_align")
         return offsets, order, place, tiles
 
     def grouped_linear(self, out, x, w, order, row_scale, offsets, tiles, top: int, act: str = "none") -> None:
@@ -977,6 +998,122 @@ class CudaOps:
         self._check(self.lib.ts_grouped_linear(_ptr(out), _ptr(x), _ptr(w), _ptr(order), _ptr(row_scale), _ptr(offsets),
                                                _ptr(tiles), P, E, top, N, K, self.ACTIVATIONS[act], _code(x.dtype),
                                                _code(out.dtype), self._stream()), "grouped_linear")
+
+    def grouped_glu(self, out, x, w, order, row_scale, offsets, tiles, top: int, glu) -> None:
+        """The grouped product whose weight rows are in turns a gate and its up (``w`` [E, 2 I, K]), with the clamped gated
+        unit in its epilogue: out [P, I] = g sigmoid(slope g) (u + offset), g = min(gate, limit), u = clamp(up, +-limit);
+        ``glu`` = (limit, slope, offset).  Operands as of ``grouped_linear``."""
+        P = out.shape[0]
+        E, N, K = w.shape
+        self._check(self.lib.ts_grouped_glu(_ptr(out), _ptr(x), _ptr(w), _ptr(order), _ptr(row_scale), _ptr(offsets),
+                                            _ptr(tiles), P, E, top, N, K, *(float(v) for v in glu), _code(x.dtype),
+                                            _code(out.dtype), self._stream()), "grouped_glu")
+
+    def glu_pairs(self, out, gu, glu) -> None:
+        """out [T, I] = the clamped gated unit of the column pairs (2 i, 2 i + 1) of ``gu`` [T, 2 I] (see ``grouped_glu``);
+        ``gu`` may be a product put off: its partial sums are summed on the way."""
+        gu = self._settle(gu)
+        part, splits = None, 0
+        if isinstance(gu, Deferred):
+            if gu.bias is None:
+                part, splits = gu.part, gu.splits
+            gu = gu.out if part is not None else self.materialize(gu)
+        T, inter = out.shape
+        self._check(self.lib.ts_glu_pairs(_ptr(out), _ptr(gu), _ptr(part), splits, T, inter, *(float(v) for v in glu),
+                                          _code(out.dtype), self._stream()), "glu_pairs")
+
+    # -- a norm on what a sublayer returns ---------------------------------------------------------------------
+    def post_norm(self, out, stream, y, weight, eps: float, base=None, rows=None, place=None, pair_weights=None,
+                  top: int = 1, scale: float = 1.0, next_weight=None, next_eps: float = 0.0) -> None:
+        """stream (float32 [T, h]) += norm(y) with norm(y) = y / sqrt(mean(y^2) + eps) * weight (``base`` [T, h]: the stream
+        starts as base + norm(y)); out = stream, or with ``next_weight`` its RMS norm times that; 32-bit, rounded once.
+        ``y``: a tensor or a product put off (its partial sums are summed here).  With ``rows`` (float32), ``place`` and
+        ``top`` what is normed is scale * sum_r (pair_weights[t, r]) rows[place[t top + r]], plus y when given."""
+        T, h = stream.shape
+        part, splits, bias = None, 0, None
+        if isinstance(y, (LazyProduct, Deferred)):
+            y = self._settle(y)
+            if isinstance(y, Deferred):
+                part, splits, bias, y = y.part, y.splits, y.bias, None
+        dt = next(t.dtype for t in (out, y, base, bias) if t is not None)
+        self._check(self.lib.ts_post_norm(_ptr(out), _ptr(stream), _ptr(base), _ptr(y), _ptr(part), splits, _ptr(bias),
+                                          _ptr(rows), _ptr(place), _ptr(pair_weights), int(top), float(scale), _ptr(weight),
+                                          float(eps), _ptr(next_weight), float(next_eps), T, h, _code(dt), self._stream()),
+                    "post_norm")
+
+    def qkv_heads_write(self, proj, k_off: int, v_off: int, positions, q_w, k_w, eps: float, freq, magnitude: float,
+                        rot_dims: int, v_norm: bool, v_freq, k_cache, v_cache, slots, H: int, G: int, D: int, V: int,
+                        page_size: int):
+        """``proj`` [T, ...]: q heads in the columns [0, H D), k heads from ``k_off``, value rows from ``v_off``, other columns
+        (gates) behind them.  q and k heads: RMS norm with the weights ``q_w`` / ``k_w`` (float32 [D]; None: none), then
+        dimension i < rot_dims / 2 turned with i + rot_dims / 2 by position * freq[i], cosine and sine times ``magnitude``.
+        Value heads: with ``v_norm`` over their root mean square, then with ``v_freq`` (float32 [V / 2]) the pairs (m, m + V/2)
+        turned by position * v_freq[m].  q in place, k and v to the caches at ``slots`` (None: nothing is cached).  ``proj`` may
+        be a product put off: the kernel then finishes its sum (of k and v only into the caches).  Returns the tensor."""
+        proj = self._settle(proj)
+        part, splits = None, 0
+        if isinstance(proj, Deferred):
+            d = proj
+            if (d.bias is None and self.lib.ts_qkv_heads_supports_parts(d.out.stride(0), k_off, v_off, D, V, int(rot_dims),
+                                                                        0 if v_freq is None else 1, _code(d.dtype))
+                    and all(t is None or t.data_ptr() % 16 == 0 for t in (d.out, d.part, k_cache, v_cache, q_w, k_w))):
+                part, splits, proj = d.part, d.splits, d.out
+            else:
+                proj = self.materialize(d)
+        extra = v_off + G * V
+        self._check(self.lib.ts_qkv_heads_write(
+            _ptr(proj), proj.stride(0), k_off, v_off, _ptr(positions), _ptr(q_w), _ptr(k_w), float(eps), _ptr(freq),
+            float(magnitude), int(rot_dims), 1 if v_norm else 0, _ptr(v_freq), _ptr(k_cache), _ptr(v_cache), _ptr(slots),
+            proj.shape[0], H, G, D, V, page_size, _code(proj.dtype), _ptr(part), splits, extra, proj.shape[1] - extra,
+            self._stream()), "qkv_heads_write")
+        return proj
+
+    # -- the real-gated linear recurrent unit ----------------------------------------------------------------------
+    def short_filter(self, out, x, x_off: int, conv_w, conv_b, state, tail_off: int, step, taps: int) -> None:
+        """out [T, W] = the columns x_off .. x_off + W of ``x`` through their causal filters (``conv_w`` float32 [W, taps], the
+        last column the present token's; ``conv_b`` float32 [W] or None); the inputs before the step's first token come from
+        the request's state slot, from ``tail_off`` on."""
+        T, W = out.shape
+        self._check(self.lib.ts_short_filter(_ptr(out), out.stride(0), _ptr(x), x.stride(0), x_off, _ptr(conv_w), _ptr(conv_b),
+                                             _ptr(state), state.stride(0), int(tail_off), _ptr(step.token_request),
+                                             _ptr(step.q_start), _ptr(step.state_slots), T, W, taps, _code(x.dtype),
+                                             self._stream()), "short_filter")
+
+    def rglru_gates(self, ab, u, ra, ri, ra_b, ri_b, rate) -> None:
+        """ab (float32 [T, W, 2]) = (a, sqrt(1 - a^2) i u) with a = exp(-rate r), r and i the sigmoids of the block-diagonal
+        products of ``u`` [T, W] with ``ra`` and ``ri`` [parts, size, size] plus ``ra_b`` / ``ri_b`` (float32 [W])."""
+        T, W = u.shape
+        self._check(self.lib.ts_rglru_gates(_ptr(ab), _ptr(u), _ptr(ra), _ptr(ri), _ptr(ra_b), _ptr(ri_b), _ptr(rate), T, W,
+                                            ra.shape[0], _code(u.dtype), self._stream()), "rglru_gates")
+
+    def rglru_scan(self, out, ab, proj, y_off: int, x_off: int, state, step, taps: int) -> None:
+        """out [T, W] = S gelu_tanh(y) with S <- a S + b over the pairs of ``rglru_gates``, y the columns of ``proj`` from
+        ``y_off``; ``state`` (float32 [slots, W + (taps - 1) W]) is read and left updated at each request's slot, the filter's
+        last inputs (the columns from ``x_off``) included."""
+        W = out.shape[1]
+        self._check(self.lib.ts_rglru_scan(_ptr(out), _ptr(ab), _ptr(proj), proj.stride(0), y_off, x_off, _ptr(state),
+                                           state.stride(0), _ptr(step.q_start), _ptr(step.state_slots), step.num_requests, W,
+                                           taps, int(getattr(step, "max_q_len", 0) or 0), _code(proj.dtype), self._stream()),
+                    "rglru_scan")
+
+    def rglru_step(self, out, proj, y_off: int, x_off: int, conv_w, conv_b, ra, ri, ra_b, ri_b, rate, state, step,
+                   taps: int) -> bool:
+        """The three above in one kernel, for a step in which every token is a request of its own.  False where the shape or
+        type is not one it takes (nothing has been launched then)."""
+        T, W = out.shape
+        parts = ra.shape[0]
+        if (step.max_q_len != 1 or step.num_requests != T
+                or not self.lib.ts_rglru_step_supported(W, parts, taps, _code(proj.dtype))):
+            return False
+        counters = self._buffer("rglru_counters", self.lib.ts_rglru_step_counters(T, parts), torch.int32, proj.device,
+                                floor=1 << 12, zero=True)
+        rc = self.lib.ts_rglru_step(_ptr(out), _ptr(proj), proj.stride(0), y_off, x_off, _ptr(conv_w), _ptr(conv_b), _ptr(ra),
+                                    _ptr(ri), _ptr(ra_b), _ptr(ri_b), _ptr(rate), _ptr(state), state.stride(0),
+                                    _ptr(step.state_slots), T, W, parts, taps, _ptr(counters), _code(proj.dtype), self._stream())
+        if rc == self.UNSUPPORTED:
+            return False
+        self._check(rc, "rglru_step")
+        return True
 
     def moe_gather(self, xs, x, order, row_scale, top: int) -> None:
         """xs[i] = x[order[i] // top] (times row_scale[order[i]], rounded to x's type): the experts' input rows

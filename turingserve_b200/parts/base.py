@@ -13,7 +13,7 @@ Norm            forward(x, residual=None) -> y          (residual updated in pla
                                                          or turns into a tensor with ops().materialize)
 PositionEncoding  tables()/apply are private to the mixers that accept it
 Mixer           forward(x, step, cache, state) -> y     cache_need() / state_need() declare memory
-FeedForward     forward(x) -> y                         (mixers and feed-forwards get tensors; they may
+FeedForward     forward(x) -> y                         (forward(x, step) where ``wants_step``; mixers and feed-forwards get tensors; they may
                                                          return what ops().linear(..., may_defer=True) gave)
 Block           forward(h, residual, step, cache, state) -> (h, residual)   (h is whatever the arrangement's own
                                                          norm takes: a tensor, a product put off, a ``BranchSum``)
@@ -41,13 +41,16 @@ class ParamSpec:
     shape: tuple[int, ...]
     compute_dtype: bool = True
     integer: bool = False
-    init: str = "normal"            # "normal" | "ones" | "zeros" | "identity": how the random-weights mode fills it
+    # how the random-weights mode fills it: "normal" | "ones" | "zeros" | "identity"; an integer table: "zeros", or
+    # "distinct": every row so many different numbers below ``high``
+    init: str = "normal"
+    high: int = 0
 
 
 @dataclass(frozen=True)
 class CacheNeed:
     """What a mixer wants from the paged cache: keys and values of ``num_kv_heads`` x ``head_dim``
-    per token; ``window`` None keeps every token, an integer keeps the last ``window`` of them.
+    per token; ``window`` None keeps every token, an integer keeps the last ``window`` of them (and the first ``keep_first``).
     ``value_dim``: the width of a value row where it differs from a key row's ``head_dim`` (the
     group's keys and values are then two tensors instead of one pool).  ``chunk`` c: a position sees only
     the keys of its own block of c positions (blocks counted from position 0), so tokens before the block of
@@ -58,6 +61,7 @@ class CacheNeed:
     window: int | None = None
     value_dim: int | None = None
     chunk: int | None = None
+    keep_first: int = 0             # with a window: the first so many tokens stay visible, so they are kept too
 
     @property
     def v_dim(self) -> int:
@@ -116,8 +120,16 @@ class Mixer(Part):
 
 
 class FeedForward(Part):
+    # whether ``forward`` also wants the step (a feed-forward that looks at the tokens' ids); the block then calls
+    # forward(x, step)
+    wants_step = False
+
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
+
+    def forward_pending(self, x: torch.Tensor, step):
+        """The output as a norm that finishes sums may take it: what ``forward`` gives, or a ``RoutedSum``."""
+        return self.forward(x, step) if self.wants_step else self.forward(x)
 
 
 @dataclass
@@ -130,6 +142,32 @@ class BranchSum:
     first: Any
     second: Any = None
     scale: float = 1.0
+
+
+@dataclass
+class RoutedSum:
+    """What a routed feed-forward leaves before its last kernel: the experts' output rows (float32, sorted by expert), the
+    sorted place of every (token, choice) pair, the weights (one per pair, or None) and a constant, and the output of an
+    expert that every token uses (``add``: a tensor, a product put off or None).  Valid until the next routed feed-forward
+    runs (``place`` is a work buffer of the kernels)."""
+
+    rows: torch.Tensor
+    place: torch.Tensor
+    top: int
+    pair_weights: Any = None
+    scale: float = 1.0
+    add: Any = None
+
+
+@dataclass
+class NormedUpdate:
+    """What a sublayer whose OUTPUT is normed leaves pending: the output ``y`` (a tensor, a product put off or a
+    ``RoutedSum``) and the norm (``parts.rmsnorm.PostRMSNorm``) through which it enters the stream.  ``base``: the rows the
+    stream starts from (where this is the model's first update)."""
+
+    y: Any
+    norm: Any
+    base: Any = None
 
 
 @dataclass
@@ -183,7 +221,7 @@ def _load_builtin() -> None:
         _loaded = True
         from turingserve_b200.parts import (  # noqa: F401
             attention, block, capped_attention, delta_rule, diff_attention, gated_mlp, latent_attention, lightning, mamba2,
-            mlp, paired_mixer, rmsnorm, rotary, routed_mlp, sink_attention, stream_link)
+            mlp, normed_attention, paired_mixer, rglru, rmsnorm, rotary, routed_mlp, sink_attention, stream_link)
 
 
 def build_block(layer_spec: Any, ctx: BuildContext):

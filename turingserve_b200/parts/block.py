@@ -10,7 +10,12 @@ from __future__ import annotations
 import torch
 
 from turingserve_b200 import kernels
-from turingserve_b200.parts.base import BranchSum, BuildContext, StreamUpdate, build, register
+from turingserve_b200.parts.base import BranchSum, BuildContext, NormedUpdate, StreamUpdate, build, register
+
+
+def _feed(ff, x, step):
+    """A feed-forward's output; one that looks at the tokens gets the step."""
+    return ff.forward(x, step) if getattr(ff, "wants_step", False) else ff.forward(x)
 
 
 class PreNormBlock:
@@ -36,7 +41,7 @@ class PreNormBlock:
             x = self.mixer_norm.forward(h, residual)
         a = self.mixer.forward(x, step, cache, state)
         x = self.ffn_norm.forward(a, residual)
-        h = self.feed_forward.forward(x)
+        h = _feed(self.feed_forward, x, step)
         return h, residual
 
 
@@ -71,7 +76,7 @@ class StreamBlock:
         h = self.mixer.forward(x, step, cache, state)
         if self.has_ff:
             x = self.ffn_norm.forward(h, residual)
-            h = self.feed_forward.forward(x)
+            h = _feed(self.feed_forward, x, step)
         return h, residual
 
 
@@ -106,7 +111,7 @@ class ParallelBlock:
             # a product whose partial sums already sit in the work buffer that all such products share: the
             # feed-forward's last product would write over them, so this one is finished first
             a = kernels.ops().materialize(a)
-        b = self.feed_forward.forward(x) if self.has_ff else None
+        b = _feed(self.feed_forward, x, step) if self.has_ff else None
         return BranchSum(a, b, self.scale), residual
 
 
@@ -147,11 +152,48 @@ class HyperBlock:
         pending = StreamUpdate(self.mixer.forward(x, step, cache, state), self.mixer_link)
         if self.has_ff:
             x = self.ffn_norm.forward(pending, residual, self.ffn_link)
-            pending = StreamUpdate(self.feed_forward.forward(x), self.ffn_link)
+            pending = StreamUpdate(_feed(self.feed_forward, x, step), self.ffn_link)
         return pending, residual
 
 
+class PostNormBlock:
+    """Norms on the sublayers' outputs only, over a residual stream in 32-bit: x <- x + norm(mixer(x)),
+    x <- x + norm(ff(x)); the sublayers read x itself, rounded to the engine's type.  Each norm and its add are put off into
+    the kernel that gives the next sublayer its input: the block carries (the embedding rows before the first layer,
+    then a ``NormedUpdate``; the stream).  Roles: ``mixer``, ``mixer_norm`` and, where the layer has a feed-forward,
+    ``feed_forward``, ``ffn_norm``."""
+
+    def __init__(self, spec, ctx: BuildContext) -> None:
+        self.mixer_norm = build("norm", spec.mixer_norm, ctx)
+        self.mixer = build("mixer", spec.mixer, ctx)
+        self.has_ff = "feed_forward" in spec.roles
+        self.ffn_norm = build("norm", spec.ffn_norm, ctx) if self.has_ff else None
+        self.feed_forward = build("feed_forward", spec.feed_forward, ctx) if self.has_ff else None
+
+    def parts(self) -> dict[str, object]:
+        p = {"mixer_norm": self.mixer_norm, "mixer": self.mixer}
+        if self.has_ff:
+            p.update(ffn_norm=self.ffn_norm, feed_forward=self.feed_forward)
+        return p
+
+    def forward(self, h, residual, step, cache, state, inject=None):
+        if inject is not None:
+            raise ValueError("post_norm_stream: nothing is injected into the stream")
+        base = None
+        if isinstance(h, NormedUpdate):
+            x = h.norm.forward(h.y, residual, base=h.base)
+        else:                                             # the embedding rows: the first update starts the stream from them
+            x = base = h
+            residual = torch.empty(h.shape, dtype=torch.float32, device=h.device)
+        y = self.mixer.forward(x, step, cache, state)
+        if not self.has_ff:
+            return NormedUpdate(y, self.mixer_norm, base), residual
+        x = self.mixer_norm.forward(y, residual, base=base)
+        return NormedUpdate(self.feed_forward.forward_pending(x, step), self.ffn_norm), residual
+
+
 register("block", "pre_norm", _build_block)
+register("block", "post_norm_stream", lambda spec, ctx: PostNormBlock(spec, ctx))
 register("block", "hyper_streams", lambda spec, ctx: HyperBlock(spec, ctx))
 register("block", "parallel", lambda spec, ctx: ParallelBlock(spec, ctx))
 register("block", "pre_norm_stream", lambda spec, ctx: StreamBlock(spec, ctx))

@@ -10,7 +10,7 @@ from __future__ import annotations
 import torch
 
 from turingserve_b200 import kernels
-from turingserve_b200.parts.base import BranchSum, BuildContext, Norm, ParamSpec, StreamUpdate, register
+from turingserve_b200.parts.base import BranchSum, BuildContext, Norm, ParamSpec, RoutedSum, StreamUpdate, register
 
 
 class RMSNorm(Norm):
@@ -140,7 +140,43 @@ class HyperRMSNorm(Norm):
         return out
 
 
+class PostRMSNorm(Norm):
+    """The norm of what a sublayer returns, over a residual stream kept in 32-bit.  ``forward(y, stream)``: stream +=
+    y / sqrt(mean(y^2) + eps) * (weight_offset + weight) in place (``base``: the stream starts as these rows plus that), then
+    the stream in the engine's type; with ``reader`` (another norm of this kind) the stream's own RMS norm with the reader's
+    weight instead, which is what a model's last norm reads.  ``y``: a tensor, a product put off, or a ``RoutedSum``, whose sum
+    is taken in the same kernel.  32-bit arithmetic, one rounding."""
+
+    def __init__(self, spec, ctx: BuildContext) -> None:
+        self.eps = float(spec.eps)
+        self.size = ctx.hidden_size
+        self.dtype = ctx.dtype
+        self.offset = float(spec.weight_offset)
+        self.weight_name = str(spec.weight_name)
+        self.weight: torch.Tensor | None = None
+
+    def parameters(self) -> dict[str, ParamSpec]:
+        return {self.weight_name: ParamSpec((self.size,), compute_dtype=False, init="zeros" if self.offset else "ones")}
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        self.weight = (tensors[self.weight_name].float() + self.offset).contiguous()
+
+    def forward(self, y, residual: torch.Tensor | None = None, base=None, reader: "PostRMSNorm | None" = None) -> torch.Tensor:
+        if residual is None:
+            raise ValueError("the norm of a sublayer's output needs the 32-bit stream it adds to")
+        out = torch.empty(residual.shape, dtype=self.dtype, device=residual.device)
+        kw = {}
+        if reader is not None:
+            kw.update(next_weight=reader.weight, next_eps=reader.eps)
+        if isinstance(y, RoutedSum):
+            kw.update(rows=y.rows, place=y.place, pair_weights=y.pair_weights, top=y.top, scale=y.scale)
+            y = y.add
+        kernels.ops().post_norm(out, residual, y, self.weight, self.eps, base=base, **kw)
+        return out
+
+
 register("norm", "rmsnorm", RMSNorm)
+register("norm", "rmsnorm_post", PostRMSNorm)
 register("norm", "rmsnorm_hyper", HyperRMSNorm)
 register("norm", "layernorm_stream", StreamLayerNorm)
 register("norm", "rmsnorm_stream", StreamRMSNorm)

@@ -31,7 +31,8 @@ class RotaryEncoding:
 
 
 class PairRotaryEncoding:
-    """Rotation of neighbouring pairs (2i, 2i+1) with YaRN-blended frequencies.  No table over positions:
+    """Rotation of neighbouring pairs (2i, 2i+1), or, with the spec's ``pairing`` "halves", of the pairs (i, i + dims / 2),
+    with YaRN-blended frequencies.  No table over positions:
     the kernels take the angle as position * ``freq[i]`` in 32-bit and multiply cosine and sine by
     ``magnitude``, so no longest sequence has to be known.  ``freq`` is float32 [dims / 2] on the device."""
 
@@ -39,6 +40,9 @@ class PairRotaryEncoding:
         self.dims = int(spec.dims)
         if self.dims % 2 or self.dims <= 0:
             raise ValueError("the rotated dimensions come in pairs")
+        self.pairing = str(getattr(spec, "pairing", "neighbours"))
+        if self.pairing not in ("neighbours", "halves"):
+            raise ValueError(f"yarn_pairs: unknown pairing {self.pairing!r}")
         base = float(spec.base)
         i = torch.arange(self.dims // 2, dtype=torch.float64)
         f = base ** (-2.0 * i / self.dims)
@@ -98,7 +102,6 @@ class BandScaledPairEncoding:
 
 
 HalfRotaryEncoding.pairing = "halves"
-PairRotaryEncoding.pairing = "neighbours"
 
 register("position", "rope", RotaryEncoding)
 register("position", "rope_pairs_banded", BandScaledPairEncoding)

@@ -21,7 +21,19 @@ from safetensors.torch import save_file
 
 from turingserve_b200.config.model_config import ModelConfig
 from turingserve_b200.config.registry import get_architecture
+from turingserve_b200.parts.base import ParamSpec
 from turingserve_b200.parts.model import DecoderModel
+
+
+def _random_table(spec: ParamSpec, g: torch.Generator, device) -> torch.Tensor:
+    """An integer table: zeros, or ("distinct") rows of different numbers below ``spec.high``."""
+    if spec.init != "distinct":
+        return torch.zeros(spec.shape, dtype=torch.int32, device=device)
+    rows, n = spec.shape
+    if n > spec.high:
+        raise ValueError(f"{n} different numbers below {spec.high}")
+    draws = torch.rand((rows, spec.high), generator=g, device=device)
+    return draws.argsort(dim=1)[:, :n].to(torch.int32).contiguous()
 
 
 def random_tensors(cfg: ModelConfig, seed: int, std: float = 0.02,
@@ -33,7 +45,7 @@ def random_tensors(cfg: ModelConfig, seed: int, std: float = 0.02,
     out: dict[str, torch.Tensor] = {}
     for name, spec in shell.parameters(names).items():
         if spec.integer:
-            out[name] = torch.zeros(spec.shape, dtype=torch.int32)
+            out[name] = _random_table(spec, g, "cpu")
         elif spec.init == "ones":
             out[name] = torch.ones(spec.shape, dtype=dtype)
         elif spec.init == "zeros":
@@ -70,7 +82,7 @@ def random_model_on_device(cfg: ModelConfig, dtype: torch.dtype, device, seed: i
     for name, spec in model.parameters(names).items():
         kind = dtype if spec.compute_dtype else torch.float32
         if spec.integer:
-            tensors[name] = torch.zeros(spec.shape, dtype=torch.int32, device=device)
+            tensors[name] = _random_table(spec, g, device)
         elif spec.init == "ones":
             tensors[name] = torch.ones(spec.shape, dtype=kind, device=device)
         elif spec.init == "zeros":
