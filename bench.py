@@ -1135,6 +1135,193 @@ def gugezen_kernels(ops, z: dict, pk: dict, T: int, B: int, ctx: int, page: int)
     return out
 
 
+# ---- Suranex (norms on the sublayers' outputs, attention with normed heads, turned values, a window that keeps the first
+# tokens and a gate per head, the real-gated linear recurrent unit, experts chosen by a table of token ids beside a shared
+# expert) beside Gugezen layers of the same width and about the same number of weights ----------------------------------
+SURANEX_SIZES = {
+    # width; attention: heads, kv heads, head width (keys and values), window, kept first tokens; recurrent unit: width,
+    # parts, taps; experts, top, expert ff, shared expert ff; the Gugezen size beside it
+    "1.5b": dict(width=1536, heads=12, kv_heads=2, dim=128, size=1024, keep=64, rwidth=2048, blocks=8, taps=4, experts=8, top=2,
+                 eff=1536, shared=1536, beside="1.5b"),
+    "7b": dict(width=3584, heads=28, kv_heads=4, dim=128, size=1024, keep=64, rwidth=4096, blocks=16, taps=4, experts=8, top=2,
+               eff=3584, shared=3584, beside="7b"),
+}
+
+
+def suranex_config(z: dict, groups: int, vocab: int):
+    """``groups`` times four layers, all with routed feed-forwards: recurrent, attention, recurrent, attention."""
+    from turingserve_b200.models.suranex import make_config
+    moe = {"kind": "moe", "expert": {"ff": z["eff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]},
+           "shared": {"ff": z["shared"], "limit": 6.0}}
+    att = {"type": "attention", "mlp": moe, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5, "softcap": 50.0,
+        "mask": {"size": z["size"], "keep_first": z["keep"]},
+        "rot": {"base": 500000.0, "dims": z["dim"], "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    rec = {"type": "rglru", "mlp": moe, "mixer": {"width": z["rwidth"], "blocks": z["blocks"], "conv": z["taps"]}}
+    return make_config(width=z["width"], vocab=vocab, layers=[rec, att, rec, att] * groups, eps=1e-6)
+
+
+def suranex_kernels(ops, z: dict, pk: dict, T: int, B: int, ctx: int, page: int) -> dict:
+    """Each kernel of the new mechanisms alone, beside the like kernel of the closest design: a portion of T tokens and B
+    single tokens at context ``ctx``."""
+    import torch
+    from types import SimpleNamespace
+    dev = torch.device("cuda", 0)
+    big = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    flush = lambda: big.fill_(1)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    out = {}
+    hbm = pk["hbm_gbs"] * 1e9
+    bf = torch.bfloat16
+    W, H, G, D = z["width"], z["heads"], z["kv_heads"], z["dim"]
+    us = lambda ms: round(ms * 1e3, 1)
+    frac = lambda byts, ms: round(byts / (ms / 1e3) / hbm, 3)
+    tensor = lambda flops, ms: round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 3)
+
+    # the norm of a sublayer's output + its add (from a tensor, and from a routed feed-forward's rows), beside the stream
+    # norm and the sum of a token's choices
+    E, top, ff = z["experts"], z["top"], z["eff"]
+    vocab = 32768
+    table = torch.rand(vocab, E, device=dev).argsort(1)[:, :top].to(torch.int32).contiguous()
+    for name, rows in (("prefill", T), ("decode", B)):
+        stream = torch.randn(rows, W, device=dev)
+        y = torch.randn(rows, W, device=dev).to(bf)
+        w_ = torch.ones(W, device=dev)
+        o = torch.empty(rows, W, dtype=bf, device=dev)
+        ms = timed(lambda: ops.post_norm(o, stream, y, w_, 1e-6), flush)
+        ms_r = timed(lambda: ops.rmsnorm_stream(o, stream, y, None, w_, 1e-6, False), flush)
+        ids = torch.randint(0, vocab, (rows,), dtype=torch.int32, device=dev)
+        offsets, order, place, tiles = ops.moe_align(ids, E, table=table)
+        er = torch.randn(rows * top, W, device=dev)
+        wts = torch.full((rows, top), 1.0 / top, device=dev)
+        ms_s = timed(lambda: ops.post_norm(o, stream, y, w_, 1e-6, rows=er, place=place, top=top, scale=1.0 / top), flush)
+        ms_c = timed(lambda: ops.moe_combine(o, er, place, wts, top, add=y), flush)
+        out[f"output_norm_{name}"] = {
+            "us": us(ms), "frac_of_hbm": frac(rows * W * 12.0, ms), "beside_stream_norm_us": us(ms_r),
+            "beside_frac_of_hbm": frac(rows * W * 12.0, ms_r), "with_choices_us": us(ms_s),
+            "with_choices_frac_of_hbm": frac(rows * W * (12.0 + 4 * top), ms_s), "beside_sum_of_choices_us": us(ms_c),
+            "beside_sum_frac_of_hbm": frac(rows * W * (4.0 + 4 * top), ms_c)}
+
+    pages = B * (-(-(ctx + 1) // page)) + -(-T // page) + 2
+    width = -(-max(ctx + 1, T) // page)
+    kc = torch.randn(pages, G, page, D, device=dev).to(bf)
+    vc = torch.randn(pages, G, page, D, device=dev).to(bf)
+    # norms, rotations and cache write of q, k and v, beside the rotation by halves with the per-head norm
+    freq = (500000.0 ** (-2.0 * torch.arange(D // 2, dtype=torch.float64) / D)).float().to(dev)
+    hw = torch.ones(D, device=dev)
+    n_in = -(-((H + 2 * G) * D + H) // 8) * 8
+    for name, rows in (("prefill", T), ("decode", B)):
+        proj = torch.randn(rows, n_in, device=dev).to(bf)
+        pos, slots = i32(list(range(rows))), i32(list(range(page, page + rows)))
+        ms = timed(lambda: ops.qkv_heads_write(proj, H * D, (H + G) * D, pos, hw, hw, 1e-6, freq, 1.2, D, True, freq, kc, vc, slots,
+                                               H, G, D, D, page), flush)
+        ms_h = timed(lambda: ops.rope_headnorm_write(proj, H * D, (H + G) * D, pos, freq, D, 1e-6, kc, vc, slots, H, G, D, D, page), flush)
+        byts = rows * (2 * H * D + 2 * 2 * G * D) * 2.0
+        out[f"norm_rotate_write_{name}"] = {"us": us(ms), "frac_of_hbm": frac(byts, ms), "beside_rotation_and_norm_us": us(ms_h),
+                                            "beside_frac_of_hbm": frac(byts, ms_h)}
+
+    # attention: window with kept first tokens, cap, outputs turned back and gated; without the window; beside it the plain
+    # sink attention of the closest design
+    sinks = torch.zeros(H, device=dev)
+    for name, reqs, per, seq in (("prefill", 1, T, T), ("decode", B, 1, ctx + 1)):
+        rows = reqs * per
+        q = torch.randn(rows, H, D, device=dev).to(bf)
+        o = torch.empty(rows, H, D, dtype=bf, device=dev)
+        gate = torch.randn(rows, n_in, device=dev).to(bf)[:, n_in - H:]
+        bt = torch.zeros(reqs, width, dtype=torch.int32, device=dev)
+        n = -(-seq // page)
+        for r in range(reqs):
+            bt[r, :n] = torch.arange(1 + r * n, 1 + (r + 1) * n, dtype=torch.int32, device=dev)
+        step = SimpleNamespace(q_start=i32([i * per for i in range(reqs + 1)]), seq_lens=i32([seq] * reqs), num_requests=reqs,
+                               num_decode=reqs if per == 1 else 0, max_q_len=per, max_seq_len=seq)
+        entry = {}
+        for tag, w, keep, mine in (("", z["size"], z["keep"], True), ("no_window_", None, 0, True), ("beside_sink_attention_", None, 0, False)):
+            kw = dict(keep=keep, out_freq=freq, gate=gate) if mine else dict(sinks=sinks)
+            cap = 50.0 if mine else 0.0
+            ms = timed(lambda: ops.attention_biased(o, q, kc, vc, bt, step, G, page, D ** -0.5, cap, None, w, **kw), flush)
+            seen = sum(min(i + 1, w + min(keep, max(0, i + 1 - w))) if w else i + 1 for i in range(seq - per, seq))
+            held = min(seq, w + keep) if w and per == 1 else seq
+            flops = 4.0 * D * H * seen * reqs
+            entry.update({tag + "us": us(ms), tag + "tflops": round(flops / ms / 1e9, 1), tag + "frac_of_bf16": tensor(flops, ms),
+                          tag + "frac_of_hbm": frac(reqs * held * G * 2 * D * 2.0 + rows * H * D * 4.0, ms)})
+        out[f"attention_{name}"] = entry
+
+    # the recurrent unit: filter, gates, scan (or, single tokens, one kernel), beside the state-space mixer of the closest
+    # design at its own size
+    R, parts, taps = z["rwidth"], z["blocks"], z["taps"]
+    bs = R // parts
+    conv, conv_b = torch.randn(R, taps, device=dev) * 0.3, torch.zeros(R, device=dev)
+    ra, ri = ((torch.randn(parts, bs, bs, device=dev) * 0.05).to(bf) for _ in range(2))
+    zero, rate = torch.zeros(R, device=dev), torch.full((R,), 0.5, device=dev)
+    g = GUGEZEN_SIZES[z["beside"]]
+    SH, P, N, SG = g["sheads"], g["sdim"], g["state"], g["sgroups"]
+    inner, channels = SH * P, SH * P + 2 * SG * N
+    for name, reqs, per in (("prefill", 1, T), ("decode", B, 1)):
+        rows = reqs * per
+        proj = torch.randn(rows, 2 * R, device=dev).to(bf)
+        state = torch.zeros(reqs + 1, (1 + taps) * R, device=dev)
+        step = SimpleNamespace(q_start=i32([i * per for i in range(reqs + 1)]), state_slots=i32(list(range(reqs))), num_requests=reqs,
+                               token_request=i32([r for r in range(reqs) for _ in range(per)]), max_q_len=per,
+                               positions=i32([ctx if per == 1 else t for _ in range(reqs) for t in range(per)]))
+        u, s_ = (torch.empty(rows, R, dtype=bf, device=dev) for _ in range(2))
+        ab = torch.empty(rows, R, 2, device=dev)
+        ms_f = timed(lambda: ops.short_filter(u, proj, R, conv, conv_b, state, R, step, taps), flush)
+        ms_g = timed(lambda: ops.rglru_gates(ab, u, ra, ri, zero, zero, rate), flush)
+        ms_s = timed(lambda: ops.rglru_scan(s_, ab, proj, 0, R, state, step, taps), flush)
+        flops = 2.0 * 2 * rows * R * bs
+        entry = {"filter_us": us(ms_f), "filter_frac_of_hbm": frac(rows * R * 4.0, ms_f), "gates_us": us(ms_g),
+                 "gates_tflops": round(flops / ms_g / 1e9, 1), "gates_frac_of_bf16": tensor(flops, ms_g),
+                 "gates_frac_of_hbm": frac(rows * R * 10.0 + 2 * R * bs * 2.0, ms_g), "scan_us": us(ms_s),
+                 "scan_frac_of_hbm": frac(rows * R * 12.0 + reqs * R * 8.0, ms_s)}
+        if per == 1:
+            ms_1 = timed(lambda: ops.rglru_step(s_, proj, 0, R, conv, conv_b, ra, ri, zero, zero, rate, state, step, taps), flush)
+            entry.update({"step_us": us(ms_1), "step_frac_of_hbm": frac(2 * R * bs * 2.0 + rows * R * (6.0 + 8.0 + 4.0 * taps), ms_1)})
+        gproj = torch.randn(rows, 2 * inner + 2 * SG * N + SH, device=dev).to(bf)
+        gstate = torch.zeros(reqs + 1, SH * N * P + (taps - 1) * channels, device=dev)
+        ready = torch.empty(rows, channels + 2 * SH, device=dev)
+        yy = torch.empty(rows, inner, device=dev)
+        gw, gb, hz = torch.randn(channels, taps, device=dev) * 0.3, torch.zeros(channels, device=dev), torch.zeros(SH, device=dev)
+        ms_p = timed(lambda: ops.ssm_prepare(ready, gproj, inner, inner + channels, gw, gb, hz, hz, gstate, SH * N * P, step, SH,
+                                             channels, taps), flush)
+        ms_q = timed(lambda: ops.ssm_scan(yy, ready, gproj, inner, gstate, hz, step, SH, SG, N, P, taps), flush)
+        entry.update({"beside_ssm_prepare_us": us(ms_p), "beside_prepare_frac_of_hbm": frac(rows * (channels * 6.0 + 8 * SH), ms_p),
+                      "beside_ssm_scan_us": us(ms_q),
+                      "beside_scan_frac_of_hbm": frac(reqs * SH * N * P * 8.0 + rows * (channels + inner) * 4.0, ms_q)})
+        out[f"recurrent_unit_{name}"] = entry
+
+    # the routed feed-forward: sort by the table (beside router + sort), the experts' products, the shared expert's activation
+    wr = torch.randn(E, W, device=dev) * 0.05
+    w_up = (torch.randn(E, 2 * ff, W, device=dev) * 0.02).to(bf)
+    w_down = (torch.randn(E, W, ff, device=dev) * 0.02).to(bf)
+    glu = (7.0, 1.702, 1.0)
+    for name, rows in (("prefill", T), ("decode", B)):
+        x = torch.randn(rows, W, device=dev).to(bf)
+        ids = torch.randint(0, vocab, (rows,), dtype=torch.int32, device=dev)
+        idx, wts = torch.empty(rows, top, dtype=torch.int32, device=dev), torch.empty(rows, top, device=dev)
+        ms_r = timed(lambda: (ops.router_topk(idx, wts, x, wr, True, True), ops.moe_align(idx, E)), flush)
+        ms_t = timed(lambda: ops.moe_align(ids, E, table=table), flush)
+        offsets, order, place, tiles = ops.moe_align(ids, E, table=table)
+        a_ = torch.empty(rows * top, ff, dtype=bf, device=dev)
+        a2 = torch.empty(rows * top, 2 * ff, dtype=bf, device=dev)
+        y = torch.empty(rows * top, W, device=dev)
+        ms_u = timed(lambda: ops.grouped_glu(a_, x, w_up, order, None, offsets, tiles, top, glu), flush)
+        ms_u2 = timed(lambda: ops.grouped_linear(a2, x, w_up, order, None, offsets, tiles, top), flush)
+        ms_d = timed(lambda: ops.grouped_linear(y, a_, w_down, None, None, offsets, tiles, 1), flush)
+        gu = torch.randn(rows, 2 * z["shared"], device=dev).to(bf)
+        sa = torch.empty(rows, z["shared"], dtype=bf, device=dev)
+        ms_a = timed(lambda: ops.glu_pairs(sa, gu, glu), flush)
+        ms_b = timed(lambda: ops.silu_mul(sa, gu, 64 if z["shared"] % 64 == 0 else 0), flush)
+        used = int((offsets[1:E + 1] > offsets[:E]).sum())
+        fl = 4.0 * rows * top * ff * W
+        out[f"routed_ff_{name}"] = {
+            "sort_by_table_us": us(ms_t), "beside_router_and_sort_us": us(ms_r), "up_with_unit_us": us(ms_u),
+            "up_frac_of_bf16": tensor(fl, ms_u), "up_frac_of_hbm": frac(used * 2 * ff * W * 2.0, ms_u), "beside_plain_up_us": us(ms_u2),
+            "down_us": us(ms_d), "down_frac_of_bf16": tensor(fl / 2, ms_d), "down_frac_of_hbm": frac(used * ff * W * 2.0, ms_d),
+            "shared_unit_us": us(ms_a), "shared_unit_frac_of_hbm": frac(rows * z["shared"] * 6.0, ms_a),
+            "beside_silu_us": us(ms_b), "beside_silu_frac_of_hbm": frac(rows * z["shared"] * 6.0, ms_b)}
+    return out
+
+
 def run_design(a) -> dict:
     """``--design komirax``: prefill and decode throughput of Komirax layers beside Qwen2 layers of the same
     width and count (random weights, bfloat16, through the step function), and each new kernel alone."""
@@ -1234,6 +1421,24 @@ def run_design(a) -> dict:
                      "decode_ratio": round(ours["decode_tok_s"] / beside["decode_tok_s"], 3)}
             if "kernels" in a.phases.split(","):
                 entry["kernels"] = gugezen_kernels(ops, z, pk, T, B, ctx, page)
+            result["sizes"][name] = entry
+            continue
+        if a.design == "suranex":
+            # beside Gugezen layers of the same width and about the same weight count, the closest design the engine has (a
+            # recurrent mixer with causal filters, a gated attention, routed feed-forwards with a shared expert, a 32-bit stream)
+            z = SURANEX_SIZES[name]
+            made = (("suranex", suranex_config(z, groups, vocab)), ("gugezen", gugezen_config(GUGEZEN_SIZES[z["beside"]], groups, vocab)))
+            entry = {"layers": 4 * groups, "width": z["width"], "beside": f"gugezen-{z['beside']}"}
+            for which, mcfg in made:
+                eng = build_engine_on_device(f"{which}-{name}", 4 * groups, ctx_len=ctx_len, page=page, max_seqs=B,
+                                             max_tokens=max(T, ctx), graph_sizes=(B,), mcfg=mcfg)
+                entry[which] = measure(eng)
+                del eng
+                torch.cuda.empty_cache()
+            entry.update(prefill_ratio=round(entry["suranex"]["prefill_tok_s"] / entry["gugezen"]["prefill_tok_s"], 3),
+                         decode_ratio=round(entry["suranex"]["decode_tok_s"] / entry["gugezen"]["decode_tok_s"], 3))
+            if "kernels" in a.phases.split(","):
+                entry["kernels"] = suranex_kernels(ops, z, pk, T, B, ctx, page)
             result["sizes"][name] = entry
             continue
         if a.design == "pizunex":
@@ -1365,7 +1570,7 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--phases", default="prefill,decode,points,e2e,kernels,mixed",
                     help="which measurements to run (decode always runs); fewer for a profiler capture")
-    ap.add_argument("--design", default="", choices=["", "komirax", "pizunex", "vofinex", "gugezen"],
+    ap.add_argument("--design", default="", choices=["", "komirax", "pizunex", "vofinex", "gugezen", "suranex"],
                     help="instead of the default workload: layers of this design beside layers of the closest other one (Komirax "
                          "beside Qwen2, Pizunex beside Komirax) at the same width "
                          "(prefill and decode throughput, and each of the design's kernels alone)")

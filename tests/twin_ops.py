@@ -672,13 +672,14 @@ def _grouped_glu(self, out, x, w, order, row_scale, offsets, tiles, top, glu):
     out.copy_(_glu(gu[:, 0::2], gu[:, 1::2], glu).to(out.dtype))
 
 
-def _short_filter(self, out, x, x_off, conv_w, conv_b, state, tail_off, step, taps):
+def _short_filter(self, out, x, x_off, conv_w, conv_b, state, ring_off, step, taps):
     W = out.shape[1]
-    qs, slots = step.q_start.tolist(), step.state_slots.tolist()
+    qs, slots, pos = step.q_start.tolist(), step.state_slots.tolist(), step.positions.tolist()
     for b in range(step.num_requests):
         lo, hi = qs[b], qs[b + 1]
-        tail = state[slots[b]][tail_off:tail_off + (taps - 1) * W].view(taps - 1, W)
-        rows = torch.cat([tail, x[lo:hi, x_off:x_off + W].float()], 0)
+        before = [state[slots[b]][ring_off + p % taps * W:ring_off + (p % taps + 1) * W] if p >= 0 else torch.zeros(W)
+                  for p in range(pos[lo] - taps + 1, pos[lo])]
+        rows = torch.cat([torch.stack(before) if before else torch.zeros(0, W), x[lo:hi, x_off:x_off + W].float()], 0)
         acc = conv_b.float().expand(hi - lo, W).clone() if conv_b is not None else torch.zeros(hi - lo, W)
         for u in range(taps):
             acc = acc + rows[u:u + hi - lo] * conv_w.float()[:, u]
@@ -697,7 +698,7 @@ def _rglru_gates(self, ab, u, ra, ri, ra_b, ri_b, rate):
 
 def _rglru_scan(self, out, ab, proj, y_off, x_off, state, step, taps):
     W = out.shape[1]
-    qs, slots = step.q_start.tolist(), step.state_slots.tolist()
+    qs, slots, pos = step.q_start.tolist(), step.state_slots.tolist(), step.positions.tolist()
     for b in range(step.num_requests):
         lo, hi = qs[b], qs[b + 1]
         row = state[slots[b]]
@@ -707,8 +708,8 @@ def _rglru_scan(self, out, ab, proj, y_off, x_off, state, step, taps):
             out[t] = (S * F.gelu(proj[t, y_off:y_off + W].float(), approximate="tanh")).to(out.dtype)
         row[:W] = S
         if taps > 1:
-            tail = row[W:].view(taps - 1, W)
-            tail.copy_(torch.cat([tail, proj[lo:hi, x_off:x_off + W].float()], 0)[-(taps - 1):].clone())
+            for t in range(max(lo, hi - taps + 1), hi):
+                row[W + pos[t] % taps * W:W + (pos[t] % taps + 1) * W] = proj[t, x_off:x_off + W].float()
 
 
 def _rglru_step(self, *args):

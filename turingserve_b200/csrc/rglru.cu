@@ -3,8 +3,11 @@
 // rate = 8 softplus(lam) (worked out when the weights are loaded):
 //     r = sigmoid(Ra u + ra_b),  i = sigmoid(Ri u + ri_b)         (Ra, Ri block-diagonal: `blocks` square matrices)
 //     a = exp(-rate r),   S <- a S + sqrt(1 - a^2) i u,   out = S gelu(y).
-// y and the filter's raw input are columns of one fused projection.  The filter's last taps - 1 inputs live behind S in
-// the request's state slot: [W | (taps - 1) x W], 32-bit.  sqrt(1 - a^2) is taken as sqrt(-expm1(-2 rate r)), which keeps
+// y and the filter's raw input are columns of one fused projection.  The filter's last inputs live behind S in the
+// request's state slot, 32-bit: [W | ring of taps x W], the input of the token at position p in place p % taps.  A token reads
+// the taps - 1 inputs before its own and writes its own place, which none of those is: nothing moves, and blocks of one
+// kernel may read and write in any order.  (Zeroed at admission, so places of positions before 0 read as zero: they are
+// not written before the tokens that would read them have run.)  sqrt(1 - a^2) is taken as sqrt(-expm1(-2 rate r)), which keeps
 // its digits where the decay is close to one.
 //
 //   ts_short_filter   u = bias + sum of taps, every channel, rounded to the engine's type; reads the slot's inputs for
@@ -15,10 +18,9 @@
 //   ts_rglru_scan     the recurrence: a block owns RS_CH channels of one request; RS_SEGS threads a channel take
 //                     RS_TOK neighbouring tokens each, fold them into one (decay, sum) pair, pick up the state in front
 //                     of them from the pairs before (shared memory), and run through their tokens once more for the
-//                     output; then the filter's new last inputs
+//                     output; then the filter's last inputs into their places
 //   ts_rglru_step     all of it in one kernel for a step of single tokens (bfloat16): the filter in shared memory, the
-//                     two products by m16n8k16 with the weights streamed from memory once, gates, state, output; the
-//                     block that comes last for its part (a ticket counter; nobody waits) moves the filter's inputs up
+//                     two products by m16n8k16 with the weights streamed from memory once, gates, state, output
 #include "activations.cuh"
 #include "common.cuh"
 #include "mma_utils.cuh"
@@ -27,61 +29,122 @@ namespace {
 
 constexpr int RG_MAX_TAPS = 8;
 
-// (decay, addend) of one channel from the two pre-activations
-__device__ __forceinline__ float2 rg_pair(float zr, float zi, float rate, float u) {
+// (decay, addend) of one channel from the two pre-activations.  bfloat16 engine: the hardware's approximate exponential and
+// reciprocal (relative errors of a few 2^-22, like the rounding of a 32-bit number; the exact functions cost
+// the gates kernel more than its products do), and 1 - a^2 by the series of -expm1(t), t = 2 log a, where a is close to
+// one (t > -1/2: seven terms, relative error below 2^-22), by the product 1 - a a elsewhere.
+template <typename T> __device__ __forceinline__ float2 rg_pair(float zr, float zi, float rate, float u) {
   const float r = 1.f / (1.f + expf(-zr)), i = 1.f / (1.f + expf(-zi));
   const float la = -rate * r;
   return make_float2(expf(la), sqrtf(-expm1f(2.f * la)) * i * u);
 }
+template <> __device__ __forceinline__ float2 rg_pair<bf16>(float zr, float zi, float rate, float u) {
+  const float r = __fdividef(1.f, 1.f + __expf(-zr)), i = __fdividef(1.f, 1.f + __expf(-zi));
+  const float la = -rate * r, t = 2.f * la;
+  const float a = __expf(la);
+  float p = fmaf(t, 1.f / 5040.f, 1.f / 720.f);
+  p = fmaf(t, p, 1.f / 120.f);
+  p = fmaf(t, p, 1.f / 24.f);
+  p = fmaf(t, p, 1.f / 6.f);
+  p = fmaf(t, p, 0.5f);
+  p = fmaf(t, p, 1.f);
+  const float left = t > -0.5f ? -t * p : fmaf(-a, a, 1.f);
+  return make_float2(a, __fsqrt_rn(left) * i * u);
+}
 
 // ---------------------------------------------------------------------------------------------------
-// grid (ceil(T / TOK), ceil(W / blockDim)): a thread takes one channel of TOK neighbouring tokens; the window of the
-// filter slides through registers and is refilled (from the rows before, or the slot's memory) only at the thread's
-// first token and where another request begins.
-template <typename T, int TOK>
-__global__ void __launch_bounds__(256)
+// V neighbouring channels of a row
+template <typename T, int V> struct RgVec;
+template <typename T> struct RgVec<T, 1> {
+  static __device__ __forceinline__ void load(const T* p, float* f) { f[0] = to_f(p[0]); }
+  static __device__ __forceinline__ void store(T* p, const float* f) { p[0] = from_f<T>(f[0]); }
+};
+template <> struct RgVec<bf16, 4> {
+  static __device__ __forceinline__ void load(const bf16* p, float* f) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+  static __device__ __forceinline__ void store(bf16* p, const float* f) {
+    uint2 v;
+    *reinterpret_cast<__nv_bfloat162*>(&v.x) = __floats2bfloat162_rn(f[0], f[1]);
+    *reinterpret_cast<__nv_bfloat162*>(&v.y) = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = v;
+  }
+};
+
+// grid (ceil(T / TOK), ceil(W / (V blockDim))): a thread takes V neighbouring channels of TOK neighbouring tokens; the
+// window of the filter slides through registers and is refilled (from the rows before, or the slot's memory) only at the
+// thread's first token and where another request begins.
+template <typename T, int TOK, int V>
+__global__ void __launch_bounds__(128)
 short_filter_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ x, int x_stride, int x_off,
                     const float* __restrict__ conv_w, const float* __restrict__ conv_b, const float* __restrict__ state,
-                    size_t state_stride, size_t tail_off, const int* __restrict__ token_request,
-                    const int* __restrict__ q_start, const int* __restrict__ slots, int T_, int W, int taps) {
+                    size_t state_stride, size_t ring_off, const int* __restrict__ token_request,
+                    const int* __restrict__ q_start, const int* __restrict__ slots, const int* __restrict__ positions, int T_,
+                    int W, int taps) {
   pdl_launch_dependents();
   pdl_wait();
   const int t_base = blockIdx.x * TOK;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= W) return;
   const int count = min(TOK, T_ - t_base), keep = taps - 1;
-  float v[TOK];
+  float v[TOK][V];
 #pragma unroll
-  for (int k = 0; k < TOK; ++k) v[k] = k < count ? to_f(x[(size_t)(t_base + k) * x_stride + x_off + c]) : 0.f;
-  float wgt[RG_MAX_TAPS];                                // wgt[d]: the tap d tokens back
+  for (int k = 0; k < TOK; ++k) {
+    if (k < count) {
+      RgVec<T, V>::load(x + (size_t)(t_base + k) * x_stride + x_off + c, v[k]);
+    } else {
 #pragma unroll
-  for (int d = 0; d < RG_MAX_TAPS; ++d) wgt[d] = d < taps ? conv_w[(size_t)c * taps + keep - d] : 0.f;
-  const float bias = conv_b != nullptr ? conv_b[c] : 0.f;
-  float win[RG_MAX_TAPS];                                // win[d]: the input d + 1 tokens back
+      for (int e = 0; e < V; ++e) v[k][e] = 0.f;
+    }
+  }
+  float wgt[RG_MAX_TAPS][V], bias[V];                    // wgt[d]: the tap d tokens back
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+    bias[e] = conv_b != nullptr ? conv_b[c + e] : 0.f;
+#pragma unroll
+    for (int d = 0; d < RG_MAX_TAPS; ++d) wgt[d][e] = d < taps ? conv_w[(size_t)(c + e) * taps + keep - d] : 0.f;
+  }
+  float win[RG_MAX_TAPS][V];                             // win[d]: the input d + 1 tokens back
+  int t_end = t_base;                                    // the end of the request the window belongs to
 #pragma unroll
   for (int k = 0; k < TOK; ++k) {
     if (k < count) {
       const int t = t_base + k;
-      const int b = token_request[t];
-      const int t0 = q_start[b], i = t - t0;
-      if (k == 0 || i == 0) {
-        const float* tail = state + (size_t)slots[b] * state_stride + tail_off;        // [taps - 1][W], oldest first
+      if (t >= t_end) {
+        const int b = token_request[t];
+        const int t0 = q_start[b], i = t - t0;
+        t_end = q_start[b + 1];
+        const int pos = positions[t];
+        const float* ring = state + (size_t)slots[b] * state_stride + ring_off;        // [taps][W]
 #pragma unroll
         for (int d = 0; d < RG_MAX_TAPS - 1; ++d)
           if (d < keep) {
             const int rel = i - 1 - d;                   // counted from the step's first token
-            win[d] = rel >= 0 ? to_f(x[(size_t)(t0 + rel) * x_stride + x_off + c]) : tail[(size_t)(rel + keep) * W + c];
+            const int at = pos - 1 - d;                  // the input's position in the sequence
+            if (rel >= 0) {
+              RgVec<T, V>::load(x + (size_t)(t0 + rel) * x_stride + x_off + c, win[d]);
+            } else {
+#pragma unroll
+              for (int e = 0; e < V; ++e) win[d][e] = at >= 0 ? ring[(size_t)(at % taps) * W + c + e] : 0.f;
+            }
           }
       }
-      float acc = bias;
+      float acc[V];
 #pragma unroll
-      for (int d = RG_MAX_TAPS - 1; d > 0; --d)
-        if (d < taps) acc = fmaf(wgt[d], win[d - 1], acc);
-      acc = fmaf(wgt[0], v[k], acc);
-      out[(size_t)t * out_stride + c] = from_f<T>(acc);
+      for (int e = 0; e < V; ++e) {
+        acc[e] = bias[e];
 #pragma unroll
-      for (int d = RG_MAX_TAPS - 2; d > 0; --d) win[d] = win[d - 1];
-      win[0] = v[k];
+        for (int d = RG_MAX_TAPS - 1; d > 0; --d)
+          if (d < taps) acc[e] = fmaf(wgt[d][e], win[d - 1][e], acc[e]);
+        acc[e] = fmaf(wgt[0][e], v[k][e], acc[e]);
+#pragma unroll
+        for (int d = RG_MAX_TAPS - 2; d > 0; --d) win[d][e] = win[d - 1][e];
+        win[0][e] = v[k][e];
+      }
+      RgVec<T, V>::store(out + (size_t)t * out_stride + c, acc);
     }
   }
 }
@@ -142,7 +205,7 @@ rglru_gates_kernel(float2* __restrict__ ab, const T* __restrict__ u, const T* __
       const int n = n0 + tx * 4 + j;
       if (n >= bs) continue;
       const int c = part * bs + n;
-      ab[(size_t)m * W + c] = rg_pair(r_acc[i][j] + ra_b[c], i_acc[i][j] + ri_b[c], rate[c], to_f(u[(size_t)m * W + c]));
+      ab[(size_t)m * W + c] = rg_pair<T>(r_acc[i][j] + ra_b[c], i_acc[i][j] + ri_b[c], rate[c], to_f(u[(size_t)m * W + c]));
     }
   }
 }
@@ -227,8 +290,8 @@ rglru_gates_mma_kernel(float2* __restrict__ ab, const bf16* __restrict__ u, cons
       const int m = m0 + warp * 16 + (lane >> 2) + 8 * h;
       if (m >= M) continue;
       const float2 uv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(u + (size_t)m * W + c));
-      const float2 p0 = rg_pair(r_acc[nt][2 * h] + rbias.x, i_acc[nt][2 * h] + ibias.x, rt.x, uv.x);
-      const float2 p1 = rg_pair(r_acc[nt][2 * h + 1] + rbias.y, i_acc[nt][2 * h + 1] + ibias.y, rt.y, uv.y);
+      const float2 p0 = rg_pair<bf16>(r_acc[nt][2 * h] + rbias.x, i_acc[nt][2 * h] + ibias.x, rt.x, uv.x);
+      const float2 p1 = rg_pair<bf16>(r_acc[nt][2 * h + 1] + rbias.y, i_acc[nt][2 * h + 1] + ibias.y, rt.y, uv.y);
       *reinterpret_cast<float4*>(ab + (size_t)m * W + c) = make_float4(p0.x, p0.y, p1.x, p1.y);
     }
   }
@@ -241,7 +304,7 @@ template <typename T>
 __global__ void __launch_bounds__(RS_CH * RS_SEGS)
 rglru_scan_kernel(T* __restrict__ out, const float2* __restrict__ ab, const T* __restrict__ proj, int proj_stride,
                   int y_off, int x_off, float* __restrict__ state, size_t state_stride, const int* __restrict__ q_start,
-                  const int* __restrict__ slots, int W, int taps) {
+                  const int* __restrict__ slots, const int* __restrict__ positions, int W, int taps) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float2 agg[2][RS_SEGS][RS_CH];
@@ -253,6 +316,8 @@ rglru_scan_kernel(T* __restrict__ out, const float2* __restrict__ ab, const T* _
   const int c = blockIdx.x * RS_CH + col;
   const bool live = c < W;
   float* base = state + (size_t)slots[b] * state_stride;
+  const bool one = n <= RS_TOK;                          // the first segment's thread runs through the request alone
+  if (one && seg > 0) return;                            // (no barrier is reached then)
   if (seg == 0) carry_s[0][col] = live ? base[c] : 0.f;
   float2 v[RS_TOK];
   T y[RS_TOK];
@@ -267,6 +332,7 @@ rglru_scan_kernel(T* __restrict__ out, const float2* __restrict__ ab, const T* _
   };
   fetch(0);
   int buf = 0;
+  const int segs_last = one ? 0 : RS_SEGS - 1;           // (a segment without tokens passes the state on)
   for (int g0 = 0; g0 < n; g0 += RS_SEGS * RS_TOK, buf ^= 1) {
     float A = 1.f, B = 0.f;
 #pragma unroll
@@ -274,9 +340,14 @@ rglru_scan_kernel(T* __restrict__ out, const float2* __restrict__ ab, const T* _
       B = fmaf(v[k].x, B, v[k].y);
       A *= v[k].x;
     }
-    agg[buf][seg][col] = make_float2(A, B);
-    __syncthreads();
-    float S = carry_s[buf][col];
+    float S;
+    if (one) {
+      S = carry_s[0][col];                               // (this thread's own)
+    } else {
+      agg[buf][seg][col] = make_float2(A, B);
+      __syncthreads();
+      S = carry_s[buf][col];
+    }
 #pragma unroll 4
     for (int s = 0; s < seg; ++s) {
       const float2 p = agg[buf][s][col];
@@ -288,149 +359,176 @@ rglru_scan_kernel(T* __restrict__ out, const float2* __restrict__ ab, const T* _
       S = fmaf(v[k].x, S, v[k].y);
       o[k] = S * ts_activate_for<T>(to_f(y[k]), TS_ACT_GELU_TANH);
     }
-    if (seg == RS_SEGS - 1) carry_s[buf ^ 1][col] = S;
+    if (!one && seg == RS_SEGS - 1) carry_s[buf ^ 1][col] = S;
     const int first = g0 + seg * RS_TOK;
     if (g0 + RS_SEGS * RS_TOK < n) fetch(g0 + RS_SEGS * RS_TOK);
 #pragma unroll
     for (int k = 0; k < RS_TOK; ++k)
       if (live && first + k < n) out[(size_t)(t0 + first + k) * W + c] = from_f<T>(o[k]);
-    if (g0 + RS_SEGS * RS_TOK >= n && seg == RS_SEGS - 1 && live) base[c] = S;
+    if (g0 + RS_SEGS * RS_TOK >= n && seg == segs_last && live) base[c] = S;
   }
-  // the filter's new last inputs: the step's last taps - 1 raw rows, or, of a shorter step, the old ones moved up
+  // the filter's last inputs into their places
   if (seg == 0 && live && taps > 1) {
-    float* tail = base + W;
-    const int keep = taps - 1;
-    float r[RG_MAX_TAPS];
-#pragma unroll
-    for (int k = 0; k < RG_MAX_TAPS - 1; ++k)
-      if (k < keep) {
-        const int rel = n - keep + k;
-        r[k] = rel >= 0 ? to_f(proj[(size_t)(t0 + rel) * proj_stride + x_off + c]) : tail[(size_t)(rel + keep) * W + c];
-      }
-#pragma unroll
-    for (int k = 0; k < RG_MAX_TAPS - 1; ++k)
-      if (k < keep) tail[(size_t)k * W + c] = r[k];
+    float* ring = base + W + c;
+    const int pos0 = positions[t0];
+    for (int i = max(0, n - (taps - 1)); i < n; ++i)
+      ring[(size_t)((pos0 + i) % taps) * W] = to_f(proj[(size_t)(t0 + i) * proj_stride + x_off + c]);
   }
 }
 
 // ---------------------------------------------------------------------------------------------------
-// A step of single tokens.  grid (channel groups of a part, parts, groups of RT_TOK tokens).
-constexpr int RT_TOK = 8, RT_WARPS = 4, RT_UNROLL = 4;
+// A step of single tokens.  grid (channel groups of a part, parts, groups of RT_TOK tokens).  Everything that is weights is on
+// its way before the wait for the predecessor, everything that is state or projection right after it.
+constexpr int RT_TOK = 8, RT_WARPS = 8, RT_UNROLL = 4;
 
 __global__ void __launch_bounds__(RT_WARPS * 32)
 rglru_step_kernel(bf16* __restrict__ out, const bf16* __restrict__ proj, int proj_stride, int y_off, int x_off,
                   const float* __restrict__ conv_w, const float* __restrict__ conv_b, const bf16* __restrict__ ra,
                   const bf16* __restrict__ ri, const float* __restrict__ ra_b, const float* __restrict__ ri_b,
                   const float* __restrict__ rate, float* __restrict__ state, size_t state_stride,
-                  const int* __restrict__ slots, int M, int W, int bs, int taps, int* __restrict__ counters) {
+                  const int* __restrict__ slots, const int* __restrict__ positions, int M, int W, int bs, int taps) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char rtm[];
   bf16* u_s = reinterpret_cast<bf16*>(rtm);              // [RT_TOK][bs + 8]
-  __shared__ int slot_s[RT_TOK];
-  __shared__ int last_flag;
+  __shared__ int slot_s[RT_TOK], pos_s[RT_TOK];
   const int part = blockIdx.y, m0 = blockIdx.z * RT_TOK;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
-  const int n0 = (blockIdx.x * RT_WARPS + warp) * 8;     // this warp's channels of the part
+  const int own0 = blockIdx.x * RT_WARPS * 8;            // this block's channels of the part
+  const int n0 = own0 + warp * 8;                        // and this warp's
   const int us = bs + 8, keep = taps - 1;
   const bool n_ok = n0 + g < bs;
   const bf16* r_row = ra + ((size_t)part * bs + (n_ok ? n0 + g : 0)) * bs + t * 8;
   const bf16* i_row = ri + ((size_t)part * bs + (n_ok ? n0 + g : 0)) * bs + t * 8;
-  // (the weights are nobody's output: the first of them are on their way before the wait)
-  uint4 rw[RT_UNROLL], iw[RT_UNROLL];
-  auto fetch = [&](int k0) {
+  uint4 rw[2][RT_UNROLL], iw[2][RT_UNROLL];
+  auto fetch = [&](int k0, int buf) {
 #pragma unroll
     for (int q = 0; q < RT_UNROLL; ++q) {
       const int k = k0 + q * 32;
       const bool ok = n_ok && k + t * 8 < bs;
-      rw[q] = ok ? *reinterpret_cast<const uint4*>(r_row + k) : make_uint4(0u, 0u, 0u, 0u);
-      iw[q] = ok ? *reinterpret_cast<const uint4*>(i_row + k) : make_uint4(0u, 0u, 0u, 0u);
+      rw[buf][q] = ok ? *reinterpret_cast<const uint4*>(r_row + k) : make_uint4(0u, 0u, 0u, 0u);
+      iw[buf][q] = ok ? *reinterpret_cast<const uint4*>(i_row + k) : make_uint4(0u, 0u, 0u, 0u);
     }
   };
-  fetch(0);
-  pdl_wait();
-  if (threadIdx.x < RT_TOK) slot_s[threadIdx.x] = m0 + threadIdx.x < M ? slots[m0 + threadIdx.x] : -1;
-  __syncthreads();
-  for (int idx = threadIdx.x; idx < RT_TOK * bs; idx += RT_WARPS * 32) {
-    const int m = idx / bs, k = idx % bs, c = part * bs + k;
-    float acc = 0.f;
-    if (slot_s[m] >= 0) {
-      const float* tail = state + (size_t)slot_s[m] * state_stride + W;
-      acc = conv_b != nullptr ? conv_b[c] : 0.f;
-      for (int d = 0; d < keep; ++d) acc = fmaf(conv_w[(size_t)c * taps + d], tail[(size_t)d * W + c], acc);
-      acc = fmaf(conv_w[(size_t)c * taps + keep], to_f(proj[(size_t)(m0 + m) * proj_stride + x_off + c]), acc);
+  fetch(0, 0);
+  fetch(32 * RT_UNROLL, 1);
+  float rb[2] = {0.f, 0.f}, ib[2] = {0.f, 0.f}, rt[2] = {0.f, 0.f};
+#pragma unroll
+  for (int e = 0; e < 2; ++e)
+    if (n0 + 2 * t + e < bs) {
+      const int c = part * bs + n0 + 2 * t + e;
+      rb[e] = ra_b[c];
+      ib[e] = ri_b[c];
+      rt[e] = rate[c];
     }
-    u_s[m * us + k] = from_f<bf16>(acc);
+  // (slots and positions come from the host, before the step's first kernel)
+  if (threadIdx.x < RT_TOK) {
+    const bool there = m0 + (int)threadIdx.x < M;
+    slot_s[threadIdx.x] = there ? slots[m0 + threadIdx.x] : -1;
+    pos_s[threadIdx.x] = there ? positions[m0 + threadIdx.x] : 0;
   }
   __syncthreads();
-  // every block of the part has taken what it needs of the filter's inputs once it has counted itself
-  if (threadIdx.x == 0) {
-    int* counter = counters + (size_t)blockIdx.z * gridDim.y + part;
-    __threadfence();
-    last_flag = atomicAdd(counter, 1) == (int)gridDim.x - 1;
-    if (last_flag) *counter = 0;                         // ready for the next launch
+  pdl_wait();
+  // what the end of this thread's work wants: its state, and the gate branch
+  float S_old[2] = {0.f, 0.f}, y_raw[2] = {0.f, 0.f};
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int n = n0 + 2 * t + e;
+    if (m0 + g < M && n < bs) {
+      S_old[e] = state[(size_t)slot_s[g] * state_stride + part * bs + n];
+      y_raw[e] = to_f(proj[(size_t)(m0 + g) * proj_stride + y_off + part * bs + n]);
+    }
   }
+  // the filter: a thread a channel of all tokens, every load independent of the others
+  for (int k = threadIdx.x; k < bs; k += RT_WARPS * 32) {
+    const int c = part * bs + k;
+    float acc[RT_TOK], x[RT_TOK];
+    const float bias = conv_b != nullptr ? conv_b[c] : 0.f, w_now = conv_w[(size_t)c * taps + keep];
+#pragma unroll
+    for (int m = 0; m < RT_TOK; ++m) {
+      x[m] = slot_s[m] >= 0 ? to_f(proj[(size_t)(m0 + m) * proj_stride + x_off + c]) : 0.f;
+      acc[m] = bias;
+    }
+#pragma unroll
+    for (int d = RG_MAX_TAPS - 1; d > 0; --d)            // d tokens back
+      if (d < taps) {
+        const float w = conv_w[(size_t)c * taps + keep - d];
+        float v[RT_TOK];
+#pragma unroll
+        for (int m = 0; m < RT_TOK; ++m) {
+          const int at = pos_s[m] - d;
+          v[m] = slot_s[m] >= 0 && at >= 0 ? state[(size_t)slot_s[m] * state_stride + W + (size_t)(at % taps) * W + c] : 0.f;
+        }
+#pragma unroll
+        for (int m = 0; m < RT_TOK; ++m) acc[m] = fmaf(w, v[m], acc[m]);
+      }
+    const bool own = taps > 1 && k >= own0 && k < own0 + RT_WARPS * 8;
+#pragma unroll
+    for (int m = 0; m < RT_TOK; ++m) {
+      u_s[m * us + k] = from_f<bf16>(slot_s[m] >= 0 ? fmaf(w_now, x[m], acc[m]) : 0.f);
+      // (its place in the ring: one that no token of this step reads)
+      if (own && slot_s[m] >= 0) state[(size_t)slot_s[m] * state_stride + W + (size_t)(pos_s[m] % taps) * W + c] = x[m];
+    }
+  }
+  __syncthreads();
   float zr[4] = {0.f, 0.f, 0.f, 0.f}, zi[4] = {0.f, 0.f, 0.f, 0.f};
-  for (int k0 = 0; k0 < bs; k0 += 32 * RT_UNROLL) {
-    if (k0 > 0) fetch(k0);
+  auto multiply = [&](int k0, int buf) {
 #pragma unroll
     for (int q = 0; q < RT_UNROLL; ++q) {
       const int k = k0 + q * 32 + t * 8;
       const uint4 uv = k < bs ? *reinterpret_cast<const uint4*>(u_s + g * us + k) : make_uint4(0u, 0u, 0u, 0u);
       // rows 8 .. 15 of the product are zero; its k index is a permutation of the real one, the same for both operands
       const unsigned a1[4] = {uv.x, 0u, uv.y, 0u}, a2[4] = {uv.z, 0u, uv.w, 0u};
-      mma_bf16(zr, a1, rw[q].x, rw[q].y);
-      mma_bf16(zr, a2, rw[q].z, rw[q].w);
-      mma_bf16(zi, a1, iw[q].x, iw[q].y);
-      mma_bf16(zi, a2, iw[q].z, iw[q].w);
+      mma_bf16(zr, a1, rw[buf][q].x, rw[buf][q].y);
+      mma_bf16(zr, a2, rw[buf][q].z, rw[buf][q].w);
+      mma_bf16(zi, a1, iw[buf][q].x, iw[buf][q].y);
+      mma_bf16(zi, a2, iw[buf][q].z, iw[buf][q].w);
     }
+  };
+  constexpr int KSTEP = 32 * RT_UNROLL;
+  for (int k0 = 0; k0 < bs; k0 += 2 * KSTEP) {
+    multiply(k0, 0);
+    if (k0 + 2 * KSTEP < bs) fetch(k0 + 2 * KSTEP, 0);
+    if (k0 + KSTEP < bs) multiply(k0 + KSTEP, 1);
+    if (k0 + 3 * KSTEP < bs) fetch(k0 + 3 * KSTEP, 1);
   }
   const int m = m0 + g;
-  if (m < M) {
-    float* S = state + (size_t)slot_s[g] * state_stride;
+  if (m >= M) return;
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int n = n0 + 2 * t + e;
-      if (n >= bs) continue;
-      const int c = part * bs + n;
-      const float2 p = rg_pair(zr[e] + ra_b[c], zi[e] + ri_b[c], rate[c], to_f(u_s[g * us + n]));
-      const float s = fmaf(p.x, S[c], p.y);
-      S[c] = s;
-      const float y = ts_activate_for<bf16>(to_f(proj[(size_t)m * proj_stride + y_off + c]), TS_ACT_GELU_TANH);
-      out[(size_t)m * W + c] = from_f<bf16>(s * y);
-    }
-  }
-  if (keep == 0) return;
-  __syncthreads();
-  if (!last_flag) return;
-  for (int idx = threadIdx.x; idx < RT_TOK * bs; idx += RT_WARPS * 32) {
-    const int mm = idx / bs, c = part * bs + idx % bs;
-    if (slot_s[mm] < 0) continue;
-    float* tail = state + (size_t)slot_s[mm] * state_stride + W + c;
-    for (int d = 0; d + 1 < keep; ++d) tail[(size_t)d * W] = tail[(size_t)(d + 1) * W];
-    tail[(size_t)(keep - 1) * W] = to_f(proj[(size_t)(m0 + mm) * proj_stride + x_off + c]);
+  for (int e = 0; e < 2; ++e) {
+    const int n = n0 + 2 * t + e;
+    if (n >= bs) continue;
+    const int c = part * bs + n;
+    const float2 p = rg_pair<bf16>(zr[e] + rb[e], zi[e] + ib[e], rt[e], to_f(u_s[g * us + n]));
+    const float s = fmaf(p.x, S_old[e], p.y);
+    state[(size_t)slot_s[g] * state_stride + c] = s;
+    out[(size_t)m * W + c] = from_f<bf16>(s * ts_activate_for<bf16>(y_raw[e], TS_ACT_GELU_TANH));
   }
 }
 
 }  // namespace
 
 // out [T, out_stride] (W columns); x [T, x_stride], the filtered channels from column x_off; conv_w [W, taps] and conv_b
-// [W] 32-bit (conv_b may be null); state [slots, state_stride] 32-bit, the inputs before the step from tail_off.
+// [W] 32-bit (conv_b may be null); state [slots, state_stride] 32-bit, the ring of the filter's inputs from ring_off;
+// positions [T]: the tokens' places in their sequences.
 TS_API int ts_short_filter(void* out, int out_stride, const void* x, int x_stride, int x_off, const float* conv_w,
-                           const float* conv_b, const float* state, long long state_stride, long long tail_off,
-                           const int* token_request, const int* q_start, const int* slots, int T, int W, int taps, int dtype,
-                           void* stream) {
+                           const float* conv_b, const float* state, long long state_stride, long long ring_off,
+                           const int* token_request, const int* q_start, const int* slots, const int* positions, int T, int W,
+                           int taps, int dtype, void* stream) {
   if (T <= 0 || W <= 0) return 0;
   if (taps < 1 || taps > RG_MAX_TAPS) TS_REFUSE(TS_ERR_LIMIT, "ts_short_filter: a filter of %d taps (1 to %d)", taps, RG_MAX_TAPS);
   cudaStream_t s = (cudaStream_t)stream;
   const bool few = T <= 64;
-  const dim3 grid(few ? T : ceil_div(T, 8), ceil_div(W, 256));
+  // bfloat16 rows on 8-byte boundaries: four channels a thread
+  const bool vec = dtype == TS_BF16 && !few && W % 4 == 0 && out_stride % 4 == 0 && x_stride % 4 == 0 && x_off % 4 == 0 &&
+                   !(((uintptr_t)out | (uintptr_t)x) & 7);
+  const dim3 grid(few ? T : ceil_div(T, 8), ceil_div(W, vec ? 512 : 128));
   if (grid.y > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_short_filter: %d channels", W);
-#define TS_SF(TT, N)                                                                                                   \
-  ts_launch(short_filter_kernel<TT, N>, grid, dim3(256), 0, s, (TT*)out, out_stride, (const TT*)x, x_stride, x_off, conv_w, \
-            conv_b, state, (size_t)state_stride, (size_t)tail_off, token_request, q_start, slots, T, W, taps)
-  if (dtype == TS_F32) { if (few) TS_SF(float, 1); else TS_SF(float, 8); }
-  else if (dtype == TS_BF16) { if (few) TS_SF(bf16, 1); else TS_SF(bf16, 8); }
+#define TS_SF(TT, N, V)                                                                                                \
+  ts_launch(short_filter_kernel<TT, N, V>, grid, dim3(128), 0, s, (TT*)out, out_stride, (const TT*)x, x_stride, x_off, conv_w, \
+            conv_b, state, (size_t)state_stride, (size_t)ring_off, token_request, q_start, slots, positions, T, W, taps)
+  if (dtype == TS_F32) { if (few) TS_SF(float, 1, 1); else TS_SF(float, 8, 1); }
+  else if (dtype == TS_BF16) { if (few) TS_SF(bf16, 1, 1); else if (vec) TS_SF(bf16, 8, 4); else TS_SF(bf16, 8, 1); }
   else TS_REFUSE(TS_ERR_DTYPE, "ts_short_filter: dtype %d", dtype);
 #undef TS_SF
   TS_LAUNCH_CHECK();
@@ -470,13 +568,13 @@ TS_API int ts_rglru_gates(float* ab, const void* u, const void* ra, const void* 
 }
 
 // out [T, W]; ab as ts_rglru_gates left it; proj [T, proj_stride]: the gate branch y from column y_off, the filter's raw
-// input from x_off; state [slots, state_stride]: [W | (taps - 1) x W], read and left updated at each request's slot.
+// input from x_off; state [slots, state_stride]: [W | ring of taps x W], read and left updated at each request's slot.
 // longest: the most tokens a request brings (0: not known); long portions are launched late (see ts_launch_late).
 constexpr int RS_LATE_TOKENS = 64;
 
 TS_API int ts_rglru_scan(void* out, const float* ab, const void* proj, int proj_stride, int y_off, int x_off, float* state,
-                         long long state_stride, const int* q_start, const int* slots, int B, int W, int taps, int longest,
-                         int dtype, void* stream) {
+                         long long state_stride, const int* q_start, const int* slots, const int* positions, int B, int W,
+                         int taps, int longest, int dtype, void* stream) {
   if (B <= 0) return 0;
   if (taps < 1 || taps > RG_MAX_TAPS) TS_REFUSE(TS_ERR_LIMIT, "ts_rglru_scan: a filter of %d taps (1 to %d)", taps, RG_MAX_TAPS);
   if (B > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_rglru_scan: %d requests per launch", B);
@@ -486,10 +584,10 @@ TS_API int ts_rglru_scan(void* out, const float* ab, const void* proj, int proj_
   do {                                                                                                                 \
     if (longest >= RS_LATE_TOKENS)                                                                                     \
       ts_launch_late(rglru_scan_kernel<TT>, grid, block, 0, s, (TT*)out, (const float2*)ab, (const TT*)proj, proj_stride, y_off, \
-                     x_off, state, (size_t)state_stride, q_start, slots, W, taps);                                     \
+                     x_off, state, (size_t)state_stride, q_start, slots, positions, W, taps);                                     \
     else                                                                                                               \
       ts_launch(rglru_scan_kernel<TT>, grid, block, 0, s, (TT*)out, (const float2*)ab, (const TT*)proj, proj_stride, y_off, \
-                x_off, state, (size_t)state_stride, q_start, slots, W, taps);                                          \
+                x_off, state, (size_t)state_stride, q_start, slots, positions, W, taps);                                          \
   } while (0)
   if (dtype == TS_F32) TS_RS(float);
   else if (dtype == TS_BF16) TS_RS(bf16);
@@ -502,24 +600,21 @@ TS_API int ts_rglru_step_supported(int W, int blocks, int taps, int dtype) {
   return dtype == TS_BF16 && blocks > 0 && blocks <= 65535 && W % blocks == 0 && (W / blocks) % 8 == 0 && W / blocks <= 2048 &&
          taps >= 1 && taps <= RG_MAX_TAPS;
 }
-// Zeroed ints ts_rglru_step wants.
-TS_API int ts_rglru_step_counters(int T, int blocks) { return ceil_div(T, RT_TOK) * blocks; }
 
-// Every token of the step is a request of its own, token m that of slots[m].  Arguments as of the three kernels above.
+// Every token of the step is a request of its own, token m that of slots[m] at positions[m].  Arguments as of the three kernels above.
 TS_API int ts_rglru_step(void* out, const void* proj, int proj_stride, int y_off, int x_off, const float* conv_w,
                          const float* conv_b, const void* ra, const void* ri, const float* ra_b, const float* ri_b,
-                         const float* rate, float* state, long long state_stride, const int* slots, int T, int W, int blocks,
-                         int taps, int* counters, int dtype, void* stream) {
+                         const float* rate, float* state, long long state_stride, const int* slots, const int* positions, int T,
+                         int W, int blocks, int taps, int dtype, void* stream) {
   if (T <= 0) return 0;
   if (!ts_rglru_step_supported(W, blocks, taps, dtype) || (((uintptr_t)ra | (uintptr_t)ri) & 15))
     TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_rglru_step: %d channels in %d parts, %d taps", W, blocks, taps);
-  if (counters == nullptr) TS_REFUSE(TS_ERR_SHAPE, "ts_rglru_step: no counters");
   const int bs = W / blocks;
   const dim3 grid(ceil_div(bs, 8 * RT_WARPS), blocks, ceil_div(T, RT_TOK));
   if (grid.z > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_rglru_step: %d tokens", T);
   const size_t smem = (size_t)RT_TOK * (bs + 8) * 2;     // (at most 33 KB)
   ts_launch(rglru_step_kernel, grid, dim3(RT_WARPS * 32), smem, (cudaStream_t)stream, (bf16*)out, (const bf16*)proj, proj_stride,
             y_off, x_off, conv_w, conv_b, (const bf16*)ra, (const bf16*)ri, ra_b, ri_b, rate, state, (size_t)state_stride, slots,
-            T, W, bs, taps, counters);
+            positions, T, W, bs, taps);
   TS_LAUNCH_CHECK();
 }

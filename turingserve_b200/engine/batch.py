@@ -67,6 +67,8 @@ class StepInputs:
     streaming_decode: bool = False
     # every row of the batch is wanted, in batch order (a captured decode step)
     all_rows_sampled: bool = False
+    # the step's token ids on the host, where it knows them all (None: some are fed back on the device)
+    host_ids: np.ndarray | None = None
 
 
 # From about this many keys under the decode rows of a step (requests x longest context), reading them
@@ -253,4 +255,5 @@ class StepInputBuilder:
             seq_lens=d(o_sl, B), state_slots=d(o_ss, B), sample_rows=d(o_sr, S), groups=groups,
             feedback_rows=d(o_fr, F), feedback_src=d(o_fs, F),
             q_lens=q_lens, starts=starts, max_q_len=max(q_lens), max_seq_len=int(sl.max()) if B else 0,
-            streaming_decode=streaming_decode(num_decode, int(sl[:num_decode].max()) if num_decode else 0))
+            streaming_decode=streaming_decode(num_decode, int(sl[:num_decode].max()) if num_decode else 0),
+            host_ids=ids.copy() if F == 0 else None)

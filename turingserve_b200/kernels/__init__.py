@@ -145,12 +145,11 @@ class CudaOps:
             "ts_post_norm": [P, P, P, P, P, I, P, P, P, P, I, F, P, F, P, F, I, I, I, P],
             "ts_qkv_heads_write": [P, I, I, I, P, P, P, F, P, F, I, I, P, P, P, P, I, I, I, I, I, I, I, P, I, I, I, P],
             "ts_qkv_heads_supports_parts": [I, I, I, I, I, I, I, I],
-            "ts_short_filter": [P, I, P, I, I, P, P, P, ctypes.c_longlong, ctypes.c_longlong, P, P, P, I, I, I, I, P],
+            "ts_short_filter": [P, I, P, I, I, P, P, P, ctypes.c_longlong, ctypes.c_longlong, P, P, P, P, I, I, I, I, P],
             "ts_rglru_gates": [P, P, P, P, P, P, P, I, I, I, I, P],
-            "ts_rglru_scan": [P, P, P, I, I, I, P, ctypes.c_longlong, P, P, I, I, I, I, I, P],
-            "ts_rglru_step": [P, P, I, I, I, P, P, P, P, P, P, P, P, ctypes.c_longlong, P, I, I, I, I, P, I, P],
+            "ts_rglru_scan": [P, P, P, I, I, I, P, ctypes.c_longlong, P, P, P, I, I, I, I, I, P],
+            "ts_rglru_step": [P, P, I, I, I, P, P, P, P, P, P, P, P, ctypes.c_longlong, P, P, I, I, I, I, I, P],
             "ts_rglru_step_supported": [I, I, I, I],
-            "ts_rglru_step_counters": [I, I],
             "ts_batched_linear": [P, I, I, P, I, I, P, I, I, I, I, I, P],
         }
         for name, args in sigs.items():
@@ -832,7 +831,7 @@ class CudaOps:
             ms = 1
             if nd > 0 and G <= 64:
                 ms = max(1, min(16, (8 if spread else 16) if splits <= 0 else splits,
-                                2 * self.num_sms // max(1, nd * KVH * chunks), reach // (256 if spread else 128)))
+                                2 * self.num_sms // max(1, nd * KVH * chunks), reach // 128))
 
             def launch(first: int, count: int, max_q: int, n_splits: int, spread_flag: int) -> int:
                 scratch = counters = None
@@ -1069,15 +1068,15 @@ class CudaOps:
         return proj
 
     # -- the real-gated linear recurrent unit ----------------------------------------------------------------------
-    def short_filter(self, out, x, x_off: int, conv_w, conv_b, state, tail_off: int, step, taps: int) -> None:
+    def short_filter(self, out, x, x_off: int, conv_w, conv_b, state, ring_off: int, step, taps: int) -> None:
         """out [T, W] = the columns x_off .. x_off + W of ``x`` through their causal filters (``conv_w`` float32 [W, taps], the
         last column the present token's; ``conv_b`` float32 [W] or None); the inputs before the step's first token come from
-        the request's state slot, from ``tail_off`` on."""
+        the request's state slot: a ring of ``taps`` rows from ``ring_off`` on, the input at position p in row p % taps."""
         T, W = out.shape
         self._check(self.lib.ts_short_filter(_ptr(out), out.stride(0), _ptr(x), x.stride(0), x_off, _ptr(conv_w), _ptr(conv_b),
-                                             _ptr(state), state.stride(0), int(tail_off), _ptr(step.token_request),
-                                             _ptr(step.q_start), _ptr(step.state_slots), T, W, taps, _code(x.dtype),
-                                             self._stream()), "short_filter")
+                                             _ptr(state), state.stride(0), int(ring_off), _ptr(step.token_request),
+                                             _ptr(step.q_start), _ptr(step.state_slots), _ptr(step.positions), T, W, taps,
+                                             _code(x.dtype), self._stream()), "short_filter")
 
     def rglru_gates(self, ab, u, ra, ri, ra_b, ri_b, rate) -> None:
         """ab (float32 [T, W, 2]) = (a, sqrt(1 - a^2) i u) with a = exp(-rate r), r and i the sigmoids of the block-diagonal
@@ -1088,12 +1087,12 @@ class CudaOps:
 
     def rglru_scan(self, out, ab, proj, y_off: int, x_off: int, state, step, taps: int) -> None:
         """out [T, W] = S gelu_tanh(y) with S <- a S + b over the pairs of ``rglru_gates``, y the columns of ``proj`` from
-        ``y_off``; ``state`` (float32 [slots, W + (taps - 1) W]) is read and left updated at each request's slot, the filter's
-        last inputs (the columns from ``x_off``) included."""
+        ``y_off``; ``state`` (float32 [slots, W + taps W]) is read and left updated at each request's slot, the ring of the
+        filter's last inputs (the columns from ``x_off``) included."""
         W = out.shape[1]
         self._check(self.lib.ts_rglru_scan(_ptr(out), _ptr(ab), _ptr(proj), proj.stride(0), y_off, x_off, _ptr(state),
-                                           state.stride(0), _ptr(step.q_start), _ptr(step.state_slots), step.num_requests, W,
-                                           taps, int(getattr(step, "max_q_len", 0) or 0), _code(proj.dtype), self._stream()),
+                                           state.stride(0), _ptr(step.q_start), _ptr(step.state_slots), _ptr(step.positions),
+                                           step.num_requests, W, taps, int(getattr(step, "max_q_len", 0) or 0), _code(proj.dtype), self._stream()),
                     "rglru_scan")
 
     def rglru_step(self, out, proj, y_off: int, x_off: int, conv_w, conv_b, ra, ri, ra_b, ri_b, rate, state, step,
@@ -1105,11 +1104,10 @@ class CudaOps:
         if (step.max_q_len != 1 or step.num_requests != T
                 or not self.lib.ts_rglru_step_supported(W, parts, taps, _code(proj.dtype))):
             return False
-        counters = self._buffer("rglru_counters", self.lib.ts_rglru_step_counters(T, parts), torch.int32, proj.device,
-                                floor=1 << 12, zero=True)
         rc = self.lib.ts_rglru_step(_ptr(out), _ptr(proj), proj.stride(0), y_off, x_off, _ptr(conv_w), _ptr(conv_b), _ptr(ra),
                                     _ptr(ri), _ptr(ra_b), _ptr(ri_b), _ptr(rate), _ptr(state), state.stride(0),
-                                    _ptr(step.state_slots), T, W, parts, taps, _ptr(counters), _code(proj.dtype), self._stream())
+                                    _ptr(step.state_slots), _ptr(step.positions), T, W, parts, taps, _code(proj.dtype),
+                                    self._stream())
         if rc == self.UNSUPPORTED:
             return False
         self._check(rc, "rglru_step")

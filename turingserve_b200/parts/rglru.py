@@ -6,9 +6,9 @@ One fused projection gives, per token, [y (W) | x (W)] with biases.  u = causal 
 parts; in part n r = sigmoid(ra[n] u + ra.b[n]) and i = sigmoid(ri[n] u + ri.b[n]), square matrices [out, in].  Per channel,
 in 32-bit: log a = -scale r softplus(lam), S <- a S + sqrt(1 - a^2) i u.  Output: W_o (S gelu_tanh(y)).
 
-Nothing is cached per token.  The mixer declares one flat 32-bit state per request, [W values of S | (taps - 1) x W last
-filter inputs], zeroed when the request is admitted, so the first portion needs no branch and a captured step's padding
-rows update the null slot.
+Nothing is cached per token.  The mixer declares one flat 32-bit state per request, [W values of S | ring of taps x W
+filter inputs, the one of position p in place p % taps], zeroed when the request is admitted, so the first portion needs no
+branch and a captured step's padding rows update the null slot.
 """
 
 from __future__ import annotations
@@ -59,7 +59,7 @@ class RGLRU(Mixer):
         self.rate = (self.decay_scale * torch.nn.functional.softplus(t["lam"].double(), threshold=40.0)).float().contiguous()
 
     def state_need(self) -> StateNeed:
-        return StateNeed((self.taps * self.W,), torch.float32)
+        return StateNeed(((1 + (self.taps if self.taps > 1 else 0)) * self.W,), torch.float32)
 
     def forward(self, x: torch.Tensor, step, cache, state: torch.Tensor) -> torch.Tensor:
         ops = kernels.ops()

@@ -15,7 +15,8 @@ captured step.  The experts' weights are stacked [E, ff, hidden] and [E, hidden,
 
 Many rows (``LIBRARY_ROWS`` pairs or more, outside a capture): the group sizes are read back once, the input
 rows are gathered in sorted order, and every expert's rows go through ``ops().linear`` as a product of their own,
-i.e. to the many-row kernels and the vendor library that the dense products of such steps use.
+i.e. to the many-row kernels and the vendor library that the dense products of such steps use.  (With a table the host
+counts the groups itself from the step's ids, and nothing is read back.)
 
 Without a router (``table_rows``): an integer table ('table' [ids, top_k]) gives every token id its experts; the choices
 weigh 1 / top_k each, and the sort reads the table itself, so neither router scores nor weights exist.
@@ -27,6 +28,7 @@ output of the two.
 
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from turingserve_b200 import kernels
@@ -75,7 +77,7 @@ class RoutedMLP(FeedForward):
         if self.glu:
             self.glu_args = (float(spec.glu_limit), float(spec.glu_slope), float(spec.glu_offset))
             self.shared_glu_args = (float(spec.shared_glu_limit), float(spec.glu_slope), float(spec.glu_offset))
-        self.table = None
+        self.table = self.host_table = None
         self.w_router = self.w_up = self.w_down = self.correction = self.w_shared_up = self.w_shared_down = None
 
     def parameters(self) -> dict[str, ParamSpec]:
@@ -100,6 +102,7 @@ class RoutedMLP(FeedForward):
     def load(self, t: dict[str, torch.Tensor]) -> None:
         if self.table_rows:
             self.table = t["table"].contiguous()
+            self.host_table = self.table.cpu().numpy()
             lo, hi = int(self.table.min()), int(self.table.max())
             if lo < 0 or hi >= self.E:
                 raise ValueError(f"routed_mlp: the table names experts {lo} to {hi} of {self.E}")
@@ -163,13 +166,14 @@ class RoutedMLP(FeedForward):
         if step is None:
             raise ValueError("routed_mlp: a table of experts needs the step's token ids")
         offsets, order, place, tiles = kernels.ops().moe_align(step.input_ids, self.E, table=self.table)
-        y = self._experts(x, offsets, order, tiles, None)
+        y = self._experts(x, offsets, order, tiles, None, getattr(step, "host_ids", None))
         # (after the experts: where its last product is put off, no other may come between it and the sum)
         add = self._shared(x, may_defer=True) if self.shared_inter else None
         return RoutedSum(y, place, self.top, None, 1.0 / self.top, add)
 
-    def _experts(self, x: torch.Tensor, offsets, order, tiles, scale) -> torch.Tensor:
-        """The experts' outputs, float32 rows sorted by expert; ``scale``: what multiplies their inputs (None: nothing)."""
+    def _experts(self, x: torch.Tensor, offsets, order, tiles, scale, ids=None) -> torch.Tensor:
+        """The experts' outputs, float32 rows sorted by expert; ``scale``: what multiplies their inputs (None: nothing);
+        ``ids``: the tokens' ids on the host, with which a table's group sizes need no read-back."""
         ops = kernels.ops()
         T, top = x.shape[0], self.top
         y = torch.empty((T * top, self.hidden), dtype=torch.float32, device=x.device)
@@ -178,7 +182,11 @@ class RoutedMLP(FeedForward):
             # the experts' input rows in sorted order, weighted and rounded once (the products then read plain rows)
             xs = torch.empty((T * top, self.hidden), dtype=x.dtype, device=x.device)
             ops.moe_gather(xs, x, order, scale, top)
-            bounds = offsets[: self.E + 1].tolist()                      # the one read-back of this path
+            if self.table_rows and ids is not None:
+                counts = np.bincount(self.host_table[ids].reshape(-1), minlength=self.E)
+                bounds = [0] + np.cumsum(counts).tolist()
+            else:
+                bounds = offsets[: self.E + 1].tolist()                  # the one read-back of this path
             a = torch.empty((T * top, up_width), dtype=x.dtype, device=x.device)
             for e in range(self.E):
                 lo, hi = bounds[e], bounds[e + 1]
