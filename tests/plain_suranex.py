@@ -175,20 +175,19 @@ def clamped_expert(x: torch.Tensor, W: dict, p: str, limit: float) -> torch.Tens
 
 def table_moe(x: torch.Tensor, ids: torch.Tensor, W: dict, p: str, f: dict) -> torch.Tensor:
     """Every token's experts are its id's row of a table, with equal weights; a shared expert is added."""
-    table = W[p + "table"].long()
-    top = int(f["router"]["top"])
+    chosen = W[p + "table"].long()[ids]                                     # [T, top]
     out = torch.zeros_like(x)
-    for t in range(x.shape[0]):
-        for r in range(top):
-            e = int(table[int(ids[t]), r])
-            out[t] += clamped_expert(x[t:t + 1], W, f"{p}e{e}.", float(f["expert"]["limit"]))[0] / top
+    for e in range(int(f["router"]["experts"])):
+        rows = (chosen == e).any(dim=1)
+        if rows.any():
+            out[rows] += clamped_expert(x[rows], W, f"{p}e{e}.", float(f["expert"].get("limit", math.inf))) / chosen.shape[1]
     if f.get("shared"):
-        out = out + clamped_expert(x, W, p + "shared.", float(f["shared"]["limit"]))
+        out = out + clamped_expert(x, W, p + "shared.", float(f["shared"].get("limit", math.inf)))
     return out
 
 
 # -- the model -----------------------------------------------------------------------------------------------------------
-def forward(cfg: dict, W: dict, ids, layers_out: list | None = None, round_to=None) -> torch.Tensor:
+def forward(cfg: dict, W: dict, ids, layers_out: list | None = None) -> torch.Tensor:
     """Logits [T, vocab].  ``layers_out`` receives the stream after every layer."""
     ids = torch.as_tensor(ids, dtype=torch.long)
     positions = torch.arange(len(ids))
