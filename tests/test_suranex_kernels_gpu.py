@@ -337,3 +337,264 @@ def test_turned_values_hold_distances_only(ops, dtype, H, G, D, V, page):
         outs.append(run_attention(ops, q, [k], [v.to(dtype)], [1], page, 0.1, 0.0, 30, 0, fv, None))
     assert close(outs[0], outs[1], dtype, 10.0 if dtype == torch.float32 else 1.0)
     assert float(outs[0].float().abs().max()) > 0.1
+
+
+# -- the real-gated linear recurrent unit --------------------------------------------------------------------------------
+def unit_consts(g, W, blocks, taps, dtype):
+    rnd = lambda *s: torch.randn(*s, generator=g, device=DEV)
+    size = W // blocks
+    return SimpleNamespace(
+        conv=rnd(W, taps) * 0.5, conv_b=rnd(W) * 0.2, ra=(rnd(blocks, size, size) * 1.5 / math.sqrt(size)).to(dtype),
+        ri=(rnd(blocks, size, size) * 1.5 / math.sqrt(size)).to(dtype), ra_b=rnd(W) * 0.5, ri_b=rnd(W) * 0.5,
+        lam=6.0 * torch.rand(W, generator=g, device=DEV) - 6.5)
+
+
+def plain_unit(proj, c, W, round_u=None):
+    """One request's rows [T, y | x] -> (S gelu(y), final S) in 64-bit; ``round_u``: the filter's output rounded so."""
+    p = proj.double().cpu()
+    d = {n: getattr(c, n).double().cpu() for n in vars(c)}
+    blocks, size = d["ra"].shape[:2]
+    u = plain.causal_filter(p[:, W:], d["conv"], d["conv_b"])
+    if round_u is not None:
+        u = u.to(round_u).double()
+    r = plain.block_gate(u, d["ra"], d["ra_b"].view(blocks, size))
+    i = plain.block_gate(u, d["ri"], d["ri_b"].view(blocks, size))
+    S = plain.gated_recurrence(u, r, i, d["lam"])
+    return S * plain.gelu_tanh(p[:, :W]), S[-1]
+
+
+def run_unit(ops, proj, state, c, cuts, slots, W, blocks, taps, one_kernel=True):
+    """The rows of ``proj`` belong to len(slots) requests of equal length; ``cuts`` are the step sizes."""
+    rate = (8.0 * torch.nn.functional.softplus(c.lam.double())).float()
+    n_req, T = len(slots), proj.shape[0] // len(slots)
+    out = torch.empty(proj.shape[0], W, dtype=proj.dtype, device=DEV)
+    at, fused = 0, 0
+    for n in cuts:
+        rows = torch.cat([torch.arange(r * T + at, r * T + at + n) for r in range(n_req)]).to(DEV)
+        step = SimpleNamespace(q_start=i32([i * n for i in range(n_req + 1)]), state_slots=i32(slots), num_requests=n_req,
+                               token_request=i32([r for r in range(n_req) for _ in range(n)]), max_q_len=n,
+                               positions=i32([at + i for _ in range(n_req) for i in range(n)]))
+        p = proj[rows].contiguous()
+        o = torch.empty(len(rows), W, dtype=proj.dtype, device=DEV)
+        if one_kernel and ops.rglru_step(o, p, 0, W, c.conv, c.conv_b, c.ra, c.ri, c.ra_b, c.ri_b, rate, state, step, taps):
+            fused += 1
+        else:
+            u = torch.empty(len(rows), W, dtype=proj.dtype, device=DEV)
+            ops.short_filter(u, p, W, c.conv, c.conv_b, state, W, step, taps)
+            ab = torch.empty(len(rows), W, 2, device=DEV)
+            ops.rglru_gates(ab, u, c.ra, c.ri, c.ra_b, c.ri_b, rate)
+            ops.rglru_scan(o, ab, p, 0, W, state, step, taps)
+        out[rows] = o
+        at += n
+    assert at == T
+    return out, fused
+
+
+@DTYPES
+@pytest.mark.parametrize("W,blocks,taps", [(60, 3, 4), (36, 1, 1), (24, 8, 2), (64, 1, 3), (256, 4, 4), (96, 2, 8), (512, 2, 2),
+                                           (35, 5, 3), (640, 1, 4)])
+def test_recurrent_unit_whole_in_portions_and_token_by_token(ops, dtype, W, blocks, taps):
+    """The same tokens as one portion, in portions down to two tokens and one (shorter than the filter's memory), and one
+    by one (through the one-kernel step where it takes the shape, and through the chain): the plain outputs, states and
+    ring of inputs; requests whose slots are not their batch rows; slots of others untouched."""
+    g = torch.Generator(device=DEV).manual_seed(W + taps)
+    T, slots = 45, [4, 1, 6]
+    c = unit_consts(g, W, blocks, taps, dtype)
+    proj = torch.randn(3 * T, 2 * W, generator=g, device=DEV).to(dtype)
+    wants = [plain_unit(proj[r * T:(r + 1) * T], c, W, dtype if dtype == torch.bfloat16 else None) for r in range(3)]
+    width = (1 + (taps if taps > 1 else 0)) * W
+    lim = dict(rtol=1e-2, atol=6e-3) if dtype == torch.bfloat16 else dict(rtol=1e-4, atol=2e-5)
+    for cuts, one_kernel in (([T], True), ([16, 2, 1, 1, 5, 2, 2, 3, 13], True), ([1] * T, True), ([1] * T, False)):
+        state = torch.zeros(8, width, device=DEV)
+        state[0] = 7.0
+        out, fused = run_unit(ops, proj, state, c, cuts, slots, W, blocks, taps, one_kernel)
+        takes = dtype == torch.bfloat16 and (W // blocks) % 8 == 0
+        assert fused == (sum(1 for n in cuts if n == 1) if takes and one_kernel else 0)
+        for r, slot in enumerate(slots):
+            mine = proj[r * T:(r + 1) * T]
+            assert torch.allclose(out[r * T:(r + 1) * T].double().cpu(), wants[r][0], **lim), (cuts[:3], r)
+            assert torch.allclose(state[slot, :W].double().cpu(), wants[r][1], **lim), (cuts[:3], r)
+            if taps > 1:
+                ring = state[slot, W:].view(taps, W)
+                for t in range(T - taps + 1, T):
+                    assert torch.equal(ring[t % taps], mine[t, W:].float()), (cuts[:3], t)
+        assert float((state[0] - 7.0).abs().max()) == 0.0 and float(state[[2, 3, 5, 7]].abs().max()) == 0.0
+
+
+@DTYPES
+def test_recurrent_unit_long_portions_unequal_requests_and_many_rows(ops, dtype):
+    """Requests of 1 to 700 tokens in one launch (the scan's groups of 256 tokens, its eight-token segments, single tokens
+    beside portions), each against itself alone in other cuts; eleven single tokens (more than a block takes)."""
+    g = torch.Generator(device=DEV).manual_seed(4)
+    W, blocks, taps = 128, 2, 3
+    c = unit_consts(g, W, blocks, taps, dtype)
+    lens = [1, 700, 9, 256, 257, 8, 1, 30]
+    proj = torch.randn(sum(lens), 2 * W, generator=g, device=DEV).to(dtype)
+    rate = (8.0 * torch.nn.functional.softplus(c.lam.double())).float()
+    starts = [sum(lens[:i]) for i in range(len(lens) + 1)]
+    state = torch.zeros(9, 4 * W, device=DEV)
+    slots = [3, 0, 7, 1, 5, 2, 8, 4]
+    step = SimpleNamespace(q_start=i32(starts), state_slots=i32(slots), num_requests=len(lens), max_q_len=max(lens),
+                           token_request=i32([r for r, n in enumerate(lens) for _ in range(n)]),
+                           positions=i32([i for n in lens for i in range(n)]))
+    u, o = (torch.empty(sum(lens), W, dtype=dtype, device=DEV) for _ in range(2))
+    ab = torch.empty(sum(lens), W, 2, device=DEV)
+    ops.short_filter(u, proj, W, c.conv, c.conv_b, state, W, step, taps)
+    ops.rglru_gates(ab, u, c.ra, c.ri, c.ra_b, c.ri_b, rate)
+    ops.rglru_scan(o, ab, proj, 0, W, state, step, taps)
+    lim = dict(rtol=1e-2, atol=6e-3) if dtype == torch.bfloat16 else dict(rtol=1e-4, atol=2e-5)
+    for r, n in enumerate(lens):
+        mine = proj[starts[r]:starts[r + 1]]
+        want, S = plain_unit(mine, c, W, dtype if dtype == torch.bfloat16 else None)
+        assert torch.allclose(o[starts[r]:starts[r + 1]].double().cpu(), want, **lim), r
+        assert torch.allclose(state[slots[r], :W].double().cpu(), S, **lim), r
+        alone = torch.zeros(1, 4 * W, device=DEV)
+        cuts = [n] if n < 3 else [2, n - 2] if n < 20 else [n // 3, 2, n - n // 3 - 2]
+        again, _ = run_unit(ops, mine, alone, c, cuts, [0], W, blocks, taps)
+        assert close(again, o[starts[r]:starts[r + 1]], dtype, 1.0), r
+    many = torch.randn(11 * 3, 2 * W, generator=g, device=DEV).to(dtype)
+    state = torch.zeros(11, 4 * W, device=DEV)
+    out, _ = run_unit(ops, many, state, c, [1, 1, 1], list(range(10, -1, -1)), W, blocks, taps)
+    for r in range(11):
+        want, _ = plain_unit(many[3 * r:3 * r + 3], c, W, dtype if dtype == torch.bfloat16 else None)
+        assert torch.allclose(out[3 * r:3 * r + 3].double().cpu(), want, **lim), r
+
+
+@DTYPES
+def test_a_slow_channel_keeps_an_input_for_hundreds_of_tokens(ops, dtype):
+    """One loud input, then silence: a channel with lam far below zero still holds its share 600 tokens later, in portions
+    and one by one, a fast one has forgotten it; the addend keeps its digits where the decay is close to one."""
+    W, taps = 16, 1
+    c = SimpleNamespace(conv=torch.ones(W, 1, device=DEV), conv_b=torch.zeros(W, device=DEV),
+                        ra=torch.zeros(2, 8, 8, dtype=dtype, device=DEV), ri=torch.zeros(2, 8, 8, dtype=dtype, device=DEV),
+                        ra_b=torch.zeros(W, device=DEV), ri_b=torch.full((W,), 20.0, device=DEV),
+                        lam=torch.linspace(-9.5, 1.0, W, device=DEV))
+    T = 600
+    proj = torch.zeros(T, 2 * W, dtype=dtype, device=DEV)
+    proj[:, :W] = 3.0
+    proj[0, W:] = 2.0
+    want, S = plain_unit(proj, c, W)
+    assert float(S[0]) > 0.01 and float(S[-1]) == 0.0
+    for cuts in ([T], [2] * 300, [250, 300, 50], [1] * T):
+        state = torch.zeros(1, W, device=DEV)
+        run_unit(ops, proj, state, c, cuts, [0], W, 2, taps)
+        assert torch.allclose(state[0].double().cpu(), S, rtol=2e-4, atol=1e-7), cuts[:2]
+
+
+def test_gates_at_their_extremes(ops):
+    """Decays of one and of nothing: no NaN, no lost digits (64-bit formulas), in both engine types."""
+    for dtype in (torch.float32, torch.bfloat16):
+        W = 64
+        zr = torch.linspace(-40, 40, W, device=DEV)
+        u = torch.ones(5, W, dtype=dtype, device=DEV)
+        zero = torch.zeros(1, W, W, dtype=dtype, device=DEV)
+        for rate in (1e-6, 1e-3, 0.2, 0.3, 3.0, 30.0):
+            ab = torch.empty(5, W, 2, device=DEV)
+            ops.rglru_gates(ab, u, zero, zero, zr, torch.full((W,), 3.0, device=DEV), torch.full((W,), rate, device=DEV))
+            la = -torch.tensor(rate, dtype=torch.float32).double() * torch.sigmoid(zr.double().cpu())
+            want = torch.sqrt(-torch.expm1(2 * la)) * torch.sigmoid(torch.tensor(3.0, dtype=torch.float64))
+            assert torch.allclose(ab[0, :, 0].double().cpu(), torch.exp(la), rtol=3e-6, atol=1e-30)
+            assert torch.allclose(ab[4, :, 1].double().cpu(), want, rtol=1e-5, atol=1e-12), (dtype, rate)
+
+
+# -- experts by table, the clamped gated unit --------------------------------------------------------------------------------
+def test_pairs_are_sorted_by_the_tables_experts(ops):
+    g = torch.Generator().manual_seed(0)
+    for T, top, E, vocab in ((1, 2, 5, 11), (37, 3, 7, 50), (700, 2, 12, 300), (5, 1, 1, 4)):
+        table = torch.rand(vocab, E, generator=g).argsort(1)[:, :top].to(torch.int32)
+        ids = torch.randint(0, vocab, (T,), generator=g).to(torch.int32)
+        ids[0] = vocab - 1
+        offsets, order, place, tiles = ops.moe_align(ids.to(DEV), E, table=table.to(DEV).contiguous())
+        flat = table[ids.long()].reshape(-1)
+        off = offsets[:E + 1].tolist()
+        assert off == [0] + torch.bincount(flat.long(), minlength=E).cumsum(0).tolist()
+        order, place = order[:T * top].cpu().long(), place[:T * top].cpu().long()
+        assert torch.equal(order[place], torch.arange(T * top))
+        for e in range(E):
+            assert bool((flat[order[off[e]:off[e + 1]]] == e).all())
+
+
+def clamped(gate, up, limit):
+    g, u = torch.clamp(gate, max=limit), torch.clamp(up, -limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+
+
+@DTYPES
+@pytest.mark.parametrize("T,inter", [(3, 24), (70, 33), (300, 256), (1, 1)])
+def test_clamped_gated_unit_of_column_pairs(ops, dtype, T, inter):
+    g = torch.Generator(device=DEV).manual_seed(inter)
+    gu = (torch.randn(T, 2 * inter, generator=g, device=DEV) * 4).to(dtype)
+    for limit in (0.5, 3.0, float("inf")):
+        out = torch.empty(T, inter, dtype=dtype, device=DEV)
+        ops.glu_pairs(out, gu, (limit, 1.702, 1.0))
+        assert close(out, clamped(gu[:, 0::2].double(), gu[:, 1::2].double(), limit), dtype, 2.0)
+
+
+def test_clamped_gated_unit_of_a_product_left_unreduced(ops):
+    from turingserve_b200 import kernels
+    g = torch.Generator(device=DEV).manual_seed(1)
+    x = torch.randn(8, 1024, generator=g, device=DEV).to(torch.bfloat16)
+    w = (torch.randn(192, 1024, generator=g, device=DEV) * 0.1).to(torch.bfloat16)
+    gu = torch.empty(8, 192, dtype=torch.bfloat16, device=DEV)
+    put_off = ops.linear(gu, x, w, may_defer=True)
+    assert isinstance(put_off, kernels.LazyProduct)
+    a, b = (torch.empty(8, 96, dtype=torch.bfloat16, device=DEV) for _ in range(2))
+    ops.glu_pairs(a, put_off, (1.0, 1.702, 1.0))
+    ops.glu_pairs(b, ops.linear(torch.empty_like(gu), x, w), (1.0, 1.702, 1.0))
+    assert torch.equal(a, b)
+
+
+def table_part(dtype, W, E, top, ff, limit, shared, vocab, seed, rank_scale=1.0):
+    from turingserve_b200.config.model_config import RoutedMLPSpec
+    from turingserve_b200.parts.base import BuildContext, build
+    kw = dict(shared_intermediate_size=shared[0], shared_glu_limit=shared[1]) if shared else {}
+    part = build("feed_forward", RoutedMLPSpec(
+        num_experts=E, top_k=top, intermediate_size=ff, activation="clamped_glu", weight_on="output", gated=True, table_rows=vocab,
+        glu_limit=limit, **kw), BuildContext(W, dtype, torch.device(DEV), 0))
+    g = torch.Generator().manual_seed(seed)
+    weights = {}
+    for n, p in part.parameters().items():
+        if p.integer:
+            weights[n] = torch.rand(vocab, E, generator=g).argsort(1)[:, :top].to(torch.int32)
+        else:
+            weights[n] = (torch.randn(p.shape, generator=g) * 1.5 / math.sqrt(p.shape[1])).to(dtype)
+    part.load({n: t.to(DEV) for n, t in weights.items()})
+    ff_cfg = {"router": {"experts": E, "top": top}, "expert": {"limit": limit}}
+    if shared:
+        ff_cfg["shared"] = {"limit": shared[1]}
+    return part, {n: (t.double() if t.dtype.is_floating_point else t) for n, t in weights.items()}, ff_cfg
+
+
+@DTYPES
+@pytest.mark.parametrize("T", [1, 4, 20, 90, 700])
+@pytest.mark.parametrize("W,E,top,ff,limit,shared", [(72, 5, 2, 24, 0.8, (16, 0.5)), (64, 4, 4, 33, 1.5, None),
+                                                     (128, 9, 3, 64, 0.9, (96, 0.3)), (40, 3, 1, 8, 0.6, (8, 2.0))])
+def test_routed_experts_by_table(ops, dtype, T, W, E, top, ff, limit, shared):
+    """The few-row, tiled and per-expert product paths, with group sizes read back and counted on the host; the rows left
+    to the norm's kernel and the sum of its own."""
+    vocab = 61
+    part, weights, cfg = table_part(dtype, W, E, top, ff, limit, shared, vocab, W + top)
+    ids = torch.randint(0, vocab, (T,), generator=torch.Generator().manual_seed(T))
+    x = torch.randn(T, W, generator=torch.Generator(device=DEV).manual_seed(T), device=DEV).to(dtype)
+    want = plain.table_moe(x.double().cpu(), ids, weights, "", cfg)
+    for host in (None, ids.numpy()):
+        step = SimpleNamespace(input_ids=ids.to(torch.int32).to(DEV), host_ids=host)
+        got = part.forward(x, step)
+        assert close(got, want, dtype, 3.0), float((got.double().cpu() - want).abs().max())
+        pending = part.forward_pending(x, step)
+        stream, out = torch.zeros(T, W, device=DEV), torch.empty(T, W, dtype=dtype, device=DEV)
+        ops.post_norm(out, stream, pending.add, torch.ones(W, device=DEV), 1e-6, rows=pending.rows, place=pending.place,
+                      top=pending.top, scale=pending.scale)
+        assert close(stream, plain.unit_rms(want, 1e-6), dtype, 3.0)
+
+
+def test_experts_depend_on_the_id_alone(ops):
+    """Equal rows with different ids go to different experts, equal ids in different rows to the same ones."""
+    part, weights, cfg = table_part(torch.float32, 32, 6, 2, 16, 1.0, None, 20, 3)
+    x = torch.ones(20, 32, device=DEV)
+    step = SimpleNamespace(input_ids=i32(list(range(20))), host_ids=None)
+    got = part.forward(x, step)
+    for a in range(20):
+        for b in range(20):
+            same = set(weights["table"][a].tolist()) == set(weights["table"][b].tolist())
+            assert bool(torch.allclose(got[a], got[b], atol=1e-6)) == same
