@@ -1572,7 +1572,7 @@ def main() -> int:
                     help="which measurements to run (decode always runs); fewer for a profiler capture")
     ap.add_argument("--design", default="", choices=["", "komirax", "pizunex", "vofinex", "gugezen", "suranex"],
                     help="instead of the default workload: layers of this design beside layers of the closest other one (Komirax "
-                         "beside Qwen2, Pizunex beside Komirax) at the same width "
+                         "beside Qwen2, Pizunex, Vofinex and Gugezen beside Komirax, Suranex beside Gugezen) at the same width "
                          "(prefill and decode throughput, and each of the design's kernels alone)")
     ap.add_argument("--design-sizes", default="1.5b,7b", help="which of the design's layer sizes to run")
     a = ap.parse_args()

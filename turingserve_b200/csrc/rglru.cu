@@ -76,8 +76,8 @@ template <> struct RgVec<bf16, 4> {
 
 // grid (ceil(T / TOK), ceil(W / (V blockDim))): a thread takes V neighbouring channels of TOK neighbouring tokens; the
 // window of the filter slides through registers and is refilled (from the rows before, or the slot's memory) only at the
-// thread's first token and where another request begins.
-template <typename T, int TOK, int V>
+// thread's first token and where another request begins.  NT: the most taps the instance takes.
+template <typename T, int TOK, int V, int NT>
 __global__ void __launch_bounds__(128)
 short_filter_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ x, int x_stride, int x_off,
                     const float* __restrict__ conv_w, const float* __restrict__ conv_b, const float* __restrict__ state,
@@ -100,14 +100,14 @@ short_filter_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ x
       for (int e = 0; e < V; ++e) v[k][e] = 0.f;
     }
   }
-  float wgt[RG_MAX_TAPS][V], bias[V];                    // wgt[d]: the tap d tokens back
+  float wgt[NT][V], bias[V];                    // wgt[d]: the tap d tokens back
 #pragma unroll
   for (int e = 0; e < V; ++e) {
     bias[e] = conv_b != nullptr ? conv_b[c + e] : 0.f;
 #pragma unroll
-    for (int d = 0; d < RG_MAX_TAPS; ++d) wgt[d][e] = d < taps ? conv_w[(size_t)(c + e) * taps + keep - d] : 0.f;
+    for (int d = 0; d < NT; ++d) wgt[d][e] = d < taps ? conv_w[(size_t)(c + e) * taps + keep - d] : 0.f;
   }
-  float win[RG_MAX_TAPS][V];                             // win[d]: the input d + 1 tokens back
+  float win[NT][V];                             // win[d]: the input d + 1 tokens back
   int t_end = t_base;                                    // the end of the request the window belongs to
 #pragma unroll
   for (int k = 0; k < TOK; ++k) {
@@ -120,7 +120,7 @@ short_filter_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ x
         const int pos = positions[t];
         const float* ring = state + (size_t)slots[b] * state_stride + ring_off;        // [taps][W]
 #pragma unroll
-        for (int d = 0; d < RG_MAX_TAPS - 1; ++d)
+        for (int d = 0; d < NT - 1; ++d)
           if (d < keep) {
             const int rel = i - 1 - d;                   // counted from the step's first token
             const int at = pos - 1 - d;                  // the input's position in the sequence
@@ -137,11 +137,11 @@ short_filter_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ x
       for (int e = 0; e < V; ++e) {
         acc[e] = bias[e];
 #pragma unroll
-        for (int d = RG_MAX_TAPS - 1; d > 0; --d)
+        for (int d = NT - 1; d > 0; --d)
           if (d < taps) acc[e] = fmaf(wgt[d][e], win[d - 1][e], acc[e]);
         acc[e] = fmaf(wgt[0][e], v[k][e], acc[e]);
 #pragma unroll
-        for (int d = RG_MAX_TAPS - 2; d > 0; --d) win[d][e] = win[d - 1][e];
+        for (int d = NT - 2; d > 0; --d) win[d][e] = win[d - 1][e];
         win[0][e] = v[k][e];
       }
       RgVec<T, V>::store(out + (size_t)t * out_stride + c, acc);
@@ -524,13 +524,19 @@ TS_API int ts_short_filter(void* out, int out_stride, const void* x, int x_strid
                    !(((uintptr_t)out | (uintptr_t)x) & 7);
   const dim3 grid(few ? T : ceil_div(T, 8), ceil_div(W, vec ? 512 : 128));
   if (grid.y > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_short_filter: %d channels", W);
-#define TS_SF(TT, N, V)                                                                                                \
-  ts_launch(short_filter_kernel<TT, N, V>, grid, dim3(128), 0, s, (TT*)out, out_stride, (const TT*)x, x_stride, x_off, conv_w, \
+#define TS_SFT(TT, N, V, NT)                                                                                                \
+  ts_launch(short_filter_kernel<TT, N, V, NT>, grid, dim3(128), 0, s, (TT*)out, out_stride, (const TT*)x, x_stride, x_off, conv_w, \
             conv_b, state, (size_t)state_stride, (size_t)ring_off, token_request, q_start, slots, positions, T, W, taps)
+#define TS_SF(TT, N, V)                                          \
+  do {                                                            \
+    if (taps <= 4) TS_SFT(TT, N, V, 4);                           \
+    else TS_SFT(TT, N, V, RG_MAX_TAPS);                           \
+  } while (0)
   if (dtype == TS_F32) { if (few) TS_SF(float, 1, 1); else TS_SF(float, 8, 1); }
   else if (dtype == TS_BF16) { if (few) TS_SF(bf16, 1, 1); else if (vec) TS_SF(bf16, 8, 4); else TS_SF(bf16, 8, 1); }
   else TS_REFUSE(TS_ERR_DTYPE, "ts_short_filter: dtype %d", dtype);
 #undef TS_SF
+#undef TS_SFT
   TS_LAUNCH_CHECK();
 }
 
