@@ -112,7 +112,7 @@ def test_a_window_keeps_the_pages_of_the_first_tokens():
 
 def test_the_frequencies_of_the_product_are_the_plain_ones():
     ctx = BuildContext(8, torch.float32, torch.device("cpu"), 0)
-    for base, dims, sc in ((100.0, 8, (8.0, 40.0, 4.0, 1.0)), (10000.0, 64, (4.0, 2048.0, 32.0, 1.0)), (30.0, 12, None),
+    for base, dims, sc in ((100.0, 8, (8.0, 40.0, 4.0, 1.0)), (20000.0, 48, (4.0, 1500.0, 24.0, 1.0)), (30.0, 12, None),
                            (500000.0, 128, (16.0, 8192.0, 32.0, 2.0)), (50.0, 2, (2.0, 10.0, 1.0, 1.0))):
         scaling = dict(zip(("factor", "original", "fast", "slow"), sc)) if sc else None
         want, mag = plain.key_frequencies(base, dims, scaling)
