@@ -191,13 +191,22 @@ class TwinOps:
                 o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * out_scale
                 out[qs:qe, h * V:(h + 1) * V] = o.to(out.dtype)
 
-    def router_topk(self, idx, weights, x, w_router, softmax, renormalize, correction=None):
+    def router_topk(self, idx, weights, x, w_router, softmax, renormalize, correction=None, groups=1, keep=1, scale=1.0, share=None):
         z = F.linear(x.float(), w_router.float())
+        if share is not None:
+            share.copy_(torch.sigmoid(z[:, -1]))
+            z = z[:, :-1]
         scores = torch.softmax(z, -1) if softmax else torch.sigmoid(z)
-        best = (z if correction is None else scores + correction.float()).topk(idx.shape[1], dim=-1)
+        by = z if correction is None and groups == 1 else scores + (0.0 if correction is None else correction.float())
+        if groups > 1:
+            parts = by.view(by.shape[0], groups, -1)
+            strength = parts.topk(min(2, parts.shape[2]), dim=-1).values.sum(-1)
+            kept = torch.zeros_like(strength, dtype=torch.bool).scatter_(1, strength.topk(keep, dim=-1).indices, True)
+            by = parts.masked_fill(~kept[..., None], float("-inf")).view_as(by)
+        best = by.topk(idx.shape[1], dim=-1)
         idx.copy_(best.indices.to(torch.int32))
         w = scores.gather(1, best.indices)
-        weights.copy_(w / w.sum(-1, keepdim=True) if renormalize else w)
+        weights.copy_((w / w.sum(-1, keepdim=True) if renormalize else w) * scale)
 
     def moe_align(self, idx, E, with_tiles=None, table=None):
         flat = (idx if table is None else table[idx.long()]).reshape(-1).long()
@@ -236,7 +245,7 @@ class TwinOps:
             rows = rows * row_scale.reshape(-1)[pairs][:, None]
         xs.copy_(rows.to(xs.dtype))
 
-    def moe_combine(self, out, y, place, pair_weights, top, x=None, pass_from=None, add=None):
+    def moe_combine(self, out, y, place, pair_weights, top, x=None, pass_from=None, add=None, share=None):
         rows = y[place.long()].view(out.shape[0], top, -1)
         if x is not None:
             own = (place.long() >= int(pass_from)).view(out.shape[0], top, 1)
@@ -247,7 +256,7 @@ class TwinOps:
         for r in range(top):
             acc += rows[:, r]
         if add is not None:
-            acc += add.float()
+            acc += add.float() if share is None else share[:, None] * add.float()
         out.copy_(acc.to(out.dtype))
 
 
@@ -346,7 +355,7 @@ def _delta_scan(self, out, ready, proj, state, step, H, G, D, V, taps):
 def _head_gated_rmsnorm(self, out, x, gate, weight, eps, H, V):
     T = x.shape[0]
     o = x.float().view(T, H, V)
-    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float() * F.silu(gate.float()).view(T, H, V)
+    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float().view(-1, V) * F.silu(gate.float()).view(T, H, V)
     out.copy_(o.reshape(T, H * V).to(out.dtype))
 
 
@@ -387,19 +396,42 @@ def _rotate(x, cos, sin):
     return out
 
 
-def _latent_kv_write(self, proj, col0, weight, eps, positions, freq, magnitude, rot_dims, k_cache, slots, rank, R, page_size):
+def _rotate_by(x, cos, sin, pairing):
+    if pairing == "neighbours":
+        return _rotate(x, cos, sin)
+    n = cos.shape[1]
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [n]
+    c, s = cos.view(shape), sin.view(shape)
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
+def _latent_kv_write(self, proj, col0, weight, eps, positions, freq, magnitude, rot_dims, k_cache, slots, rank, R, page_size,
+                     pairing="neighbours", cq=None, q_weight=None, keep=(0, 0)):
+    if cq is not None:
+        _rms_rows(self, cq, proj, 0, q_weight, eps)
+    if slots is None:
+        return proj
     c = proj[:, col0:col0 + rank].float()
     c = c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
     cos, sin = _pair_angles(positions, freq, magnitude)
-    kr = _rotate(proj[:, col0 + rank:col0 + rank + R].float(), cos[:, :rot_dims // 2], sin[:, :rot_dims // 2])
+    kr = _rotate_by(proj[:, col0 + rank:col0 + rank + R].float(), cos[:, :rot_dims // 2], sin[:, :rot_dims // 2], pairing)
     m = slots >= 0
     sl = slots[m].long()
     k_cache[sl // page_size, 0, sl % page_size, :] = torch.cat([c, kr], -1)[m].to(k_cache.dtype)
+    return proj
 
 
-def _rotate_pairs(self, dst, src, positions, freq, magnitude, rot_dims):
+def _rotate_pairs(self, dst, src, positions, freq, magnitude, rot_dims, pairing="neighbours"):
     cos, sin = _pair_angles(positions, freq, magnitude)
-    dst.copy_(_rotate(src.float(), cos[:, :rot_dims // 2], sin[:, :rot_dims // 2]).to(dst.dtype))
+    dst.copy_(_rotate_by(src.float(), cos[:, :rot_dims // 2], sin[:, :rot_dims // 2], pairing).to(dst.dtype))
+
+
+def _latent_queries(self, qa, q, w, positions, freq, magnitude, rot_dims, pairing):
+    H, N, K = w.shape
+    heads = q.view(q.shape[0], H, -1)
+    self.batched_linear(qa[:, :, :N], heads[:, :, :K], w)
+    self.rotate_pairs(qa[:, :, N:], heads[:, :, K:], positions, freq, magnitude, rot_dims, pairing)
 
 
 def _batched_linear(self, out, x, w):
@@ -715,6 +747,52 @@ def _rglru_scan(self, out, ab, proj, y_off, x_off, state, step, taps):
 def _rglru_step(self, *args):
     return False                        # (the chain of the three above serves every step here)
 
+
+# -- the time mixer with a state that fades channel by channel ------------------------------------------------------------
+def _token_shift(self, out, h, mu, state, prev_off, step):
+    qs, slots = step.q_start.tolist(), step.state_slots.tolist()
+    hidden = h.shape[1]
+    before = torch.zeros(h.shape)
+    before[1:] = h[:-1].float()
+    for b in range(step.num_requests):
+        if qs[b + 1] > qs[b]:
+            before[qs[b]] = state[slots[b]][prev_off:prev_off + hidden]
+    x = h.float()
+    for i in range(out.shape[0]):
+        out[i] = (x + (before - x) * mu[i].float()).to(out.dtype)
+
+
+def _wkv_decay(self, out, z, w2, w0):
+    out.copy_(torch.exp(-torch.exp(torch.tanh(z.float()) @ w2.float().t() + w0.float())))
+
+
+def _wkv_scan(self, out, r, k, v, w, u, h, state, step, H, D):
+    qs, slots = step.q_start.tolist(), step.state_slots.tolist()
+    heads = lambda x, t: x[t].float().view(H, D)
+    for b in range(step.num_requests):
+        lo, hi = qs[b], qs[b + 1]
+        if hi <= lo:
+            continue
+        row = state[slots[b]]
+        S = row[:H * D * D].view(H, D, D)
+        for t in range(lo, hi):
+            kv = heads(k, t)[:, :, None] * heads(v, t)[:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S + u.view(H, D, 1) * kv, heads(r, t)).reshape(-1)
+            S.mul_(heads(w, t)[:, :, None]).add_(kv)
+        row[H * D * D:] = h[hi - 1].float()
+
+
+def _wkv_project(self, *args):
+    return False                        # (the general chain serves every step here)
+
+
+def _wkv_step(self, *args):
+    return False
+
+
+for _name, _fn in (("token_shift", _token_shift), ("wkv_decay", _wkv_decay), ("wkv_scan", _wkv_scan), ("wkv_project", _wkv_project),
+                   ("wkv_step", _wkv_step), ("latent_queries", _latent_queries)):
+    setattr(TwinOps, _name, _fn)
 
 for _name, _fn in (("post_norm", _post_norm), ("qkv_heads_write", _qkv_heads_write), ("glu_pairs", _glu_pairs),
                    ("grouped_glu", _grouped_glu), ("short_filter", _short_filter), ("rglru_gates", _rglru_gates),

@@ -367,7 +367,9 @@ class LatentAttentionSpec:
     """Attention through low-rank latents: queries W_uq rms(W_dq h), per head [``nope_dim`` plain |
     ``rope_dim`` rotated]; per token one latent c = rms(first ``kv_rank`` rows of W_dkv h) and one rotated key
     part (the last ``rope_dim`` rows) that every head uses; head by head the keys are W_uk c and the values W_uv c.
-    Causal softmax of (q_plain . k_plain + q_rot . k_rot) * scale.  The cache holds c and the rotated key part only."""
+    Causal softmax of (q_plain . k_plain + q_rot . k_rot) * scale.  The cache holds c and the rotated key part only.
+    ``window`` w: position i sees i - w < j <= i.  ``sinks``: the softmax's denominator also holds exp(sink_h) ('sink').
+    ``head_gate``: head h's output times sigmoid(W_g h)_h, one number per head ('g')."""
 
     num_heads: int
     nope_dim: int
@@ -378,7 +380,25 @@ class LatentAttentionSpec:
     scale: float
     norm_eps: float
     position: Any = None                # a position-encoding spec for the rotated parts
+    window: int | None = None
+    sinks: bool = False
+    head_gate: bool = False
     kind: str = "latent_attention"
+
+
+@dataclass(frozen=True)
+class WKVSpec:
+    """Time mixer with a matrix state per head that fades channel by channel at rates the token chooses (RWKV, sixth
+    generation).  r, k, v, the gate and the decay each read a mix h + (h' - h) mu of the present input and the one before; the decay
+    is exp(-exp(W_w2 tanh(W_w1 mix) + w0)); per head o = (S + diag(u) k v^T)^T r, S <- diag(w) S + k v^T; every head's o is
+    divided by its root mean square, times a weight, times silu(gate), then projected.  ``decay_rank``: the rows of W_w1
+    (None: as many as the checkpoint has)."""
+
+    num_heads: int
+    head_dim: int
+    norm_eps: float
+    decay_rank: int | None = None
+    kind: str = "wkv"
 
 
 @dataclass(frozen=True)
@@ -402,7 +422,10 @@ class RoutedMLPSpec:
     form ('shared.up', 'shared.down') that every token uses, added unweighted.  ``table_rows`` not None: no router; an integer
     table ('table' [table_rows, top_k]) gives every token id its experts, each with weight 1 / top_k.  ``activation``
     "clamped_glu" (gated only): g sigmoid(glu_slope g) (u + glu_offset) with g = min(gate, glu_limit), u = clamp(up, +-glu_limit);
-    the shared expert has a limit of its own (``shared_glu_limit``)."""
+    the shared expert has a limit of its own (``shared_glu_limit``).  ``groups``: so many equal groups of neighbouring experts, of
+    which only the ``groups_kept`` whose two largest choice scores (with the correction) have the largest sums may be chosen
+    from.  ``weight_scale``: a constant the weights are multiplied by.  ``shared_gate``: the shared expert's output times
+    sigmoid(W_sg h), one number a token ('shared.sg')."""
 
     num_experts: int
     top_k: int
@@ -420,6 +443,10 @@ class RoutedMLPSpec:
     shared_glu_limit: float = float("inf")
     glu_slope: float = 1.702
     glu_offset: float = 1.0
+    groups: int = 1
+    groups_kept: int = 1
+    weight_scale: float = 1.0
+    shared_gate: bool = False
     kind: str = "routed_mlp"
 
 

@@ -129,3 +129,5 @@ def _load_builtin() -> None:
         from turingserve_b200.models import gugezen  # noqa: F401
     if "Suranex" not in _ARCHITECTURES:
         from turingserve_b200.models import suranex  # noqa: F401
+    if "Fetedra" not in _ARCHITECTURES:
+        from turingserve_b200.models import fetedra  # noqa: F401

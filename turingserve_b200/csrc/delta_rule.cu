@@ -11,7 +11,7 @@
 //                         inputs for the tokens before the step's first, writes nothing to the slot
 //   ts_delta_scan         the recurrence, token by token for portions and single tokens alike (cutting a prompt
 //                         changes no bit); afterwards the request's blocks store the filter's new last inputs
-//   ts_head_gated_rmsnorm o / rms(o) per head, times a weight shared by the heads, times silu(gate)
+//   ts_head_gated_rmsnorm o / rms(o) per head, times a weight (shared by the heads or one a head), times silu(gate)
 //
 // The scan: one pass over the state per token.  With a = (g S)^T k and c = (g S)^T q, both sums over the old
 // state, u = beta (v - a) and o = c + (k.q) u, so the read-out needs no second pass after the write.  A column
@@ -251,7 +251,7 @@ delta_scan_kernel(float* __restrict__ out, const float* __restrict__ ready, cons
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_gated_rmsnorm_kernel(T* __restrict__ out, const float* __restrict__ x, const T* __restrict__ gate, int gate_stride,
-                          const float* __restrict__ w, float eps, int H, int V) {
+                          const float* __restrict__ w, int w_stride, float eps, int H, int V) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -259,13 +259,14 @@ head_gated_rmsnorm_kernel(T* __restrict__ out, const float* __restrict__ x, cons
   for (int h = blockIdx.y * nwarps + warp; h < H; h += gridDim.y * nwarps) {      // a warp a head
     const float* xr = x + ((size_t)t * H + h) * V;
     const T* gr = gate + (size_t)t * gate_stride + (size_t)h * V;
+    const float* wh = w + (size_t)h * w_stride;
     float ss = 0.f;
     for (int i = lane; i < V; i += 32) ss = fmaf(xr[i], xr[i], ss);
     ss = warp_sum(ss);
     const float rstd = 1.f / sqrtf(ss / (float)V + eps);
     for (int i = lane; i < V; i += 32) {
       const float z = to_f(gr[i]);
-      out[((size_t)t * H + h) * V + i] = from_f<T>(xr[i] * rstd * w[i] * (z / (1.f + expf(-z))));
+      out[((size_t)t * H + h) * V + i] = from_f<T>(xr[i] * rstd * wh[i] * silu_for<T>(z));
     }
   }
 }
@@ -358,18 +359,18 @@ TS_API int ts_delta_scan(float* out, const float* ready, const void* proj, int p
   TS_LAUNCH_CHECK();
 }
 
-// out [T, H V] = x / sqrt(mean over a head's V of x^2 + eps) * w[V] * silu(gate); x 32-bit [T, H V]; gate rows
-// gate_stride apart.
-TS_API int ts_head_gated_rmsnorm(void* out, const float* x, const void* gate, int gate_stride, const float* w, float eps,
-                                 int T, int H, int V, int dtype, void* stream) {
+// out [T, H V] = x / sqrt(mean over a head's V of x^2 + eps) * w * silu(gate); x 32-bit [T, H V]; gate rows gate_stride
+// apart; w: head h's weights [V] from h * w_stride on (w_stride 0: the same for all heads).
+TS_API int ts_head_gated_rmsnorm(void* out, const float* x, const void* gate, int gate_stride, const float* w, int w_stride,
+                                 float eps, int T, int H, int V, int dtype, void* stream) {
   if (T <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   // few tokens: the heads of a token spread over blocks of four warps; many: one block a token
   const int heads_y = T >= 512 ? 1 : min(ceil_div(H, 4), 65535);
   if (dtype == TS_F32)
-    ts_launch(head_gated_rmsnorm_kernel<float>, dim3(T, heads_y), dim3(128), 0, s, (float*)out, x, (const float*)gate, gate_stride, w, eps, H, V);
+    ts_launch(head_gated_rmsnorm_kernel<float>, dim3(T, heads_y), dim3(128), 0, s, (float*)out, x, (const float*)gate, gate_stride, w, w_stride, eps, H, V);
   else if (dtype == TS_BF16)
-    ts_launch(head_gated_rmsnorm_kernel<bf16>, dim3(T, heads_y), dim3(128), 0, s, (bf16*)out, x, (const bf16*)gate, gate_stride, w, eps, H, V);
+    ts_launch(head_gated_rmsnorm_kernel<bf16>, dim3(T, heads_y), dim3(128), 0, s, (bf16*)out, x, (const bf16*)gate, gate_stride, w, w_stride, eps, H, V);
   else
     TS_REFUSE(TS_ERR_DTYPE, "ts_head_gated_rmsnorm: dtype %d", dtype);
   TS_LAUNCH_CHECK();

@@ -6,7 +6,9 @@
 //   ts_router_topk     z = Wr x in 32-bit (one block a token, fixed summation order), score = sigmoid(z) or
 //                      softmax(z); the `top` largest by z (ties: the lower index), or, with a correction vector, by
 //                      score + correction; weights = their scores (never the correction), optionally divided by
-//                      their sum.
+//                      their sum, times a constant.  With groups of neighbouring experts only those of the groups whose
+//                      two largest choice scores have the largest sums may be chosen.  One more router row may give
+//                      every token the sigmoid by which a shared expert is weighted.
 //   ts_moe_align       pairs p = t * top + r sorted by expert: offsets[E + 1], order[P] (sorted place -> pair),
 //                      place[P] (pair -> sorted place), and the list of row tiles (expert, first row) the
 //                      grouped products walk; experts from `with_tiles` on get a group but no tiles (experts
@@ -41,24 +43,26 @@ template <typename T>
 __global__ void __launch_bounds__(RT_THREADS)
 router_topk_kernel(int* __restrict__ idx_out, float* __restrict__ w_out, const T* __restrict__ x,
                    const float* __restrict__ wr, int T_, int E, int K, int top, int softmax, int renorm,
-                   const float* __restrict__ correction) {
+                   const float* __restrict__ correction, int groups, int keep, float scale, float* __restrict__ share) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float smem[];
-  float* z = smem;                       // [E]
-  float* part = smem + E;                // [RT_THREADS / 32][8]
+  const int rows = E + (share != nullptr ? 1 : 0);     // (the shared expert's row lies behind the experts')
+  float* z = smem;                       // [E + 1]
+  float* part = z + E + 1;               // [RT_THREADS / 32][8]
   float* pick = part + RT_THREADS / 32 * 8;   // [E] what the choice goes by, when it is not z itself
+  float* gsum = pick + E;                // [groups]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
   const T* xr = x + (size_t)t * K;
-  for (int e0 = 0; e0 < E; e0 += 8) {
+  for (int e0 = 0; e0 < rows; e0 += 8) {
     float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
 #pragma unroll 2
     for (int k = threadIdx.x; k < K; k += RT_THREADS) {
       const float xv = to_f(xr[k]);
 #pragma unroll
       for (int i = 0; i < 8; ++i)
-        if (e0 + i < E) acc[i] = fmaf(xv, __ldg(wr + (size_t)(e0 + i) * K + k), acc[i]);
+        if (e0 + i < rows) acc[i] = fmaf(xv, __ldg(wr + (size_t)(e0 + i) * K + k), acc[i]);
     }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
@@ -66,7 +70,7 @@ router_topk_kernel(int* __restrict__ idx_out, float* __restrict__ w_out, const T
       if (lane == 0) part[warp * 8 + i] = v;
     }
     __syncthreads();
-    if (threadIdx.x < 8 && e0 + threadIdx.x < E) {
+    if (threadIdx.x < 8 && e0 + threadIdx.x < rows) {
       float v = 0.f;
       for (int w = 0; w < RT_THREADS / 32; ++w) v += part[w * 8 + threadIdx.x];
       z[e0 + threadIdx.x] = v;
@@ -84,10 +88,38 @@ router_topk_kernel(int* __restrict__ idx_out, float* __restrict__ w_out, const T
     denom = warp_sum(d);
   }
   const float* by = z;
-  if (correction != nullptr) {
+  if (share != nullptr && lane == 0) share[t] = 1.f / (1.f + expf(-z[E]));
+  const bool own_pick = correction != nullptr || groups > 1;
+  if (own_pick) {
     for (int e = lane; e < E; e += 32)
-      pick[e] = (softmax ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e]))) + correction[e];
+      pick[e] = (softmax ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e]))) + (correction != nullptr ? correction[e] : 0.f);
     by = pick;
+    __syncwarp();
+  }
+  if (groups > 1) {
+    const int size = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;                // the two largest of the group
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = pick[e];
+        if (v > a) {
+          b = a;
+          a = v;
+        } else if (v > b) {
+          b = v;
+        }
+      }
+      gsum[g] = size > 1 ? a + b : a;
+    }
+    __syncwarp();
+    // a group stays when fewer than `keep` others stand before it (a larger sum, or an equal one and a lower index)
+    for (int g = lane; g < groups; g += 32) {
+      const float own = gsum[g];
+      int before = 0;
+      for (int o = 0; o < groups; ++o) before += (gsum[o] > own || (gsum[o] == own && o < g)) ? 1 : 0;
+      if (before >= keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) pick[e] = -INFINITY;
+    }
     __syncwarp();
   }
   float total = 0.f;
@@ -111,19 +143,20 @@ router_topk_kernel(int* __restrict__ idx_out, float* __restrict__ w_out, const T
       }
     }
     if (arg == 0x7fffffff) arg = 0;              // only when every score left is -inf or NaN
-    const float logit = correction != nullptr ? z[arg] : best;
+    const float logit = own_pick ? z[arg] : best;
     const float score = softmax ? expf(logit - zmax) / denom : 1.f / (1.f + expf(-logit));
     total += score;
     if (lane == 0) {
       idx_out[(size_t)t * top + r] = arg;
       w_out[(size_t)t * top + r] = score;
-      if (correction != nullptr) pick[arg] = -INFINITY;
+      if (own_pick) pick[arg] = -INFINITY;
       else z[arg] = -INFINITY;
     }
     __syncwarp();
   }
-  if (renorm && lane == 0)
-    for (int r = 0; r < top; ++r) w_out[(size_t)t * top + r] /= (total + 1e-20f);
+  if ((renorm || scale != 1.f) && lane == 0)
+    for (int r = 0; r < top; ++r)
+      w_out[(size_t)t * top + r] = (renorm ? w_out[(size_t)t * top + r] / (total + 1e-20f) : w_out[(size_t)t * top + r]) * scale;
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -492,7 +525,8 @@ __global__ void moe_gather_kernel(T* __restrict__ xs, const T* __restrict__ x, c
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ y, const int* __restrict__ place,
                                    const float* __restrict__ pair_w, int top, int N, const T* __restrict__ x,
-                                   const int* __restrict__ pass_from, const T* __restrict__ add) {
+                                   const int* __restrict__ pass_from, const T* __restrict__ add,
+                                   const float* __restrict__ share) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -505,7 +539,8 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
       const float v = at >= first_pass ? to_f(x[(size_t)t * N + n]) : y[(size_t)at * N + n];
       acc += pair_w != nullptr ? pair_w[p] * v : v;
     }
-    if (add != nullptr) acc += to_f(add[(size_t)t * N + n]);       // (an expert that every token uses)
+    // (an expert that every token uses, weighted where a weight per token is given)
+    if (add != nullptr) acc += share != nullptr ? share[t] * to_f(add[(size_t)t * N + n]) : to_f(add[(size_t)t * N + n]);
     out[(size_t)t * N + n] = from_f<T>(acc);
   }
 }
@@ -589,20 +624,25 @@ TS_API int ts_glu_pairs(void* out, const void* gu, const float* part, int splits
 TS_API int ts_moe_tile_rows() { return GL_BM; }
 
 // x: [T, K] in `dtype`; wr: [E, K] 32-bit.  idx_out / w_out: [T, top].
-// correction: 32-bit [E] or null.
+// correction: 32-bit [E] or null.  groups, keep: groups of E / groups neighbouring experts of which the best `keep` may be
+// chosen from (1, 1: no groups).  scale: what the weights are multiplied by.  share [T] not null: wr has one more row, and the
+// sigmoid of its logit goes there.
 TS_API int ts_router_topk(int* idx_out, float* w_out, const void* x, const float* wr, int T, int E, int K, int top,
-                          int softmax, int renorm, int dtype, const float* correction, void* stream) {
+                          int softmax, int renorm, int dtype, const float* correction, int groups, int keep, float scale,
+                          float* share, void* stream) {
   if (T <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E) TS_REFUSE(TS_ERR_SHAPE, "ts_router_topk: top %d of %d experts", top, E);
   if (E > 2048) TS_REFUSE(TS_ERR_LIMIT, "ts_router_topk: %d experts (limit 2048)", E);
   cudaStream_t s = (cudaStream_t)stream;
-  const size_t smem = sizeof(float) * (2 * E + RT_THREADS / 32 * 8);
+  if (groups < 1 || keep < 1 || keep > groups || E % groups || (groups > 1 && top > E / groups * keep))
+    TS_REFUSE(TS_ERR_SHAPE, "ts_router_topk: %d of %d groups of %d experts, top %d", keep, groups, E, top);
+  const size_t smem = sizeof(float) * (2 * E + 1 + RT_THREADS / 32 * 8 + groups);
   if (dtype == TS_F32)
     ts_launch(router_topk_kernel<float>, dim3(T), dim3(RT_THREADS), smem, s, idx_out, w_out, (const float*)x, wr, T,
-              E, K, top, softmax, renorm, correction);
+              E, K, top, softmax, renorm, correction, groups, keep, scale, share);
   else if (dtype == TS_BF16)
     ts_launch(router_topk_kernel<bf16>, dim3(T), dim3(RT_THREADS), smem, s, idx_out, w_out, (const bf16*)x, wr, T,
-              E, K, top, softmax, renorm, correction);
+              E, K, top, softmax, renorm, correction, groups, keep, scale, share);
   else
     TS_REFUSE(TS_ERR_DTYPE, "ts_router_topk: dtype %d", dtype);
   TS_LAUNCH_CHECK();
@@ -710,15 +750,15 @@ TS_API int ts_grouped_glu(void* out, const void* x, const void* w, const int* or
 
 // x (out's type, [T, N]) and pass_from (one int on the device): pairs sorted to place *pass_from or later add the
 // token's own row of x instead of a row of y; both null: none do.  add (out's type, [T, N], may be null): added to
-// every token's sum.
+// every token's sum, times share[t] where share (32-bit [T]) is given.
 TS_API int ts_moe_combine(void* out, const float* y, const int* place, const float* pair_w, int T, int top, int N, int dtype,
-                          const void* x, const int* pass_from, const void* add, void* stream) {
+                          const void* x, const int* pass_from, const void* add, const float* share, void* stream) {
   if (T <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == TS_F32)
-    ts_launch(moe_combine_kernel<float>, dim3(T), dim3(256), 0, s, (float*)out, y, place, pair_w, top, N, (const float*)x, pass_from, (const float*)add);
+    ts_launch(moe_combine_kernel<float>, dim3(T), dim3(256), 0, s, (float*)out, y, place, pair_w, top, N, (const float*)x, pass_from, (const float*)add, share);
   else if (dtype == TS_BF16)
-    ts_launch(moe_combine_kernel<bf16>, dim3(T), dim3(256), 0, s, (bf16*)out, y, place, pair_w, top, N, (const bf16*)x, pass_from, (const bf16*)add);
+    ts_launch(moe_combine_kernel<bf16>, dim3(T), dim3(256), 0, s, (bf16*)out, y, place, pair_w, top, N, (const bf16*)x, pass_from, (const bf16*)add, share);
   else
     TS_REFUSE(TS_ERR_DTYPE, "ts_moe_combine: dtype %d", dtype);
   TS_LAUNCH_CHECK();

@@ -3,15 +3,17 @@
 //   ts_rms_rows          out = x[:, col0 : col0 + n] / rms * w               (a column slice of wider rows)
 //   ts_qk_rownorm_write  q and k normed over their WHOLE rows (all heads at once), q times a temperature that grows
 //                        with the position; normed keys into the key cache, the keys as projected into the value cache
-//   ts_latent_kv_write   one cached row a token: [rms(latent) * w | rotated key part]
-//   ts_rotate_pairs      rotation of neighbouring pairs (2i, 2i+1), angle = position * freq[i] in 32-bit, cosine and
-//                        sine times a magnitude; strided source and destination
+//   ts_latent_kv_write   one cached row a token: [rms(latent) * w | rotated key part]; beside it the normed query latent
+//   ts_rotate_pairs      rotation of pairs, neighbours (2i, 2i+1) or halves (i, i + R/2), angle = position * freq[i] in
+//                        32-bit, cosine and sine times a magnitude; strided source and destination
+//   ts_latent_queries    few rows: a query's plain part into the latent space (a product per head) and its rotated part turned
 //   ts_rope_headnorm_write  rotation of the pairs (i, i + R/2) of every q and k head, angle = position * freq[i] in 32-bit,
 //                        then each head over its root mean square (no weight); q in place, k and v rows into a cache
 //                        whose key and value rows have widths of their own
-//   ts_batched_linear    out[t, h, :] = w[h] x[t, h, :], a product per head over strided rows (FFMA, fixed k order; up to
-//                        16 rows: a warp an output column, streaming its weight row)
+//   ts_batched_linear    out[t, h, :] = w[h] x[t, h, :], a product per head over strided rows (up to 16 rows, bfloat16: tensor
+//                        cores, a warp eight output columns; 32-bit: a warp an output column; else FFMA tiles, fixed k order)
 #include "common.cuh"
+#include "mma_utils.cuh"
 
 namespace {
 
@@ -79,65 +81,93 @@ __device__ __forceinline__ void pair_angle(int pos, float f, float magnitude, fl
   s *= magnitude;
 }
 
+// The pair (low, high) of rotated dimensions number i: neighbours (2i, 2i + 1) or, with halves, (i, i + rot_dims / 2).
+__device__ __forceinline__ void pair_dims(int i, int rot_dims, int halves, int& low, int& high) {
+  low = halves ? i : 2 * i;
+  high = halves ? i + rot_dims / 2 : 2 * i + 1;
+}
+
+// One block a token (blockIdx.y == 0): the cached row; with `cq`, a second one: the query latent, rms(columns 0 .. q_rank) * q_w.
+// `part` set: the projection is still [splits, T, stride] partial sums; a column's value is their sum in ascending order
+// rounded to the storage type, and the columns [keep0, keep0 + keep_n), which a later kernel reads, are left finished in `proj`.
 template <typename T>
-__global__ void latent_kv_write_kernel(const T* __restrict__ proj, int stride, int col0, const float* __restrict__ w,
+__global__ void latent_kv_write_kernel(T* __restrict__ proj, int stride, int col0, const float* __restrict__ w,
                                        float eps, const int* __restrict__ positions, const float* __restrict__ freq,
-                                       float magnitude, int rot_dims, T* __restrict__ k_cache,
-                                       const int* __restrict__ slots, int rank, int R, int page) {
+                                       float magnitude, int rot_dims, int halves, T* __restrict__ k_cache,
+                                       const int* __restrict__ slots, int rank, int R, int page, T* __restrict__ cq,
+                                       const float* __restrict__ q_w, int q_rank, const float* __restrict__ part, int splits,
+                                       int keep0, int keep_n) {
   pdl_launch_dependents();
   pdl_wait();
+  extern __shared__ float lk_s[];
   __shared__ float scratch[32];
   const int t = blockIdx.x;
-  const int slot = slots[t];
-  if (slot < 0) return;
-  const T* row = proj + (size_t)t * stride + col0;
+  T* row = proj + (size_t)t * stride;
+  const float* prow = part != nullptr ? part + (size_t)t * stride : nullptr;
+  const size_t split_stride = (size_t)gridDim.x * stride;
+  auto value = [&](int c) {
+    if (prow == nullptr) return to_f(row[c]);
+    float v = 0.f;
+    for (int sp = 0; sp < splits; ++sp) v += __ldcg(prow + sp * split_stride + c);
+    return round_to<T>(v);
+  };
+  const bool query = blockIdx.y == 1;
+  const int slot = (query || slots == nullptr) ? -1 : slots[t];
+  if (!query && prow != nullptr)
+    for (int i = threadIdx.x; i < keep_n; i += blockDim.x) row[keep0 + i] = from_f<T>(value(keep0 + i));
+  if (!query && slot < 0) return;
+  const int first = query ? 0 : col0, n = query ? q_rank : rank;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-    const float v = to_f(row[i]);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float v = value(first + i);
+    lk_s[i] = v;
     ss = fmaf(v, v, ss);
   }
-  ss = block_sum(ss, scratch);
-  const float rstd = 1.f / sqrtf(ss / (float)rank + eps);
-  T* dst = k_cache + ((size_t)(slot / page) * page + slot % page) * (rank + R);        // one kv head
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f<T>(to_f(row[i]) * rstd * w[i]);
+  if (!query)
+    for (int i = threadIdx.x; i < R; i += blockDim.x) lk_s[rank + i] = value(col0 + rank + i);
+  ss = block_sum(ss, scratch);                           // (its barriers also publish lk_s)
+  const float rstd = 1.f / sqrtf(ss / (float)n + eps);
+  T* dst = query ? cq + (size_t)t * q_rank : k_cache + ((size_t)(slot / page) * page + slot % page) * (rank + R);   // one kv head
+  const float* wt = query ? q_w : w;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_f<T>(lk_s[i] * rstd * wt[i]);
+  if (query) return;
   const int pos = positions[t];
-  for (int i = threadIdx.x; i < R / 2 + (R & 1); i += blockDim.x) {
-    const int d = 2 * i;
-    if (d < rot_dims) {                                  // (rot_dims is even and at most R)
-      float c, s;
-      pair_angle(pos, freq[i], magnitude, c, s);
-      const float u = to_f(row[rank + d]), v = to_f(row[rank + d + 1]);
-      dst[rank + d] = from_f<T>(u * c - v * s);
-      dst[rank + d + 1] = from_f<T>(v * c + u * s);
-    } else {
-      dst[rank + d] = row[rank + d];
-      if (d + 1 < R) dst[rank + d + 1] = row[rank + d + 1];
-    }
+  const float* kr = lk_s + rank;
+  for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {      // (rot_dims is even and at most R)
+    int lo, hi;
+    pair_dims(i, rot_dims, halves, lo, hi);
+    float c, s;
+    pair_angle(pos, freq[i], magnitude, c, s);
+    const float u = kr[lo], v = kr[hi];
+    dst[rank + lo] = from_f<T>(u * c - v * s);
+    dst[rank + hi] = from_f<T>(v * c + u * s);
   }
+  for (int i = rot_dims + threadIdx.x; i < R; i += blockDim.x) dst[rank + i] = from_f<T>(kr[i]);
 }
 
 template <typename T>
 __global__ void rotate_pairs_kernel(T* __restrict__ dst, int dst_ts, int dst_hs, const T* __restrict__ src, int src_ts,
                                     int src_hs, const int* __restrict__ positions, const float* __restrict__ freq,
-                                    float magnitude, int rot_dims, int H, int R) {
+                                    float magnitude, int rot_dims, int halves, int H, int R) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   const int pos = positions[t];
-  const int half = R / 2 + (R & 1);
-  for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
-    const int h = idx / half, i = idx % half, d = 2 * i;
+  const int pairs = rot_dims / 2, per = pairs + R - rot_dims;          // (rot_dims is even and at most R)
+  for (int idx = threadIdx.x; idx < H * per; idx += blockDim.x) {
+    const int h = idx / per, i = idx % per;
     const T* a = src + (size_t)t * src_ts + (size_t)h * src_hs;
     T* o = dst + (size_t)t * dst_ts + (size_t)h * dst_hs;
-    if (d < rot_dims) {                                  // (rot_dims is even and at most R)
+    if (i < pairs) {
+      int lo, hi;
+      pair_dims(i, rot_dims, halves, lo, hi);
       float c, s;
       pair_angle(pos, freq[i], magnitude, c, s);
-      const float u = to_f(a[d]), v = to_f(a[d + 1]);
-      o[d] = from_f<T>(u * c - v * s);
-      o[d + 1] = from_f<T>(v * c + u * s);
+      const float u = to_f(a[lo]), v = to_f(a[hi]);
+      o[lo] = from_f<T>(u * c - v * s);
+      o[hi] = from_f<T>(v * c + u * s);
     } else {
-      o[d] = a[d];
-      if (d + 1 < R) o[d + 1] = a[d + 1];
+      o[rot_dims + i - pairs] = a[rot_dims + i - pairs];
     }
   }
 }
@@ -236,6 +266,169 @@ batched_linear_rows_kernel(T* __restrict__ out, int out_ts, int out_hs, const T*
       if (lane == 0 && m0 + r < M) out[(size_t)(m0 + r) * out_ts + (size_t)h * out_hs + n] = from_f<T>(v);
     }
   }
+}
+
+// Few bfloat16 rows on the tensor cores: out[m, h, :] = w[h] x[m, h, :] for up to ROWS (8 or 16) rows.  A warp owns eight output
+// columns of one head and one of KS shares of k, whose weights it has on their way before the wait for the predecessor; the
+// rows go through shared memory once a block.  `x` may be the partial sums of a product cut along its own k (part [splits, M,
+// x_ts] 32-bit, summed in ascending order and rounded as that product's last pass would have).  (The products' k index is a
+// permutation of the real one, the same for both operands.)  The last block of a head (rot_dst set) turns R further columns of
+// its rows, those behind the first K, instead: the rotated part of a query beside its plain part's product.
+constexpr int BRM_WARPS = 8, BRM_UNROLL = 8, BRM_PAD = 32;
+
+struct RowRotation {
+  bf16* dst;                     // [M, H, R] by out's strides; null: none
+  const int* positions;
+  const float* freq;
+  float magnitude;
+  int rot_dims, halves, R;
+};
+
+template <int ROWS, int KS>
+__global__ void __launch_bounds__(BRM_WARPS * 32)
+batched_rows_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, const bf16* __restrict__ x, int x_ts, int x_hs,
+                        const float* __restrict__ part, int splits, const bf16* __restrict__ w, int M, int N, int K,
+                        RowRotation rot) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) unsigned char brm_smem[];
+  bf16* x_s = reinterpret_cast<bf16*>(brm_smem);                      // [ROWS][K + BRM_PAD]
+  __shared__ float red[BRM_WARPS][ROWS][8];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  const int h = blockIdx.y;
+  const size_t split_stride = (size_t)M * x_ts;
+  auto value = [&](int m, int c) {
+    const size_t at = (size_t)m * x_ts + (size_t)h * x_hs + c;
+    if (part == nullptr) return to_f(x[at]);
+    float v = 0.f;
+    for (int sp = 0; sp < splits; ++sp) v += __ldcg(part + sp * split_stride + at);
+    return round_to<bf16>(v);
+  };
+  if (rot.dst != nullptr && blockIdx.x == gridDim.x - 1) {
+    pdl_wait();
+    const int pairs = rot.rot_dims / 2, per = pairs + rot.R - rot.rot_dims;
+    for (int idx = threadIdx.x; idx < M * per; idx += blockDim.x) {
+      const int m = idx / per, i = idx % per;
+      bf16* o = rot.dst + (size_t)m * out_ts + (size_t)h * out_hs;
+      if (i < pairs) {
+        int lo, hi;
+        pair_dims(i, rot.rot_dims, rot.halves, lo, hi);
+        float c, s;
+        pair_angle(rot.positions[m], rot.freq[i], rot.magnitude, c, s);
+        const float u = value(m, K + lo), v = value(m, K + hi);
+        o[lo] = from_f<bf16>(u * c - v * s);
+        o[hi] = from_f<bf16>(v * c + u * s);
+      } else {
+        const int d = rot.rot_dims + i - pairs;
+        o[d] = from_f<bf16>(value(m, K + d));
+      }
+    }
+    return;
+  }
+  constexpr int GROUPS = BRM_WARPS / KS;                              // column groups a block
+  const int ks = warp % KS, cg = warp / KS;
+  const int n0 = (blockIdx.x * GROUPS + cg) * 8;
+  const bool n_ok = n0 + g < N;
+  const bf16* wrow = w + ((size_t)h * N + (n_ok ? n0 + g : 0)) * K + t * 8;
+  const int steps = (K + 31) / 32, share = (steps + KS - 1) / KS;
+  const int st0 = ks * share, st1 = min(st0 + share, steps);
+  uint4 wv[BRM_UNROLL];
+  auto fetch = [&](int st) {
+#pragma unroll
+    for (int q = 0; q < BRM_UNROLL; ++q)
+      wv[q] = (n_ok && st + q < st1 && (st + q) * 32 + t * 8 < K) ? *reinterpret_cast<const uint4*>(wrow + (st + q) * 32)
+                                                                  : make_uint4(0u, 0u, 0u, 0u);
+  };
+  fetch(st0);
+  pdl_wait();
+  const int xs = K + BRM_PAD;
+  for (int i = threadIdx.x * 8; i < ROWS * K; i += BRM_WARPS * 32 * 8) {
+    const int m = i / K, c = i - m * K;
+    uint4 o = make_uint4(0u, 0u, 0u, 0u);
+    if (m < M) {
+      const size_t at = (size_t)m * x_ts + (size_t)h * x_hs + c;
+      if (part == nullptr) {
+        o = *reinterpret_cast<const uint4*>(x + at);
+      } else {
+        float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        for (int sp = 0; sp < splits; ++sp) {
+          const float4* p4 = reinterpret_cast<const float4*>(part + sp * split_stride + at);
+          const float4 a = __ldcg(p4), b = __ldcg(p4 + 1);
+          f[0] += a.x; f[1] += a.y; f[2] += a.z; f[3] += a.w;
+          f[4] += b.x; f[5] += b.y; f[6] += b.z; f[7] += b.w;
+        }
+        __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) oh[j] = __floats2bfloat162_rn(f[2 * j], f[2 * j + 1]);
+      }
+    }
+    *reinterpret_cast<uint4*>(x_s + m * xs + c) = o;
+  }
+  __syncthreads();
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int st = st0; st < st1; st += BRM_UNROLL) {
+    if (st != st0) fetch(st);
+#pragma unroll
+    for (int q = 0; q < BRM_UNROLL; ++q) {
+      const int kk = (st + q) * 32 + t * 8;
+      const bool ok = st + q < st1 && kk < K;
+      const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+      const uint4 xv = ok ? *reinterpret_cast<const uint4*>(x_s + g * xs + kk) : zero;
+      uint4 yv = zero;
+      if constexpr (ROWS == 16) yv = ok ? *reinterpret_cast<const uint4*>(x_s + (g + 8) * xs + kk) : zero;
+      const unsigned a1[4] = {xv.x, yv.x, xv.y, yv.y}, a2[4] = {xv.z, yv.z, xv.w, yv.w};
+      mma_bf16(acc, a1, wv[q].x, wv[q].y);
+      mma_bf16(acc, a2, wv[q].z, wv[q].w);
+    }
+  }
+  if constexpr (KS > 1) {
+    if (ks != 0) {
+#pragma unroll
+      for (int hh = 0; hh < ROWS / 8; ++hh)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) red[warp][g + 8 * hh][2 * t + e] = acc[2 * hh + e];
+    }
+    __syncthreads();
+    if (ks != 0) return;
+#pragma unroll
+    for (int o = 1; o < KS; ++o)
+#pragma unroll
+      for (int hh = 0; hh < ROWS / 8; ++hh)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) acc[2 * hh + e] += red[warp + o][g + 8 * hh][2 * t + e];
+  }
+#pragma unroll
+  for (int hh = 0; hh < ROWS / 8; ++hh)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int m = g + 8 * hh, c = n0 + 2 * t + e;
+      if (m < M && c < N) out[(size_t)m * out_ts + (size_t)h * out_hs + c] = from_f<bf16>(acc[2 * hh + e]);
+    }
+}
+
+int launch_batched_rows_mma(bf16* out, int out_ts, int out_hs, const bf16* x, int x_ts, int x_hs, const float* part, int splits,
+                            const bf16* w, int M, int H, int N, int K, const RowRotation& rot, cudaStream_t s) {
+  const int ks = K >= 256 ? 4 : 1;
+  const dim3 grid(ceil_div(N, BRM_WARPS / ks * 8) + (rot.dst != nullptr ? 1 : 0), H);
+#define TS_BRM(ROWS, KS)                                                                                                     \
+  do {                                                                                                                       \
+    const size_t smem = (size_t)ROWS * (K + BRM_PAD) * 2;                                                                    \
+    static size_t configured = 0;                                                                                            \
+    if (smem > 40 * 1024 && smem > configured) {                                                                             \
+      cudaError_t e = cudaFuncSetAttribute(batched_rows_mma_kernel<ROWS, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      if (e != cudaSuccess) TS_REFUSE((int)e, "ts_batched_linear: shared memory %zu: %s", smem, cudaGetErrorString(e));      \
+      configured = smem;                                                                                                     \
+    }                                                                                                                        \
+    ts_launch(batched_rows_mma_kernel<ROWS, KS>, grid, dim3(BRM_WARPS * 32), smem, s, out, out_ts, out_hs, x, x_ts, x_hs, part, splits, \
+              w, M, N, K, rot);                                                                                              \
+  } while (0)
+  if (M <= 8) { if (ks == 4) TS_BRM(8, 4); else TS_BRM(8, 1); }
+  else { if (ks == 4) TS_BRM(16, 4); else TS_BRM(16, 1); }
+#undef TS_BRM
+  TS_LAUNCH_CHECK();
+}
+
+bool rows_mma_takes(int M, int x_ts, int x_hs, int K, const void* x, const void* w) {
+  return M <= 16 && K % 8 == 0 && K <= 4096 && x_ts % 8 == 0 && x_hs % 8 == 0 && !(((uintptr_t)x | (uintptr_t)w) & 15);
 }
 
 // One warp a (token, head), RHN_WARPS heads a block.  The head's D values pass through shared memory: rotated in
@@ -452,30 +645,53 @@ TS_API int ts_qk_rownorm_write(void* proj, int stride, const float* q_w, const f
   TS_LAUNCH_CHECK();
 }
 
-// proj [T, stride]: the latent in columns [col0, col0 + rank), the key part to rotate in the R columns behind it.
-// k_cache [pages, 1, page, rank + R].
-TS_API int ts_latent_kv_write(const void* proj, int stride, int col0, const float* w, float eps, const int* positions,
-                              const float* freq, float magnitude, int rot_dims, void* k_cache, const int* slots, int T,
-                              int rank, int R, int page, int dtype, void* stream) {
+// proj [T, stride]: the latent in columns [col0, col0 + rank), the key part to rotate in the R columns behind it; halves: pairs
+// (i, i + rot_dims / 2), else neighbours.  k_cache [pages, 1, page, rank + R]; slots null: nothing is cached.  cq [T, q_rank]
+// (null: none): the columns [0, q_rank) normed with q_w.  part [splits, T, stride] (null: proj is finished): the projection's
+// partial sums; the columns [keep0, keep0 + keep_n) are then left finished in proj.
+TS_API int ts_latent_kv_write(void* proj, int stride, int col0, const float* w, float eps, const int* positions,
+                              const float* freq, float magnitude, int rot_dims, int halves, void* k_cache, const int* slots,
+                              int T, int rank, int R, int page, void* cq, const float* q_w, int q_rank, const float* part,
+                              int splits, int keep0, int keep_n, int dtype, void* stream) {
   if (T <= 0) return 0;
   if (rot_dims % 2 || rot_dims > R) TS_REFUSE(TS_ERR_SHAPE, "ts_latent_kv_write: %d rotated dimensions of %d", rot_dims, R);
+  const int widest = max(rank + R, cq != nullptr ? q_rank : 0);
+  const size_t smem = sizeof(float) * widest;
+  if (smem > 47 * 1024) TS_REFUSE(TS_ERR_LIMIT, "ts_latent_kv_write: rows of %d", widest);
   cudaStream_t s = (cudaStream_t)stream;
   TS_BY_TYPE("ts_latent_kv_write",
-             ts_launch(latent_kv_write_kernel<TT>, dim3(T), dim3(threads_for_row(rank)), 0, s, (const TT*)proj, stride, col0, w,
-                       eps, positions, freq, magnitude, rot_dims, (TT*)k_cache, slots, rank, R, page));
+             ts_launch(latent_kv_write_kernel<TT>, dim3(T, cq != nullptr ? 2 : 1), dim3(threads_for_row(widest)), smem, s, (TT*)proj,
+                       stride, col0, w, eps, positions, freq, magnitude, rot_dims, halves, (TT*)k_cache, slots, rank, R, page,
+                       (TT*)cq, q_w, q_rank, part, splits, keep0, keep_n));
   TS_LAUNCH_CHECK();
 }
 
 // dst[t, h, :R] = rotate(src[t, h, :R]); strides in elements.
 TS_API int ts_rotate_pairs(void* dst, int dst_ts, int dst_hs, const void* src, int src_ts, int src_hs, const int* positions,
-                           const float* freq, float magnitude, int rot_dims, int T, int H, int R, int dtype, void* stream) {
+                           const float* freq, float magnitude, int rot_dims, int halves, int T, int H, int R, int dtype,
+                           void* stream) {
   if (T <= 0 || H <= 0 || R <= 0) return 0;
   if (rot_dims % 2 || rot_dims > R) TS_REFUSE(TS_ERR_SHAPE, "ts_rotate_pairs: %d rotated dimensions of %d", rot_dims, R);
   cudaStream_t s = (cudaStream_t)stream;
   TS_BY_TYPE("ts_rotate_pairs",
              ts_launch(rotate_pairs_kernel<TT>, dim3(T), dim3(threads_for_row(H * R / 2)), 0, s, (TT*)dst, dst_ts, dst_hs,
-                       (const TT*)src, src_ts, src_hs, positions, freq, magnitude, rot_dims, H, R));
+                       (const TT*)src, src_ts, src_hs, positions, freq, magnitude, rot_dims, halves, H, R));
   TS_LAUNCH_CHECK();
+}
+
+// Queries of a latent attention, at most 16 bfloat16 rows: qa[m, h, :N] = w[h] q[m, h, :K], qa[m, h, N : N + R] = rotate(q[m, h, K
+// : K + R]).  q [M, H, K + R] contiguous, or its partial sums part [splits, M, H (K + R)].  UNSUPPORTED: the caller takes the
+// product, ts_batched_linear and ts_rotate_pairs.
+TS_API int ts_latent_queries(void* qa, int qa_ts, int qa_hs, const void* q, const float* part, int splits, const void* w,
+                             const int* positions, const float* freq, float magnitude, int rot_dims, int halves, int M, int H,
+                             int N, int K, int R, int dtype, void* stream) {
+  if (M <= 0 || H <= 0) return 0;
+  if (rot_dims % 2 || rot_dims > R) TS_REFUSE(TS_ERR_SHAPE, "ts_latent_queries: %d rotated dimensions of %d", rot_dims, R);
+  if (dtype != TS_BF16 || !rows_mma_takes(M, H * (K + R), K + R, K, q, w) || ((uintptr_t)part & 15) || H > 65535)
+    TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_latent_queries: %d rows of %d + %d", M, K, R);
+  RowRotation rot = {(bf16*)qa + N, positions, freq, magnitude, rot_dims, halves, R};
+  return launch_batched_rows_mma((bf16*)qa, qa_ts, qa_hs, (const bf16*)q, H * (K + R), K + R, part, splits, (const bf16*)w, M, H, N,
+                                 K, rot, (cudaStream_t)stream);
 }
 
 // proj [T, stride]: q heads in columns [0, H D), k heads in [k_off, k_off + G D), value rows in [v_off, v_off + G V).
@@ -599,6 +815,9 @@ TS_API int ts_batched_linear(void* out, int out_ts, int out_hs, const void* x, i
   dim3 grid(ceil_div(N, BL_N), ceil_div(T, BL_M), H);
   if (grid.y > 65535 || H > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_batched_linear: %d rows / %d heads per launch", T, H);
   cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == TS_BF16 && rows_mma_takes(T, x_ts, x_hs, K, x, w))
+    return launch_batched_rows_mma((bf16*)out, out_ts, out_hs, (const bf16*)x, x_ts, x_hs, nullptr, 0, (const bf16*)w, T, H, N, K,
+                                   RowRotation{}, s);
   const int per = dtype == TS_F32 ? 4 : 8;
   if (T <= 2 * BLR_ROWS && K % per == 0 && x_ts % per == 0 && x_hs % per == 0 && !((uintptr_t)x & 15) && !((uintptr_t)w & 15)) {
     dim3 rows_grid(ceil_div(N, BLR_WARPS), H);

@@ -1,0 +1,653 @@
+// A time mixer whose matrix state fades channel by channel at rates the token chooses (the sixth generation of RWKV; Peng et
+// al., "Eagle and Finch: RWKV with Matrix-Valued States and Dynamic Recurrence").  For every request and head a state S [D, V]
+// in 32-bit lives in a state slot between steps; per token, with r, k, v and a decay w in (0, 1) per key channel,
+//     o = (S + diag(u) k v^T)^T r,        S <- diag(w) S + k v^T          (the bonus u counts for the present token only).
+// r, k, v, the gate and the decay each read a mix of the token's input h and the one before it, h + (h' - h) mu; the decay is
+// w = exp(-exp(w2 tanh(w1 mix) + w0)).  The slot holds [H D V values of S | the last input h], all 32-bit.
+//
+//   ts_token_shift    the mixes of every token, [n, T, hidden]; the row before a request's first token comes from the slot
+//   ts_wkv_decay      w [T, H D] in 32-bit from the first product's 32-bit rows (tanh, second product, the two exponentials)
+//   ts_wkv_scan       the recurrence, token by token for portions and single tokens alike (cutting a prompt changes no bit);
+//                     afterwards the request's blocks store the last input
+//   ts_wkv_project    steps in which every token is a request of its own: the mixes and their products in one kernel
+//   ts_wkv_step       ... and the decay's second product, the recurrence, the heads' norm and the gate in another
+#include "activations.cuh"
+#include "common.cuh"
+#include "mma_utils.cuh"
+
+namespace {
+
+__device__ __forceinline__ void wk_cp_async_4(void* smem, const void* gmem) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(s), "l"(gmem));
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// A thread owns PER neighbouring channels of TOK neighbouring tokens; the row before slides through registers.
+constexpr int SH_MAX = 8;                                     // mixes a launch makes
+
+template <typename T, int PER, int TOK>
+__global__ void __launch_bounds__(128)
+token_shift_kernel(T* __restrict__ out, const T* __restrict__ h, const T* __restrict__ mu, const float* __restrict__ state,
+                   size_t state_stride, size_t prev_off, const int* __restrict__ token_request, const int* __restrict__ q_start,
+                   const int* __restrict__ slots, int T_, int hidden, int n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * PER;
+  if (c >= hidden) return;
+  const int t_base = blockIdx.x * TOK;
+  const int count = min(TOK, T_ - t_base);
+  float cur[TOK][PER], before[PER];
+#pragma unroll
+  for (int k = 0; k < TOK; ++k)
+    if (k < count) {
+      if constexpr (PER == 8) {
+        const uint4 v = *reinterpret_cast<const uint4*>(h + (size_t)(t_base + k) * hidden + c);
+        const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+        for (int j = 0; j < PER; ++j) cur[k][j] = to_f(e[j]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) cur[k][j] = to_f(h[(size_t)(t_base + k) * hidden + c + j]);
+      }
+    }
+#pragma unroll
+  for (int k = 0; k < TOK; ++k) {
+    if (k < count) {
+      const int t = t_base + k, b = token_request[t];
+      if (t == q_start[b]) {
+        const float* prev = state + (size_t)slots[b] * state_stride + prev_off + c;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) before[j] = prev[j];
+      } else if (k == 0) {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) before[j] = to_f(h[(size_t)(t - 1) * hidden + c + j]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) before[j] = cur[k > 0 ? k - 1 : 0][j];
+      }
+#pragma unroll
+      for (int i = 0; i < SH_MAX; ++i) {
+        if (i < n) {
+          T* dst = out + ((size_t)i * T_ + t) * hidden + c;
+          const T* m = mu + (size_t)i * hidden + c;
+          if constexpr (PER == 8) {
+            const uint4 mv = __ldg(reinterpret_cast<const uint4*>(m));
+            const T* me = reinterpret_cast<const T*>(&mv);
+            uint4 o;
+            T* oe = reinterpret_cast<T*>(&o);
+#pragma unroll
+            for (int j = 0; j < PER; ++j) oe[j] = from_f<T>(fmaf(before[j] - cur[k][j], to_f(me[j]), cur[k][j]));
+            *reinterpret_cast<uint4*>(dst) = o;
+          } else {
+#pragma unroll
+            for (int j = 0; j < PER; ++j) dst[j] = from_f<T>(fmaf(before[j] - cur[k][j], to_f(m[j]), cur[k][j]));
+          }
+        }
+      }
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// out[t, c] = exp(-exp(sum_r w2[c, r] tanh(z[t, r]) + w0[c])): FFMA tiles of 64 tokens x 64 channels, r in ascending order.
+constexpr int DC_M = 64, DC_N = 64, DC_K = 16, DC_PAD = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+wkv_decay_kernel(float* __restrict__ out, const float* __restrict__ z, const T* __restrict__ w2, const float* __restrict__ w0,
+                 int M, int N, int R) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ __align__(16) float As[DC_K][DC_M + DC_PAD];
+  __shared__ __align__(16) float Ws[DC_K][DC_N + DC_PAD];
+  const int tid = threadIdx.x;
+  const int m0 = blockIdx.y * DC_M, n0 = blockIdx.x * DC_N;
+  const int lr = tid >> 2, lk = (tid & 3) * 4;
+  const int ty = tid >> 4, tx = tid & 15;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < R; k0 += DC_K) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int k = k0 + lk + i;
+      As[lk + i][lr] = (m0 + lr < M && k < R) ? tanhf(z[(size_t)(m0 + lr) * R + k]) : 0.f;
+      Ws[lk + i][lr] = (n0 + lr < N && k < R) ? to_f(w2[(size_t)(n0 + lr) * R + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < DC_K; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&As[k][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&Ws[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n < N) out[(size_t)m * N + n] = expf(-expf(acc[i][j] + w0[n]));
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// One block owns WK_COLS columns of one (head, request) state and keeps them in registers over the step's tokens: thread
+// (part, col) holds rows part * WK_ROWS .. of column col.  Tokens come in groups; a warp brings whole tokens (r, k, v as
+// stored, w in 32-bit) by cp.async while the group before is computed, turns its own tokens into 32-bit rows in shared memory
+// and sums r u k, the weight with which the token's own value enters its output.  Two block-wide barriers a group.
+constexpr int WK_GROUP = 16, WK_COLS = 16, WK_ROWS = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(512, 1)
+wkv_scan_kernel(float* __restrict__ out, const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v,
+                const float* __restrict__ w, const float* __restrict__ u, const T* __restrict__ h_in,
+                float* __restrict__ state, size_t state_stride, const int* __restrict__ q_start,
+                const int* __restrict__ slots, int H, int D, int V, int hidden, int parts, int fast) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float smem[];
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int t0 = q_start[b], n = q_start[b + 1] - t0;
+  if (n <= 0) return;
+  const int Dp = parts * WK_ROWS;                          // D rounded up: rows beyond D hold zeros
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+  const int col = threadIdx.x & (WK_COLS - 1), part = threadIdx.x / WK_COLS;
+  const int j = blockIdx.x * WK_COLS + col;
+  const int cols_here = min(WK_COLS, V - (int)blockIdx.x * WK_COLS);
+  const bool live = col < cols_here;
+  float* base = state + (size_t)slots[b] * state_stride;
+  float* S = base + (size_t)h * D * V;
+  float* r_s = smem;                                       // [WK_GROUP][Dp]
+  float* k_s = r_s + WK_GROUP * Dp;                        // [WK_GROUP][Dp]
+  float* w_s = k_s + WK_GROUP * Dp;                        // [2][WK_GROUP][Dp]
+  float* u_s = w_s + 2 * WK_GROUP * Dp;                    // [Dp]
+  float* v_s = u_s + Dp;                                   // [2][WK_GROUP][WK_COLS]
+  float* c_s = v_s + 2 * WK_GROUP * WK_COLS;               // [2][WK_GROUP]: the sum of r u k
+  float* o_s = c_s + 2 * WK_GROUP;                         // [WK_GROUP][parts][WK_COLS]
+  T* raw = reinterpret_cast<T*>(o_s + WK_GROUP * parts * WK_COLS);   // [2][WK_GROUP][D r | D k | WK_COLS v]
+  const int raw_row = 2 * D + WK_COLS;
+  const int HD = H * D, HV = H * V;
+  constexpr int PER = 16 / (int)sizeof(T);
+
+  float s[WK_ROWS];
+#pragma unroll
+  for (int i = 0; i < WK_ROWS; ++i) {
+    const int d = part * WK_ROWS + i;
+    s[i] = (live && d < D) ? S[(size_t)d * V + j] : 0.f;
+  }
+  for (int i = threadIdx.x; i < 4 * WK_GROUP * Dp; i += blockDim.x) smem[i] = 0.f;
+  for (int i = threadIdx.x; i < Dp; i += blockDim.x) u_s[i] = i < D ? u[h * D + i] : 0.f;
+  __syncthreads();
+
+  auto fetch = [&](int g0, int buf) {
+    const int gn = min(WK_GROUP, n - g0);
+    for (int q = warp; q < gn; q += nwarps) {
+      const size_t t = t0 + g0 + q;
+      const T* rr = r + t * HD + h * D;
+      const T* kr = k + t * HD + h * D;
+      const T* vr = v + t * HV + h * V + blockIdx.x * WK_COLS;
+      const float* wr = w + t * HD + h * D;
+      T* dst = raw + ((size_t)buf * WK_GROUP + q) * raw_row;
+      float* wd = w_s + ((size_t)buf * WK_GROUP + q) * Dp;
+      if (fast) {
+        for (int c = lane * PER; c < D; c += 32 * PER) {
+          cp_async_16(dst + c, rr + c, true);
+          cp_async_16(dst + D + c, kr + c, true);
+        }
+        for (int c = lane * 4; c < D; c += 128) cp_async_16(wd + c, wr + c, true);
+        if (lane * PER < cols_here) cp_async_16(dst + 2 * D + lane * PER, vr + lane * PER, true);
+      } else {
+        for (int c = lane; c < D; c += 32) {
+          dst[c] = rr[c];
+          dst[D + c] = kr[c];
+          wk_cp_async_4(wd + c, wr + c);
+        }
+        for (int c = lane; c < cols_here; c += 32) dst[2 * D + c] = vr[c];
+      }
+    }
+  };
+  fetch(0, 0);
+  cp_async_commit();
+  int buf = 0;
+  for (int g0 = 0; g0 < n; g0 += WK_GROUP, buf ^= 1) {
+    const int gn = min(WK_GROUP, n - g0);
+    if (g0 + WK_GROUP < n) fetch(g0 + WK_GROUP, buf ^ 1);
+    cp_async_commit();
+    cp_async_wait<1>();
+    __syncwarp();                                          // (a warp turns the tokens that it brought itself)
+    float* vg = v_s + buf * WK_GROUP * WK_COLS;
+    float* cg = c_s + buf * WK_GROUP;
+    for (int q = warp; q < gn; q += nwarps) {
+      const T* src = raw + ((size_t)buf * WK_GROUP + q) * raw_row;
+      float c = 0.f;
+      if (fast) {                                          // (D is even then)
+        for (int d = 2 * lane; d < D; d += 64) {
+          const float r0 = to_f(src[d]), r1 = to_f(src[d + 1]), k0 = to_f(src[D + d]), k1 = to_f(src[D + d + 1]);
+          *reinterpret_cast<float2*>(r_s + q * Dp + d) = make_float2(r0, r1);
+          *reinterpret_cast<float2*>(k_s + q * Dp + d) = make_float2(k0, k1);
+          const float2 uu = *reinterpret_cast<const float2*>(u_s + d);
+          c = fmaf(r0 * uu.x, k0, c);
+          c = fmaf(r1 * uu.y, k1, c);
+        }
+      } else {
+        for (int d = lane; d < D; d += 32) {
+          const float r0 = to_f(src[d]), k0 = to_f(src[D + d]);
+          r_s[q * Dp + d] = r0;
+          k_s[q * Dp + d] = k0;
+          c = fmaf(r0 * u_s[d], k0, c);
+        }
+      }
+      if (lane < WK_COLS) vg[q * WK_COLS + lane] = lane < cols_here ? to_f(src[2 * D + lane]) : 0.f;
+      c = warp_sum(c);
+      if (lane == 0) cg[q] = c;
+    }
+    __syncthreads();                                       // the group is ready; the sums of the one before are out
+    const float* wg = w_s + (size_t)buf * WK_GROUP * Dp;
+#pragma unroll 4
+    for (int q = 0; q < gn; ++q) {
+      const float vj = vg[q * WK_COLS + col];
+      const float4* rr = reinterpret_cast<const float4*>(r_s + q * Dp + part * WK_ROWS);
+      const float4* kr = reinterpret_cast<const float4*>(k_s + q * Dp + part * WK_ROWS);
+      const float4* wr = reinterpret_cast<const float4*>(wg + q * Dp + part * WK_ROWS);
+      float o = 0.f, o2 = 0.f;
+#pragma unroll
+      for (int i = 0; i < WK_ROWS / 4; ++i) {
+        const float4 r4 = rr[i], k4 = kr[i], w4 = wr[i];
+        o = fmaf(s[4 * i + 0], r4.x, o);
+        o2 = fmaf(s[4 * i + 1], r4.y, o2);
+        o = fmaf(s[4 * i + 2], r4.z, o);
+        o2 = fmaf(s[4 * i + 3], r4.w, o2);
+        s[4 * i + 0] = fmaf(w4.x, s[4 * i + 0], k4.x * vj);
+        s[4 * i + 1] = fmaf(w4.y, s[4 * i + 1], k4.y * vj);
+        s[4 * i + 2] = fmaf(w4.z, s[4 * i + 2], k4.z * vj);
+        s[4 * i + 3] = fmaf(w4.w, s[4 * i + 3], k4.w * vj);
+      }
+      o_s[(q * parts + part) * WK_COLS + col] = o + o2;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < gn * WK_COLS; i += blockDim.x) {
+      const int q = i / WK_COLS, c = i % WK_COLS;
+      if (c >= cols_here) continue;
+      float o = cg[q] * vg[i];
+      for (int p = 0; p < parts; ++p) o += o_s[(q * parts + p) * WK_COLS + c];
+      out[(size_t)(t0 + g0 + q) * HV + h * V + blockIdx.x * WK_COLS + c] = o;
+    }
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int i = 0; i < WK_ROWS; ++i) {
+    const int d = part * WK_ROWS + i;
+    if (live && d < D) S[(size_t)d * V + j] = s[i];
+  }
+  // the request's last input, for its next token; every block of the request takes a share of the channels
+  float* prev = base + (size_t)H * D * V;
+  const T* last = h_in + (size_t)(t0 + n - 1) * hidden;
+  for (int c = (h * gridDim.x + blockIdx.x) * blockDim.x + threadIdx.x; c < hidden; c += H * gridDim.x * blockDim.x)
+    prev[c] = to_f(last[c]);
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// Single tokens (bfloat16): out[s, m, :] = W[s] mix_s(m) for the s < n stacked matrices [n, N, K], and z[m, :] = w1 mix_n(m) in
+// 32-bit.  A block takes 64 columns of one matrix: it puts the first weights of its 16 warps on their way (they are nobody's
+// output), then makes its mix of all rows in shared memory and multiplies on the tensor cores; two warps share 8 columns,
+// each half of k.  (The products' k index is a permutation of the real one, the same for both operands.)
+constexpr int PJ_WARPS = 16, PJ_COLS = 64, PJ_UNROLL = 8, PJ_PAD = 32;
+
+template <int ROWS>
+__global__ void __launch_bounds__(PJ_WARPS * 32)
+wkv_project_kernel(bf16* __restrict__ out, float* __restrict__ z, const bf16* __restrict__ h, const bf16* __restrict__ mu,
+                   const bf16* __restrict__ w, const bf16* __restrict__ w1, const float* __restrict__ state,
+                   size_t state_stride, size_t prev_off, const int* __restrict__ slots, int M, int n, int N, int R, int K) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) unsigned char pj_smem[];
+  bf16* x_s = reinterpret_cast<bf16*>(pj_smem);                       // [ROWS][K + PJ_PAD]
+  __shared__ float red[PJ_WARPS / 2][ROWS][8];
+  const int xs = K + PJ_PAD;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int g = lane >> 2, t = lane & 3;
+  const int per = (N + PJ_COLS - 1) / PJ_COLS;
+  const int s = min((int)blockIdx.x / per, n);                        // which mix; n: the decay's
+  const int n_cols = s < n ? N : R;
+  const int n0 = ((int)blockIdx.x - s * per) * PJ_COLS + (warp >> 1) * 8;
+  const bool n_ok = n0 + g < n_cols;
+  const bf16* mat = s < n ? w + (size_t)s * N * K : w1;
+  const int steps = (K + 31) / 32, half = (steps + 1) / 2;
+  const int st0 = (warp & 1) * half, st1 = min(st0 + half, steps);
+  const bf16* wrow = mat + (size_t)(n_ok ? n0 + g : 0) * K + t * 8;
+  uint4 wv[2][PJ_UNROLL];
+  auto fetch = [&](int st, int bf) {
+#pragma unroll
+    for (int q = 0; q < PJ_UNROLL; ++q) {
+      const int kk = (st + q) * 32;
+      wv[bf][q] = (n_ok && st + q < st1 && kk + t * 8 < K) ? __ldcs(reinterpret_cast<const uint4*>(wrow + kk)) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  fetch(st0, 0);
+  if constexpr (ROWS == 8) fetch(st0 + PJ_UNROLL, 1);
+  pdl_wait();
+  for (int i = threadIdx.x * 8; i < ROWS * K; i += PJ_WARPS * 32 * 8) {
+    const int m = i / K, c = i - m * K;
+    uint4 o = make_uint4(0u, 0u, 0u, 0u);
+    if (m < M) {
+      const uint4 hv = *reinterpret_cast<const uint4*>(h + (size_t)m * K + c);
+      const uint4 mv = *reinterpret_cast<const uint4*>(mu + (size_t)s * K + c);
+      const float4* pv = reinterpret_cast<const float4*>(state + (size_t)slots[m] * state_stride + prev_off + c);
+      const float4 p0 = pv[0], p1 = pv[1];
+      const float pe[8] = {p0.x, p0.y, p0.z, p0.w, p1.x, p1.y, p1.z, p1.w};
+      const bf16* he = reinterpret_cast<const bf16*>(&hv);
+      const bf16* me = reinterpret_cast<const bf16*>(&mv);
+      bf16* oe = reinterpret_cast<bf16*>(&o);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float x = to_f(he[j]);
+        oe[j] = from_f<bf16>(fmaf(pe[j] - x, to_f(me[j]), x));
+      }
+    }
+    *reinterpret_cast<uint4*>(x_s + m * xs + c) = o;
+  }
+  __syncthreads();
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  auto multiply = [&](int st, int bf) {
+#pragma unroll
+    for (int q = 0; q < PJ_UNROLL; ++q) {
+      const int kk = (st + q) * 32 + t * 8;
+      const bool ok = st + q < st1 && kk < K;
+      const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+      const uint4 xv = ok ? *reinterpret_cast<const uint4*>(x_s + g * xs + kk) : zero;
+      uint4 yv = zero;
+      if constexpr (ROWS == 16) yv = ok ? *reinterpret_cast<const uint4*>(x_s + (g + 8) * xs + kk) : zero;
+      const unsigned a1[4] = {xv.x, yv.x, xv.y, yv.y}, a2[4] = {xv.z, yv.z, xv.w, yv.w};
+      mma_bf16(acc, a1, wv[bf][q].x, wv[bf][q].y);
+      mma_bf16(acc, a2, wv[bf][q].z, wv[bf][q].w);
+    }
+  };
+  if constexpr (ROWS == 8) {
+    for (int st = st0; st < st1; st += 2 * PJ_UNROLL) {
+      multiply(st, 0);
+      if (st + 2 * PJ_UNROLL < st1) fetch(st + 2 * PJ_UNROLL, 0);
+      if (st + PJ_UNROLL < st1) multiply(st + PJ_UNROLL, 1);
+      if (st + 3 * PJ_UNROLL < st1) fetch(st + 3 * PJ_UNROLL, 1);
+    }
+  } else {
+    for (int st = st0; st < st1; st += 2 * PJ_UNROLL) {
+      if (st + PJ_UNROLL < st1) fetch(st + PJ_UNROLL, 1);
+      multiply(st, 0);
+      if (st + 2 * PJ_UNROLL < st1) fetch(st + 2 * PJ_UNROLL, 0);
+      if (st + PJ_UNROLL < st1) multiply(st + PJ_UNROLL, 1);
+    }
+  }
+  // (lane (g, t) holds rows g and g + 8 of columns 2 t and 2 t + 1)
+  if (warp & 1) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      red[warp >> 1][g][2 * t + e] = acc[e];
+      if constexpr (ROWS == 16) red[warp >> 1][g + 8][2 * t + e] = acc[2 + e];
+    }
+  }
+  __syncthreads();
+  if (warp & 1) return;
+#pragma unroll
+  for (int hh = 0; hh < ROWS / 8; ++hh)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int m = g + 8 * hh, c = n0 + 2 * t + e;
+      if (m >= M || c >= n_cols) continue;
+      const float val = acc[2 * hh + e] + red[warp >> 1][m][2 * t + e];
+      if (s < n) out[((size_t)s * M + m) * N + c] = from_f<bf16>(val);
+      else z[(size_t)m * R + c] = val;
+    }
+}
+
+// One block a (head, request), every token a request of its own: thread (part, col) holds ST_ROWS rows of state column col,
+// fetched before the wait for the predecessor (no kernel but this one writes the state in a step).
+constexpr int ST_ROWS = 16;
+
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS, THREADS == 256 ? 3 : 1)
+wkv_step_kernel(T* __restrict__ out, const T* __restrict__ rkvg, const float* __restrict__ z, const T* __restrict__ w2,
+                const float* __restrict__ w0, const float* __restrict__ u, const float* __restrict__ norm_w, float eps,
+                const T* __restrict__ h_in, float* __restrict__ state, size_t state_stride, const int* __restrict__ slots,
+                int M, int H, int D, int R, int hidden, int cols, int w2_in_smem) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float st_smem[];
+  __shared__ float scratch[32];
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int col = threadIdx.x % cols, part = threadIdx.x / cols, parts = blockDim.x / cols;
+  const int HD = H * D;
+  constexpr int PER = 16 / (int)sizeof(T);
+  T* w2_s = reinterpret_cast<T*>(st_smem);                 // [D][R] where w2_in_smem
+  float* z_s = st_smem + (w2_in_smem ? (D * R * (int)sizeof(T) + 15) / 16 * 4 : 0);   // [R], rounded up to 16 bytes
+  float* r_s = z_s + (R + 3) / 4 * 4;                      // [D] each
+  float* k_s = r_s + D;
+  float* w_s = k_s + D;
+  float* c_s = w_s + D;                                    // r u k
+  float* o_s = c_s + D;                                    // [parts][cols]
+  float* base = state + (size_t)slots[b] * state_stride;
+  float* S = base + (size_t)h * D * D;
+  const T* w2_h = w2 + (size_t)h * D * R;
+  if (w2_in_smem)
+    for (int i = threadIdx.x * PER; i < D * R; i += blockDim.x * PER) cp_async_16(w2_s + i, w2_h + i, true);
+  cp_async_commit();
+  float s[ST_ROWS];
+#pragma unroll
+  for (int i = 0; i < ST_ROWS; ++i) {
+    const int d = part * ST_ROWS + i;
+    s[i] = (col < D && d < D) ? S[(size_t)d * D + col] : 0.f;
+  }
+  const bool mine = threadIdx.x < D;                       // (the block has a thread for every channel)
+  const float u_d = mine ? u[h * D + threadIdx.x] : 0.f, n_d = mine ? norm_w[h * D + threadIdx.x] : 0.f;
+  if (mine) w_s[threadIdx.x] = w0[h * D + threadIdx.x];
+  pdl_wait();
+  const T* row = rkvg + (size_t)b * HD + h * D;            // (r, k, v, gate: one matrix of rows each)
+  const size_t plane = (size_t)M * HD;
+  float r_d = 0.f, k_d = 0.f, vj = 0.f, gate = 0.f;
+  if (mine) {
+    r_d = to_f(row[threadIdx.x]);
+    k_d = to_f(row[plane + threadIdx.x]);
+    gate = to_f(row[3 * plane + threadIdx.x]);
+  }
+  if (col < D) vj = to_f(row[2 * plane + col]);
+  for (int i = threadIdx.x; i < R; i += blockDim.x) z_s[i] = tanhf(z[(size_t)b * R + i]);
+  if (mine) {
+    r_s[threadIdx.x] = r_d;
+    k_s[threadIdx.x] = k_d;
+    c_s[threadIdx.x] = r_d * u_d * k_d;
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // the decays: eight lanes a channel; a warp's four channels lie inside or outside [0, D rounded up) together
+  for (int d0 = threadIdx.x >> 3; d0 < (D + 3) / 4 * 4; d0 += blockDim.x >> 3) {
+    const int sub = threadIdx.x & 7;
+    float a = 0.f;
+    if (d0 < D) {
+      if (w2_in_smem) {
+        for (int i = sub * PER; i < R; i += 8 * PER) {
+          const uint4 v = *reinterpret_cast<const uint4*>(w2_s + (size_t)d0 * R + i);
+          const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+          for (int j = 0; j < PER; ++j) a = fmaf(to_f(e[j]), z_s[i + j], a);
+        }
+      } else {
+        for (int i = sub; i < R; i += 8) a = fmaf(to_f(w2_h[(size_t)d0 * R + i]), z_s[i], a);
+      }
+    }
+    a += __shfl_xor_sync(0xffffffffu, a, 1);
+    a += __shfl_xor_sync(0xffffffffu, a, 2);
+    a += __shfl_xor_sync(0xffffffffu, a, 4);
+    if (sub == 0 && d0 < D) w_s[d0] = expf(-expf(a + w_s[d0]));
+  }
+  __syncthreads();
+  float o = 0.f;
+#pragma unroll
+  for (int i = 0; i < ST_ROWS; ++i) {
+    const int d = part * ST_ROWS + i;
+    if (d < D) {
+      o = fmaf(s[i], r_s[d], fmaf(c_s[d], vj, o));
+      s[i] = fmaf(w_s[d], s[i], k_s[d] * vj);
+      if (col < D) S[(size_t)d * D + col] = s[i];
+    }
+  }
+  o_s[part * cols + col] = o;
+  __syncthreads();
+  float total = 0.f;
+  if (mine)                                                // (column threadIdx.x, whose row part is the first)
+    for (int p = 0; p < parts; ++p) total += o_s[p * cols + threadIdx.x];
+  const float ss = block_sum(total * total, scratch);
+  if (mine) {
+    const float rstd = 1.f / sqrtf(ss / (float)D + eps);
+    out[(size_t)b * HD + h * D + threadIdx.x] = from_f<T>(total * rstd * n_d * silu_for<T>(gate));
+  }
+  float* prev = base + (size_t)H * D * D;
+  for (int c = h * blockDim.x + threadIdx.x; c < hidden; c += H * blockDim.x) prev[c] = to_f(h_in[(size_t)b * hidden + c]);
+}
+
+}  // namespace
+
+// out [n, T, hidden]; h [T, hidden]; mu [n, hidden] (all in `dtype`); state [slots, state_stride] 32-bit with the row before
+// the step's first token at prev_off.
+TS_API int ts_token_shift(void* out, const void* h, const void* mu, const float* state, long long state_stride,
+                          long long prev_off, const int* token_request, const int* q_start, const int* slots, int T, int hidden,
+                          int n, int dtype, void* stream) {
+  if (T <= 0 || n <= 0 || hidden <= 0) return 0;
+  if (n > SH_MAX) TS_REFUSE(TS_ERR_LIMIT, "ts_token_shift: %d mixes (limit %d)", n, SH_MAX);
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool vec = dtype == TS_BF16 && hidden % 8 == 0 && !(((uintptr_t)out | (uintptr_t)h | (uintptr_t)mu) & 15);
+  const bool few = T <= 256;
+  const dim3 grid(few ? T : ceil_div(T, 4), ceil_div(hidden, vec ? 1024 : 128));
+  if (grid.y > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_token_shift: rows of %d", hidden);
+#define TS_SHIFT(TT, PER, TOK)                                                                                            \
+  ts_launch(token_shift_kernel<TT, PER, TOK>, grid, dim3(128), 0, s, (TT*)out, (const TT*)h, (const TT*)mu, state, (size_t)state_stride, \
+            (size_t)prev_off, token_request, q_start, slots, T, hidden, n)
+  if (dtype == TS_F32) { if (few) TS_SHIFT(float, 1, 1); else TS_SHIFT(float, 1, 4); }
+  else if (dtype == TS_BF16) {
+    if (vec) { if (few) TS_SHIFT(bf16, 8, 1); else TS_SHIFT(bf16, 8, 4); }
+    else { if (few) TS_SHIFT(bf16, 1, 1); else TS_SHIFT(bf16, 1, 4); }
+  } else TS_REFUSE(TS_ERR_DTYPE, "ts_token_shift: dtype %d", dtype);
+#undef TS_SHIFT
+  TS_LAUNCH_CHECK();
+}
+
+// out [T, N] 32-bit; z [T, R] 32-bit; w2 [N, R] in `dtype`; w0 [N] 32-bit.
+TS_API int ts_wkv_decay(float* out, const float* z, const void* w2, const float* w0, int T, int N, int R, int dtype, void* stream) {
+  if (T <= 0 || N <= 0) return 0;
+  if (R <= 0) TS_REFUSE(TS_ERR_SHAPE, "ts_wkv_decay: a rank of %d", R);
+  const dim3 grid(ceil_div(N, DC_N), ceil_div(T, DC_M));
+  if (grid.y > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_decay: %d tokens", T);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == TS_F32) ts_launch(wkv_decay_kernel<float>, grid, dim3(256), 0, s, out, z, (const float*)w2, w0, T, N, R);
+  else if (dtype == TS_BF16) ts_launch(wkv_decay_kernel<bf16>, grid, dim3(256), 0, s, out, z, (const bf16*)w2, w0, T, N, R);
+  else TS_REFUSE(TS_ERR_DTYPE, "ts_wkv_decay: dtype %d", dtype);
+  TS_LAUNCH_CHECK();
+}
+
+// out [T, H V] 32-bit; r, k [T, H D] and v [T, H V] in `dtype`; w [T, H D] and u [H, D] 32-bit; h_in [T, hidden]: the mixer's
+// input; state [slots, state_stride]: [H D V | hidden].  longest: the most tokens a request brings (0: not known); long
+// portions are launched late (see ts_launch_late).
+constexpr int WK_LATE_TOKENS = 64;
+
+TS_API int ts_wkv_scan(float* out, const void* r, const void* k, const void* v, const float* w, const float* u, const void* h_in,
+                       float* state, long long state_stride, const int* q_start, const int* slots, int B, int H, int D, int V,
+                       int hidden, int longest, int dtype, void* stream) {
+  if (B <= 0) return 0;
+  if (H <= 0 || D <= 0 || V <= 0) TS_REFUSE(TS_ERR_SHAPE, "ts_wkv_scan: %d heads of %d x %d", H, D, V);
+  const int parts = ceil_div(ceil_div(D, WK_ROWS), 2) * 2;            // (whole warps)
+  if (parts * WK_COLS > 512) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_scan: keys of %d (limit %d)", D, 512 / WK_COLS * WK_ROWS);
+  if (B > 65535 || H > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_scan: %d requests / %d heads per launch", B, H);
+  cudaStream_t s = (cudaStream_t)stream;
+  const int elem = dtype == TS_F32 ? 4 : 2, per = 16 / elem;
+  const int fast = D % per == 0 && V % per == 0 && D % 4 == 0 &&
+                   !(((uintptr_t)r | (uintptr_t)k | (uintptr_t)v | (uintptr_t)w) & 15);
+  const int Dp = parts * WK_ROWS;
+  const size_t smem = sizeof(float) * ((size_t)4 * WK_GROUP * Dp + Dp + 2 * WK_GROUP * (WK_COLS + 1) + (size_t)WK_GROUP * parts * WK_COLS) +
+                      (size_t)2 * WK_GROUP * (2 * D + WK_COLS) * elem;
+  const dim3 grid(ceil_div(V, WK_COLS), H, B);
+#define TS_WK(TT)                                                                                                       \
+  do {                                                                                                                  \
+    static size_t configured = 0;                                                                                       \
+    if (smem > 48 * 1024 && smem > configured) {                                                                        \
+      cudaError_t e = cudaFuncSetAttribute(wkv_scan_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_scan: shared memory %zu: %s", smem, cudaGetErrorString(e));       \
+      configured = smem;                                                                                                \
+    }                                                                                                                   \
+    if (longest >= WK_LATE_TOKENS)                                                                                      \
+      ts_launch_late(wkv_scan_kernel<TT>, grid, dim3(parts * WK_COLS), smem, s, out, (const TT*)r, (const TT*)k, (const TT*)v, w, u, \
+                     (const TT*)h_in, state, (size_t)state_stride, q_start, slots, H, D, V, hidden, parts, fast);       \
+    else                                                                                                                \
+      ts_launch(wkv_scan_kernel<TT>, grid, dim3(parts * WK_COLS), smem, s, out, (const TT*)r, (const TT*)k, (const TT*)v, w, u, \
+                (const TT*)h_in, state, (size_t)state_stride, q_start, slots, H, D, V, hidden, parts, fast);            \
+  } while (0)
+  if (dtype == TS_F32) TS_WK(float);
+  else if (dtype == TS_BF16) TS_WK(bf16);
+  else TS_REFUSE(TS_ERR_DTYPE, "ts_wkv_scan: dtype %d", dtype);
+#undef TS_WK
+  TS_LAUNCH_CHECK();
+}
+
+// bfloat16; M <= 16 tokens, each a request of its own (that of slots[m]); h [M, K]; mu [n + 1, K] (the last row the decay's);
+// w [n, N, K]; w1 [R, K]; out [n, M, N]; z [M, R] 32-bit.
+TS_API int ts_wkv_project_supported(int M, int K, int dtype) { return dtype == TS_BF16 && M > 0 && M <= 16 && K % 8 == 0 && K <= 6144; }
+
+TS_API int ts_wkv_project(void* out, float* z, const void* h, const void* mu, const void* w, const void* w1, const float* state,
+                          long long state_stride, long long prev_off, const int* slots, int M, int n, int N, int R, int K,
+                          void* stream) {
+  if (M <= 0 || n <= 0 || N <= 0 || R <= 0) return 0;
+  if (!ts_wkv_project_supported(M, K, TS_BF16) || state_stride % 4 || prev_off % 4 ||
+      (((uintptr_t)h | (uintptr_t)mu | (uintptr_t)w | (uintptr_t)w1 | (uintptr_t)state) & 15))
+    TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_wkv_project: %d tokens, rows of %d", M, K);
+  const dim3 grid(n * ceil_div(N, PJ_COLS) + ceil_div(R, PJ_COLS));
+  cudaStream_t s = (cudaStream_t)stream;
+#define TS_PJ(ROWS)                                                                                                      \
+  do {                                                                                                                   \
+    const size_t smem = (size_t)ROWS * (K + PJ_PAD) * 2;                                                                      \
+    static size_t configured = 0;                                                                                        \
+    if (smem > 40 * 1024 && smem > configured) {                                                                         \
+      cudaError_t e = cudaFuncSetAttribute(wkv_project_kernel<ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_project: shared memory %zu: %s", smem, cudaGetErrorString(e));     \
+      configured = smem;                                                                                                 \
+    }                                                                                                                    \
+    ts_launch(wkv_project_kernel<ROWS>, grid, dim3(PJ_WARPS * 32), smem, s, (bf16*)out, z, (const bf16*)h, (const bf16*)mu, \
+              (const bf16*)w, (const bf16*)w1, state, (size_t)state_stride, (size_t)prev_off, slots, M, n, N, R, K);     \
+  } while (0)
+  if (M <= 8) TS_PJ(8);
+  else TS_PJ(16);
+#undef TS_PJ
+  TS_LAUNCH_CHECK();
+}
+
+// Heads whose state a block holds in registers: value columns rounded up to whole warps times row parts of 16.
+TS_API int ts_wkv_step_supported(int D, int V) {
+  return D > 0 && V == D && ceil_div(V, 32) * 32 * ceil_div(D, ST_ROWS) <= 1024;
+}
+
+// out [M, H V]; rkvg [4, M, H D] in `dtype`; z [M, R] 32-bit (before the tanh); w2 [H D, R] in `dtype`; w0 [H D], u [H, D] and
+// norm_w [H V] 32-bit; every token a request of its own (that of slots[m]).
+TS_API int ts_wkv_step(void* out, const void* rkvg, const float* z, const void* w2, const float* w0, const float* u,
+                       const float* norm_w, float eps, const void* h_in, float* state, long long state_stride, const int* slots,
+                       int M, int H, int D, int R, int hidden, int dtype, void* stream) {
+  if (M <= 0) return 0;
+  if (!ts_wkv_step_supported(D, D)) TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_wkv_step: heads of %d", D);
+  if (M > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_step: %d requests per launch", M);
+  const int cols = ceil_div(D, 32) * 32, parts = ceil_div(D, ST_ROWS), elem = dtype == TS_F32 ? 4 : 2;
+  // (R a multiple of what 16 bytes hold, so that a row's pieces start on 16-byte boundaries)
+  const int w2_in_smem = R % (16 / elem) == 0 && !((uintptr_t)w2 & 15) && D * R * elem <= 32 * 1024;
+  const size_t smem = (w2_in_smem ? ((size_t)D * R * elem + 15) / 16 * 16 : 0) +
+                      sizeof(float) * ((size_t)4 * D + (R + 3) / 4 * 4 + cols * parts);
+  if (smem > 47 * 1024) TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_wkv_step: a rank of %d", R);
+  cudaStream_t s = (cudaStream_t)stream;
+#define TS_ST(TT, TH)                                                                                                      \
+  ts_launch(wkv_step_kernel<TT, TH>, dim3(H, M), dim3(cols * parts), smem, s, (TT*)out, (const TT*)rkvg, z, (const TT*)w2, w0, u, \
+            norm_w, eps, (const TT*)h_in, state, (size_t)state_stride, slots, M, H, D, R, hidden, cols, w2_in_smem)
+  if (dtype == TS_F32) { if (cols * parts <= 256) TS_ST(float, 256); else TS_ST(float, 1024); }
+  else if (dtype == TS_BF16) { if (cols * parts <= 256) TS_ST(bf16, 256); else TS_ST(bf16, 1024); }
+  else TS_REFUSE(TS_ERR_DTYPE, "ts_wkv_step: dtype %d", dtype);
+#undef TS_ST
+  TS_LAUNCH_CHECK();
+}

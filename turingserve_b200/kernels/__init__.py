@@ -68,7 +68,7 @@ class LazyProduct:
 class CudaOps:
     """ctypes front of ``libturingserve_b200.so``."""
 
-    ABI = 15
+    ABI = 16
     UNSUPPORTED = -4            # a kernel's refusal of a shape or layout another kernel takes
 
     def __init__(self, lib_path: str) -> None:
@@ -77,7 +77,7 @@ class CudaOps:
         self.lib.ts_last_error.restype = ctypes.c_char_p
         if self.lib.ts_abi_version() != self.ABI:
             raise KernelError(f"{lib_path} has ABI {self.lib.ts_abi_version()}, this package needs {self.ABI}")
-        P, I, F = c_void_p, c_int, c_float
+        P, I, F, L = c_void_p, c_int, c_float, ctypes.c_longlong
         sigs = {
             "ts_embedding": [P, P, P, I, I, I, I, P],
             "ts_gather_rows": [P, P, P, I, I, I, P],
@@ -116,10 +116,10 @@ class CudaOps:
             "ts_kv_write_pair": [P, I, I, I, P, P, P, I, I, I, I, I, I, P],
             "ts_attention_diff": [P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, F, F, I, P],
             "ts_attention_diff_mma": [P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, F, F, P, P, I, I, P],
-            "ts_router_topk": [P, P, P, P, I, I, I, I, I, I, I, P, P],
+            "ts_router_topk": [P, P, P, P, I, I, I, I, I, I, I, P, I, I, F, P, P],
             "ts_moe_align": [P, I, I, P, P, P, P, I, P, I, I, P],
             "ts_grouped_linear": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
-            "ts_moe_combine": [P, P, P, P, I, I, I, I, P, P, P, P],
+            "ts_moe_combine": [P, P, P, P, I, I, I, I, P, P, P, P, P],
             "ts_hyper_norm": [P, P, P, P, I, P, P, P, P, P, F, I, I, I, I, F, I, P],
             "ts_ssm_prepare": [P, P, I, I, I, P, P, P, P, P, ctypes.c_longlong, ctypes.c_longlong, P, P, P, I, I, I, I, I, P],
             "ts_ssm_scan": [P, P, P, I, I, P, ctypes.c_longlong, P, P, P, I, I, I, I, I, I, I, I, P],
@@ -131,15 +131,23 @@ class CudaOps:
             "ts_moe_gather": [P, P, P, P, I, I, I, I, P],
             "ts_delta_prepare": [P, P, I, P, P, P, P, ctypes.c_longlong, P, P, P, I, I, I, I, I, I, F, I, P],
             "ts_delta_scan": [P, P, P, I, P, ctypes.c_longlong, P, P, I, I, I, I, I, I, I, I, P],
-            "ts_head_gated_rmsnorm": [P, P, P, I, P, F, I, I, I, I, P],
+            "ts_head_gated_rmsnorm": [P, P, P, I, P, I, F, I, I, I, I, P],
             "ts_attention_biased": [P, I, I, P, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, I, I, P, P, I, I, P, I, P, P, I, P],
             "ts_attention_biased_mma": [P, I, I, P, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P, I, I, P, P, I, I, P, I, P, P, I, P],
             "ts_rope_headnorm_write": [P, I, I, I, P, P, I, I, F, P, P, P, I, I, I, I, I, I, I, P, I, P],
             "ts_rope_headnorm_write_supports_parts": [I, I, I, I],
             "ts_rms_rows": [P, P, I, I, I, P, F, I, I, P],
             "ts_qk_rownorm_write": [P, I, P, P, F, P, F, I, P, P, P, I, I, I, I, I, I, P],
-            "ts_latent_kv_write": [P, I, I, P, F, P, P, F, I, P, P, I, I, I, I, I, P],
-            "ts_rotate_pairs": [P, I, I, P, I, I, P, P, F, I, I, I, I, I, P],
+            "ts_latent_kv_write": [P, I, I, P, F, P, P, F, I, I, P, P, I, I, I, I, P, P, I, P, I, I, I, I, P],
+            "ts_rotate_pairs": [P, I, I, P, I, I, P, P, F, I, I, I, I, I, I, P],
+            "ts_latent_queries": [P, I, I, P, P, I, P, P, P, F, I, I, I, I, I, I, I, I, P],
+            "ts_token_shift": [P, P, P, P, L, L, P, P, P, I, I, I, I, P],
+            "ts_wkv_decay": [P, P, P, P, I, I, I, I, P],
+            "ts_wkv_scan": [P, P, P, P, P, P, P, P, L, P, P, I, I, I, I, I, I, I, P],
+            "ts_wkv_project": [P, P, P, P, P, P, P, L, L, P, I, I, I, I, I, P],
+            "ts_wkv_project_supported": [I, I, I],
+            "ts_wkv_step": [P, P, P, P, P, P, P, F, P, P, L, P, I, I, I, I, I, I, P],
+            "ts_wkv_step_supported": [I, I],
             "ts_grouped_glu": [P, P, P, P, P, P, P, I, I, I, I, I, F, F, F, I, I, P],
             "ts_glu_pairs": [P, P, P, I, I, I, F, F, F, I, P],
             "ts_post_norm": [P, P, P, P, P, I, P, P, P, P, I, F, P, F, P, F, I, I, I, P],
@@ -706,12 +714,12 @@ class CudaOps:
                                            int(getattr(step, "max_q_len", 0) or 0), _code(proj.dtype), self._stream()), "delta_scan")
 
     def head_gated_rmsnorm(self, out, x, gate, weight, eps: float, H: int, V: int) -> None:
-        """out [T, HV] = x / rms over each head's V * weight[V] * silu(gate); x float32; ``gate`` possibly a column
-        slice of a wider tensor."""
+        """out [T, HV] = x / rms over each head's V * weight * silu(gate); x float32; ``weight`` [V], common to the heads, or
+        [H V]; ``gate`` possibly a column slice of a wider tensor."""
         if gate.stride(1) != 1:
             raise ValueError("head_gated_rmsnorm: the gate's rows must be contiguous")
-        self._check(self.lib.ts_head_gated_rmsnorm(_ptr(out), _ptr(x), _ptr(gate), gate.stride(0), _ptr(weight), float(eps),
-                                                   x.shape[0], H, V, _code(out.dtype), self._stream()), "head_gated_rmsnorm")
+        self._check(self.lib.ts_head_gated_rmsnorm(_ptr(out), _ptr(x), _ptr(gate), gate.stride(0), _ptr(weight),
+                                                   V if weight.numel() == H * V and H > 1 else 0, float(eps), x.shape[0], H, V, _code(out.dtype), self._stream()), "head_gated_rmsnorm")
 
     # -- norms, rotations and per-head products around an attention ----------------------------------------------------
     def rms_rows(self, out, x, col0: int, weight, eps: float) -> None:
@@ -730,24 +738,59 @@ class CudaOps:
                                                  proj.shape[0], H, G, D, page_size, _code(proj.dtype), self._stream()),
                     "qk_rownorm_write")
 
-    def latent_kv_write(self, proj, col0: int, weight, eps: float, positions, freq, magnitude: float, rot_dims: int, k_cache,
-                        slots, rank: int, R: int, page_size: int) -> None:
-        """The cached row of every token, [rms(latent) * weight | rotated key part], from the columns col0 .. of
-        ``proj`` into ``k_cache`` [pages, 1, page, rank + R] at ``slots``."""
-        self._check(self.lib.ts_latent_kv_write(_ptr(proj), proj.stride(0), col0, _ptr(weight), float(eps), _ptr(positions),
-                                                _ptr(freq), float(magnitude), rot_dims, _ptr(k_cache), _ptr(slots),
-                                                proj.shape[0], rank, R, page_size, _code(proj.dtype), self._stream()),
-                    "latent_kv_write")
+    PAIRINGS = {"neighbours": 0, "halves": 1}
 
-    def rotate_pairs(self, dst, src, positions, freq, magnitude: float, rot_dims: int) -> None:
-        """dst[t, h, :] = src[t, h, :] with its first ``rot_dims`` dimensions rotated in neighbouring pairs by
-        position * freq[i] (cosine and sine times ``magnitude``); [T, H, R] views with unit last stride."""
+    def latent_kv_write(self, proj, col0: int, weight, eps: float, positions, freq, magnitude: float, rot_dims: int, k_cache,
+                        slots, rank: int, R: int, page_size: int, pairing: str = "neighbours", cq=None, q_weight=None,
+                        keep: tuple[int, int] = (0, 0)):
+        """The cached row of every token, [rms(latent) * weight | rotated key part], from the columns col0 .. of
+        ``proj`` into ``k_cache`` [pages, 1, page, rank + R] at ``slots`` (None: nothing is cached).  ``cq`` [T, q_rank]: receives
+        rms(columns 0 .. q_rank) * q_weight.  ``proj`` may be a product put off: its partial sums are summed on the way and
+        only the columns ``keep`` (first, count) are left finished in the returned tensor."""
+        proj = self._settle(proj)
+        part, splits = None, 0
+        if isinstance(proj, Deferred):
+            if proj.bias is None:
+                part, splits, proj = proj.part, proj.splits, proj.out
+            else:
+                proj = self.materialize(proj)
+        self._check(self.lib.ts_latent_kv_write(
+            _ptr(proj), proj.stride(0), col0, _ptr(weight), float(eps), _ptr(positions), _ptr(freq), float(magnitude), rot_dims,
+            self.PAIRINGS[pairing], _ptr(k_cache), _ptr(slots), proj.shape[0], rank, R, page_size, _ptr(cq), _ptr(q_weight),
+            0 if cq is None else cq.shape[1], _ptr(part), splits, int(keep[0]), int(keep[1]), _code(proj.dtype), self._stream()),
+            "latent_kv_write")
+        return proj
+
+    def latent_queries(self, qa, q, w, positions, freq, magnitude: float, rot_dims: int, pairing: str) -> None:
+        """qa [T, H, N + R] = [w[h] q_plain | rotated part] of the queries ``q`` [T, H (K + R)] (``w`` [H, N, K]).  ``q`` may be a
+        product put off.  Up to 16 bfloat16 rows: one kernel; else the product per head and the rotation."""
+        H, N, K = w.shape
+        T, R = qa.shape[0], qa.shape[2] - N
+        q = self._settle(q)
+        part, splits, src = None, 0, q
+        if isinstance(q, Deferred):
+            part, splits, src = (q.part, q.splits, q.out) if q.bias is None else (None, 0, self.materialize(q))
+        if T <= 16 and src.dtype == torch.bfloat16:
+            rc = self.lib.ts_latent_queries(_ptr(qa), qa.stride(0), qa.stride(1), _ptr(src), _ptr(part), splits, _ptr(w),
+                                            _ptr(positions), _ptr(freq), float(magnitude), rot_dims, self.PAIRINGS[pairing], T, H,
+                                            N, K, R, _code(src.dtype), self._stream())
+            if rc != self.UNSUPPORTED:
+                self._check(rc, "latent_queries")
+                return
+        heads = self.materialize(q).view(T, H, K + R)
+        self.batched_linear(qa[:, :, :N], heads[:, :, :K], w)
+        self.rotate_pairs(qa[:, :, N:], heads[:, :, K:], positions, freq, magnitude, rot_dims, pairing)
+
+    def rotate_pairs(self, dst, src, positions, freq, magnitude: float, rot_dims: int, pairing: str = "neighbours") -> None:
+        """dst[t, h, :] = src[t, h, :] with its first ``rot_dims`` dimensions rotated in pairs, neighbours (2i, 2i + 1) or
+        halves (i, i + rot_dims / 2), by position * freq[i] (cosine and sine times ``magnitude``); [T, H, R] views with unit
+        last stride."""
         T, H, R = src.shape
         if dst.stride(2) != 1 or src.stride(2) != 1:
             raise ValueError("rotate_pairs: rows must be contiguous")
         self._check(self.lib.ts_rotate_pairs(_ptr(dst), dst.stride(0), dst.stride(1), _ptr(src), src.stride(0), src.stride(1),
-                                             _ptr(positions), _ptr(freq), float(magnitude), rot_dims, T, H, R,
-                                             _code(src.dtype), self._stream()), "rotate_pairs")
+                                             _ptr(positions), _ptr(freq), float(magnitude), rot_dims,
+                                             self.PAIRINGS[pairing], T, H, R, _code(src.dtype), self._stream()), "rotate_pairs")
 
     def rope_headnorm_write(self, proj, k_off: int, v_off: int, positions, freq, rot_dims: int, norm_eps, k_cache, v_cache,
                             slots, H: int, G: int, D: int, V: int, page_size: int):
@@ -778,8 +821,8 @@ class CudaOps:
 
     def batched_linear(self, out, x, w) -> None:
         """out[t, h, :] = w[h] x[t, h, :]: ``x`` [T, H, K] and ``out`` [T, H, N] views with unit last stride,
-        ``w`` [H, N, K] contiguous.  This library's kernels (up to 16 rows: a warp an output column, streaming
-        its weight row; float32 above: FFMA tiles, fixed k order); bfloat16 with more rows: the vendor's batched product."""
+        ``w`` [H, N, K] contiguous.  This library's kernels (up to 16 rows: tensor cores in bfloat16, a warp an
+        output column in float32; float32 above: FFMA tiles, fixed k order); bfloat16 with more rows: the vendor's batched product."""
         T, H, K = x.shape
         N = w.shape[1]
         if out.stride(2) != 1 or x.stride(2) != 1 or not w.is_contiguous():
@@ -961,15 +1004,19 @@ class CudaOps:
                     "rope_pairs_write")
 
     # -- routed feed-forward ---------------------------------------------------------------------------------
-    def router_topk(self, idx, weights, x, w_router, softmax: bool, renormalize: bool, correction=None) -> None:
+    def router_topk(self, idx, weights, x, w_router, softmax: bool, renormalize: bool, correction=None, groups: int = 1,
+                    keep: int = 1, scale: float = 1.0, share=None) -> None:
         """idx (int32 [T, top]), weights (float32 [T, top]): the ``top`` experts with the largest router
-        logits w_router (float32 [E, K]) . x, and their scores (sigmoid, or softmax over all experts).  With
-        ``correction`` (float32 [E]) the choice goes by score + correction; the weights stay the scores."""
+        logits w_router (float32 [E, K]) . x, and their scores (sigmoid, or softmax over all experts) times ``scale``.  With
+        ``correction`` (float32 [E]) the choice goes by score + correction; the weights stay the scores.  ``groups`` > 1: only
+        the experts of the ``keep`` groups of neighbours whose two largest choice scores have the largest sums may be chosen.
+        ``share`` (float32 [T]): ``w_router`` has one more row, and the sigmoid of its logit goes there."""
         T, top = idx.shape
         E, K = w_router.shape
+        E -= 0 if share is None else 1
         self._check(self.lib.ts_router_topk(_ptr(idx), _ptr(weights), _ptr(x), _ptr(w_router), T, E, K, top,
                                             1 if softmax else 0, 1 if renormalize else 0, _code(x.dtype), _ptr(correction),
-                                            self._stream()), "router_topk")
+                                            int(groups), int(keep), float(scale), _ptr(share), self._stream()), "router_topk")
 
     def moe_align(self, idx, E: int, with_tiles: int | None = None, table=None):
         """Sorts the (token, choice) pairs of ``idx`` by expert on the device; with ``table`` (int32 [rows, top]) ``idx`` holds
@@ -1113,6 +1160,58 @@ class CudaOps:
         self._check(rc, "rglru_step")
         return True
 
+    # -- the time mixer with a state that fades channel by channel ---------------------------------------------------
+    def token_shift(self, out, h, mu, state, prev_off: int, step) -> None:
+        """out[i, t] = h[t] + (h[t - 1] - h[t]) * mu[i] (``out`` [n, T, hidden], ``mu`` [n, hidden] in h's type); the row before
+        a request's first token of the step comes from its state slot, from ``prev_off`` on."""
+        n, T, hidden = out.shape
+        self._check(self.lib.ts_token_shift(_ptr(out), _ptr(h), _ptr(mu), _ptr(state), state.stride(0), int(prev_off),
+                                            _ptr(step.token_request), _ptr(step.q_start), _ptr(step.state_slots), T, hidden, n,
+                                            _code(h.dtype), self._stream()), "token_shift")
+
+    def wkv_decay(self, out, z, w2, w0) -> None:
+        """out (float32 [T, N]) = exp(-exp(w2 tanh(z) + w0)); z float32 [T, R], ``w2`` [N, R], ``w0`` float32 [N]."""
+        T, N = out.shape
+        self._check(self.lib.ts_wkv_decay(_ptr(out), _ptr(z), _ptr(w2), _ptr(w0), T, N, w2.shape[1], _code(w2.dtype),
+                                          self._stream()), "wkv_decay")
+
+    def wkv_scan(self, out, r, k, v, w, u, h, state, step, H: int, D: int) -> None:
+        """out (float32 [T, H D]): per head o = (S + diag(u) k v^T)^T r, then S <- diag(w) S + k v^T; r, k, v [T, H D], w float32
+        [T, H D], u float32 [H, D]; ``state`` (float32 [slots, H D D + hidden]) is read and left updated at each request's
+        slot, the request's last input (from ``h`` [T, hidden]) included."""
+        self._check(self.lib.ts_wkv_scan(_ptr(out), _ptr(r), _ptr(k), _ptr(v), _ptr(w), _ptr(u), _ptr(h), _ptr(state),
+                                         state.stride(0), _ptr(step.q_start), _ptr(step.state_slots), step.num_requests, H, D, D,
+                                         h.shape[1], int(getattr(step, "max_q_len", 0) or 0), _code(r.dtype), self._stream()),
+                    "wkv_scan")
+
+    def wkv_project(self, out, z, h, mu, w, w1, state, prev_off: int, step) -> bool:
+        """A step in which every token is a request of its own: out[i] = w[i] mix_i (``out`` [n, T, N], ``w`` [n, N, K]) and z
+        (float32 [T, R]) = w1 mix_n, the mixes as ``token_shift`` makes them.  False where the kernel does not take the step."""
+        n, T, N = out.shape
+        if (step.max_q_len != 1 or step.num_requests != T
+                or not self.lib.ts_wkv_project_supported(T, h.shape[1], _code(h.dtype))):
+            return False
+        rc = self.lib.ts_wkv_project(_ptr(out), _ptr(z), _ptr(h), _ptr(mu), _ptr(w), _ptr(w1), _ptr(state), state.stride(0),
+                                     int(prev_off), _ptr(step.state_slots), T, n, N, w1.shape[0], h.shape[1], self._stream())
+        if rc == self.UNSUPPORTED:
+            return False
+        self._check(rc, "wkv_project")
+        return True
+
+    def wkv_step(self, out, rkvg, z, w2, w0, u, norm_w, eps: float, h, state, step, H: int, D: int) -> bool:
+        """A step in which every token is a request of its own: decay, recurrence, the heads' norm (times ``norm_w`` [H D]) and
+        the gate silu(rkvg[3]) in one kernel; ``out`` [T, H D], ``rkvg`` [4, T, H D].  False where the kernel does not take it."""
+        T = out.shape[0]
+        if step.max_q_len != 1 or step.num_requests != T or not self.lib.ts_wkv_step_supported(D, D):
+            return False
+        rc = self.lib.ts_wkv_step(_ptr(out), _ptr(rkvg), _ptr(z), _ptr(w2), _ptr(w0), _ptr(u), _ptr(norm_w), float(eps), _ptr(h),
+                                  _ptr(state), state.stride(0), _ptr(step.state_slots), T, H, D, w2.shape[1], h.shape[1],
+                                  _code(out.dtype), self._stream())
+        if rc == self.UNSUPPORTED:
+            return False
+        self._check(rc, "wkv_step")
+        return True
+
     def moe_gather(self, xs, x, order, row_scale, top: int) -> None:
         """xs[i] = x[order[i] // top] (times row_scale[order[i]], rounded to x's type): the experts' input rows
         in sorted order."""
@@ -1120,14 +1219,16 @@ class CudaOps:
         self._check(self.lib.ts_moe_gather(_ptr(xs), _ptr(x), _ptr(order), _ptr(row_scale), P, top, K, _code(x.dtype),
                                            self._stream()), "moe_gather")
 
-    def moe_combine(self, out, y, place, pair_weights, top: int, x=None, pass_from=None, add=None) -> None:
+    def moe_combine(self, out, y, place, pair_weights, top: int, x=None, pass_from=None, add=None,
+                    share=None) -> None:
         """out[t] = sum over a token's choices r of (pair_weights[t, r] *) y[place[t top + r]] (y float32).  With ``x``
         ([T, N], out's type) and ``pass_from`` (one int32 on the device): a pair sorted to that place or a later
         one adds x[t] instead of a row of y (experts that return their input).  ``add`` ([T, N], out's type): added
-        to every token's sum (the output of an expert that every token uses)."""
+        to every token's sum (the output of an expert that every token uses), times ``share`` (float32 [T]) where given."""
         T, N = out.shape
         self._check(self.lib.ts_moe_combine(_ptr(out), _ptr(y), _ptr(place), _ptr(pair_weights), T, top, N,
-                                            _code(out.dtype), _ptr(x), _ptr(pass_from), _ptr(add), self._stream()),
+                                            _code(out.dtype), _ptr(x), _ptr(pass_from), _ptr(add), _ptr(share),
+                                            self._stream()),
                     "moe_combine")
 
     PAIR_PLAIN, PAIR_GATED = 0, 1

@@ -16,15 +16,12 @@ after the model's norm, times ``logit_scale``.  Every size and constant comes fr
 
 from __future__ import annotations
 
-import torch
-
 from turingserve_b200.config.model_config import (
     BandScaledRotarySpec, GatedMLPSpec, HyperRMSNormSpec, LayerRun, LayerSpec, LightningSpec, Mamba2Spec, ModelConfig,
     PairedMixerSpec, RoutedMLPSpec, SinkAttentionSpec, StreamLinkSpec)
 from turingserve_b200.config.registry import (
     Architecture, LayerTensorNames, TensorNames, register_architecture)
-from turingserve_b200.parts.base import BranchSum
-from turingserve_b200.parts.model import DecoderModel
+from turingserve_b200.parts.model import HyperStreamModel
 
 NAME = "Gugezen"
 # the rotation's angles are computed from the position itself: nothing in the design bounds a sequence
@@ -211,27 +208,4 @@ def make_config(*, width: int, vocab: int, layers: list[dict], eps: float = 1e-6
     return parse_config(c)
 
 
-class GugezenModel(DecoderModel):
-    """The decoder with what this family adds around the layers: the embedding rows, times a constant, start every copy
-    of the 32-bit stream (inside the first layer's norm kernel); the model's last norm reads the sum of the copies; the
-    logits are multiplied by a constant (folded into the last norm's 32-bit weight when it is loaded: the head has no
-    bias)."""
-
-    def __init__(self, cfg: ModelConfig, dtype: torch.dtype, device, max_positions: int) -> None:
-        super().__init__(cfg, dtype, device, max_positions)
-        self.embedding_scale = float(cfg.extra("embedding_scale", 1.0))
-        self.logit_scale = float(cfg.extra("logit_scale", 1.0))
-
-    def embed(self, step):
-        return BranchSum(super().embed(step), None, self.embedding_scale)
-
-    def finish(self, h, residual):
-        return self.final_norm.forward(h, residual, None)
-
-    def load(self, names, tensors) -> None:
-        super().load(names, tensors)
-        if self.logit_scale != 1.0:
-            self.final_norm.weight = (self.final_norm.weight * self.logit_scale).contiguous()
-
-
-register_architecture(Architecture(NAME, parse_config, tensor_names, to_config_json, build_model=GugezenModel))
+register_architecture(Architecture(NAME, parse_config, tensor_names, to_config_json, build_model=HyperStreamModel))

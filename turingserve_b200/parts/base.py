@@ -36,15 +36,26 @@ class ParamSpec:
     ``compute_dtype`` True: converted to the engine's dtype (operands of matrix products,
     embeddings).  False: a tensor stored in 32 bits stays in 32 bits, anything else is converted.
     ``integer`` True: an integer table, kept as int32.
+    A dimension None is whatever the checkpoint has (the part reads it from the tensor it gets); the random-weights mode
+    makes it ``free`` long.
     """
 
-    shape: tuple[int, ...]
+    shape: tuple[int | None, ...]
     compute_dtype: bool = True
     integer: bool = False
     # how the random-weights mode fills it: "normal" | "ones" | "zeros" | "identity"; an integer table: "zeros", or
     # "distinct": every row so many different numbers below ``high``
     init: str = "normal"
     high: int = 0
+    free: int = 0
+
+    def fits(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(n is None or n == got for n, got in zip(self.shape, shape))
+
+    @property
+    def sizes(self) -> tuple[int, ...]:
+        """The shape the random-weights mode gives it."""
+        return tuple(self.free if n is None else n for n in self.shape)
 
 
 @dataclass(frozen=True)
@@ -221,7 +232,7 @@ def _load_builtin() -> None:
         _loaded = True
         from turingserve_b200.parts import (  # noqa: F401
             attention, block, capped_attention, delta_rule, diff_attention, gated_mlp, latent_attention, lightning, mamba2,
-            mlp, normed_attention, paired_mixer, rglru, rmsnorm, rotary, routed_mlp, sink_attention, stream_link)
+            mlp, normed_attention, paired_mixer, rglru, rmsnorm, rotary, routed_mlp, sink_attention, stream_link, wkv)
 
 
 def build_block(layer_spec: Any, ctx: BuildContext):

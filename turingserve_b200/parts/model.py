@@ -11,7 +11,7 @@ import torch
 from turingserve_b200 import kernels
 from turingserve_b200.config.model_config import ModelConfig
 from turingserve_b200.config.registry import TensorNames
-from turingserve_b200.parts.base import BuildContext, ParamSpec, build, build_block
+from turingserve_b200.parts.base import BranchSum, BuildContext, ParamSpec, build, build_block
 
 
 class DecoderModel:
@@ -113,3 +113,26 @@ class DecoderModel:
         """What happens to the head's output before anyone sees it (nothing here; a cap or a scale in
         a model class that overrides this)."""
         return logits
+
+
+class HyperStreamModel(DecoderModel):
+    """The decoder over a residual stream in copies: the embedding rows, times a constant, start every copy of the 32-bit
+    stream (inside the first layer's norm kernel); the model's last norm reads the sum of the copies; the logits are multiplied
+    by a constant (folded into the last norm's 32-bit weight when it is loaded: the head has no bias).  Both constants are
+    ``ModelConfig.extras`` (``embedding_scale``, ``logit_scale``)."""
+
+    def __init__(self, cfg: ModelConfig, dtype: torch.dtype, device, max_positions: int) -> None:
+        super().__init__(cfg, dtype, device, max_positions)
+        self.embedding_scale = float(cfg.extra("embedding_scale", 1.0))
+        self.logit_scale = float(cfg.extra("logit_scale", 1.0))
+
+    def embed(self, step):
+        return BranchSum(super().embed(step), None, self.embedding_scale)
+
+    def finish(self, h, residual):
+        return self.final_norm.forward(h, residual, None)
+
+    def load(self, names: TensorNames, tensors: dict[str, torch.Tensor]) -> None:
+        super().load(names, tensors)
+        if self.logit_scale != 1.0:
+            self.final_norm.weight = (self.final_norm.weight * self.logit_scale).contiguous()

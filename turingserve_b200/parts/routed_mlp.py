@@ -5,7 +5,10 @@ more outputs than there are experts with tensors: the outputs behind them are ex
 which cost no product (their pairs are sorted behind the others and the sum takes the token's own row for them).
 
 A shared expert (``shared_intermediate_size``: one more feed-forward of the experts' form under 'shared.') runs for every
-token and is added, unweighted, in the kernel that sums a token's choices.
+token and is added in the kernel that sums a token's choices, unweighted or (``shared_gate``) times sigmoid(W_sg x), one number
+a token, which the router's kernel works out beside its scores.
+With ``groups`` the experts fall into equal groups of neighbours, and only those of the ``groups_kept`` groups whose two largest
+choice scores have the largest sums may be chosen.  ``weight_scale`` multiplies the weights.
 
 Router logits and scores are 32-bit.  The (token, choice) pairs are sorted by expert on the device and the
 two products run over the sorted groups; the chosen score multiplies the expert's input (``weight_on``
@@ -68,12 +71,21 @@ class RoutedMLP(FeedForward):
             raise ValueError(f"routed_mlp: top {self.top} of {self.outputs} router outputs")
         shared = getattr(spec, "shared_intermediate_size", None)
         self.shared_inter = int(shared) if shared else 0
+        self.groups, self.groups_kept = int(getattr(spec, "groups", 1)), int(getattr(spec, "groups_kept", 1))
+        self.weight_scale, self.has_share = float(getattr(spec, "weight_scale", 1.0)), bool(getattr(spec, "shared_gate", False))
+        if self.groups < 1 or self.outputs % self.groups or not 1 <= self.groups_kept <= self.groups:
+            raise ValueError(f"routed_mlp: {self.groups_kept} of {self.groups} groups of {self.outputs} experts")
+        if self.top > self.outputs // self.groups * self.groups_kept:
+            raise ValueError(f"routed_mlp: top {self.top} of {self.groups_kept} groups of {self.outputs // self.groups} experts")
+        if self.has_share and not self.shared_inter:
+            raise ValueError("routed_mlp: a shared expert's gate without a shared expert")
         rows = getattr(spec, "table_rows", None)
         self.table_rows = int(rows) if rows else 0
         self.wants_step = self.table_rows > 0
-        if self.table_rows and (self.has_correction or self.identity or self.on_input or self.E == 0):
-            raise ValueError("routed_mlp: a table of experts comes without router, correction and identity outputs, its "
-                             "weights on the output")
+        if self.table_rows and (self.has_correction or self.identity or self.on_input or self.E == 0 or self.groups > 1
+                                or self.has_share or self.weight_scale != 1.0):
+            raise ValueError("routed_mlp: a table of experts comes without router, correction, groups, shared gate and identity "
+                             "outputs, its weights on the output")
         if self.glu:
             self.glu_args = (float(spec.glu_limit), float(spec.glu_slope), float(spec.glu_offset))
             self.shared_glu_args = (float(spec.shared_glu_limit), float(spec.glu_slope), float(spec.glu_offset))
@@ -97,6 +109,8 @@ class RoutedMLP(FeedForward):
                 p["shared.gate"] = ParamSpec((self.shared_inter, self.hidden))
             p["shared.up"] = ParamSpec((self.shared_inter, self.hidden))
             p["shared.down"] = ParamSpec((self.hidden, self.shared_inter))
+            if self.has_share:
+                p["shared.sg"] = ParamSpec((1, self.hidden), compute_dtype=False)
         return p
 
     def load(self, t: dict[str, torch.Tensor]) -> None:
@@ -107,7 +121,9 @@ class RoutedMLP(FeedForward):
             if lo < 0 or hi >= self.E:
                 raise ValueError(f"routed_mlp: the table names experts {lo} to {hi} of {self.E}")
         else:
-            self.w_router = t["router"].float().contiguous()
+            # (the shared expert's gate is one more row of the router)
+            rows = [t["router"].float()] + ([t["shared.sg"].float()] if self.has_share else [])
+            self.w_router = torch.cat(rows, dim=0).contiguous()
         if self.has_correction:
             self.correction = t["correction"].float().contiguous()
         if self.shared_inter:
@@ -140,7 +156,9 @@ class RoutedMLP(FeedForward):
         T, top = x.shape[0], self.top
         idx = torch.empty((T, top), dtype=torch.int32, device=x.device)
         weights = torch.empty((T, top), dtype=torch.float32, device=x.device)
-        ops.router_topk(idx, weights, x, self.w_router, self.softmax, self.renormalize, self.correction)
+        share = torch.empty((T,), dtype=torch.float32, device=x.device) if self.has_share else None
+        ops.router_topk(idx, weights, x, self.w_router, self.softmax, self.renormalize, self.correction, self.groups,
+                        self.groups_kept, self.weight_scale, share)
         out = torch.empty((T, self.hidden), dtype=x.dtype, device=x.device)
         if self.identity:
             # the pairs of the experts with tensors are sorted first; the others' output is the token's own row
@@ -150,7 +168,7 @@ class RoutedMLP(FeedForward):
             offsets, order, place, tiles = ops.moe_align(idx, self.E)
             passing = {}
         if self.shared_inter:
-            passing["add"] = self._shared(x)
+            passing.update(add=self._shared(x), share=share)
         if self.E == 0:
             y = torch.empty((T * top, self.hidden), dtype=torch.float32, device=x.device)
         else:

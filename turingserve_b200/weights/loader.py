@@ -95,7 +95,7 @@ def load_into(model: DecoderModel, model_dir: str, names=None) -> None:
     for n, spec in expected.items():
         if n in files:
             got = tuple(handle(files[n]).get_slice(n).get_shape())
-            if got != tuple(spec.shape):
+            if not spec.fits(got):
                 wrong.append((n, got, tuple(spec.shape)))
     if missing or unexpected or wrong:
         raise WeightsError(missing, unexpected, wrong, model_dir)

@@ -28,8 +28,8 @@ from turingserve_b200.parts.model import DecoderModel
 def _random_table(spec: ParamSpec, g: torch.Generator, device) -> torch.Tensor:
     """An integer table: zeros, or ("distinct") rows of different numbers below ``spec.high``."""
     if spec.init != "distinct":
-        return torch.zeros(spec.shape, dtype=torch.int32, device=device)
-    rows, n = spec.shape
+        return torch.zeros(spec.sizes, dtype=torch.int32, device=device)
+    rows, n = spec.sizes
     if n > spec.high:
         raise ValueError(f"{n} different numbers below {spec.high}")
     draws = torch.rand((rows, spec.high), generator=g, device=device)
@@ -47,13 +47,13 @@ def random_tensors(cfg: ModelConfig, seed: int, std: float = 0.02,
         if spec.integer:
             out[name] = _random_table(spec, g, "cpu")
         elif spec.init == "ones":
-            out[name] = torch.ones(spec.shape, dtype=dtype)
+            out[name] = torch.ones(spec.sizes, dtype=dtype)
         elif spec.init == "zeros":
-            out[name] = torch.zeros(spec.shape, dtype=dtype)
+            out[name] = torch.zeros(spec.sizes, dtype=dtype)
         elif spec.init == "identity":
-            out[name] = torch.eye(*spec.shape, dtype=dtype)
+            out[name] = torch.eye(*spec.sizes, dtype=dtype)
         else:
-            out[name] = (torch.randn(spec.shape, generator=g, dtype=torch.float32) * std).to(dtype)
+            out[name] = (torch.randn(spec.sizes, generator=g, dtype=torch.float32) * std).to(dtype)
     return out
 
 
@@ -84,13 +84,13 @@ def random_model_on_device(cfg: ModelConfig, dtype: torch.dtype, device, seed: i
         if spec.integer:
             tensors[name] = _random_table(spec, g, device)
         elif spec.init == "ones":
-            tensors[name] = torch.ones(spec.shape, dtype=kind, device=device)
+            tensors[name] = torch.ones(spec.sizes, dtype=kind, device=device)
         elif spec.init == "zeros":
-            tensors[name] = torch.zeros(spec.shape, dtype=kind, device=device)
+            tensors[name] = torch.zeros(spec.sizes, dtype=kind, device=device)
         elif spec.init == "identity":
-            tensors[name] = torch.eye(*spec.shape, dtype=kind, device=device)
+            tensors[name] = torch.eye(*spec.sizes, dtype=kind, device=device)
         else:
-            t = torch.empty(spec.shape, dtype=kind, device=device)
+            t = torch.empty(spec.sizes, dtype=kind, device=device)
             t.normal_(0.0, std, generator=g)
             tensors[name] = t
     model.load(names, tensors)
