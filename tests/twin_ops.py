@@ -779,7 +779,7 @@ def _wkv_scan(self, out, r, k, v, w, u, h, state, step, H, D):
             kv = heads(k, t)[:, :, None] * heads(v, t)[:, None, :]
             out[t] = torch.einsum("hdv,hd->hv", S + u.view(H, D, 1) * kv, heads(r, t)).reshape(-1)
             S.mul_(heads(w, t)[:, :, None]).add_(kv)
-        row[H * D * D:] = h[hi - 1].float()
+        row[H * D * D:H * D * D + h.shape[1]] = h[hi - 1].float()
 
 
 def _wkv_project(self, *args):

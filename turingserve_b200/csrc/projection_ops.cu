@@ -272,7 +272,8 @@ batched_linear_rows_kernel(T* __restrict__ out, int out_ts, int out_hs, const T*
 // columns of one head and one of KS shares of k, whose weights it has on their way before the wait for the predecessor; the
 // rows go through shared memory once a block.  `x` may be the partial sums of a product cut along its own k (part [splits, M,
 // x_ts] 32-bit, summed in ascending order and rounded as that product's last pass would have).  (The products' k index is a
-// permutation of the real one, the same for both operands.)  The last block of a head (rot_dst set) turns R further columns of
+// permutation of the real one, the same for both operands.)  (What the predecessor writes comes through pointers that are not
+// __restrict__, so that no load of it may move ahead of the wait.)  The last block of a head (rot_dst set) turns R further columns of
 // its rows, those behind the first K, instead: the rotated part of a query beside its plain part's product.
 constexpr int BRM_WARPS = 8, BRM_UNROLL = 8, BRM_PAD = 32;
 
@@ -286,9 +287,8 @@ struct RowRotation {
 
 template <int ROWS, int KS>
 __global__ void __launch_bounds__(BRM_WARPS * 32)
-batched_rows_mma_kernel(bf16* __restrict__ out, int out_ts, int out_hs, const bf16* __restrict__ x, int x_ts, int x_hs,
-                        const float* __restrict__ part, int splits, const bf16* __restrict__ w, int M, int N, int K,
-                        RowRotation rot) {
+batched_rows_mma_kernel(bf16* out, int out_ts, int out_hs, const bf16* x, int x_ts, int x_hs, const float* part, int splits,
+                        const bf16* __restrict__ w, int M, int N, int K, RowRotation rot) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char brm_smem[];
   bf16* x_s = reinterpret_cast<bf16*>(brm_smem);                      // [ROWS][K + BRM_PAD]

@@ -11,6 +11,9 @@
 //                     afterwards the request's blocks store the last input
 //   ts_wkv_project    steps in which every token is a request of its own: the mixes and their products in one kernel
 //   ts_wkv_step       ... and the decay's second product, the recurrence, the heads' norm and the gate in another
+//
+// What a predecessor writes is read through pointers that are not __restrict__: the compiler holds the memory behind one that
+// is for constant over the whole kernel and may move its loads ahead of the wait for the predecessor.
 #include "activations.cuh"
 #include "common.cuh"
 #include "mma_utils.cuh"
@@ -28,7 +31,7 @@ constexpr int SH_MAX = 8;                                     // mixes a launch 
 
 template <typename T, int PER, int TOK>
 __global__ void __launch_bounds__(128)
-token_shift_kernel(T* __restrict__ out, const T* __restrict__ h, const T* __restrict__ mu, const float* __restrict__ state,
+token_shift_kernel(T* out, const T* h, const T* __restrict__ mu, const float* state,
                    size_t state_stride, size_t prev_off, const int* __restrict__ token_request, const int* __restrict__ q_start,
                    const int* __restrict__ slots, int T_, int hidden, int n) {
   pdl_launch_dependents();
@@ -95,7 +98,7 @@ constexpr int DC_M = 64, DC_N = 64, DC_K = 16, DC_PAD = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-wkv_decay_kernel(float* __restrict__ out, const float* __restrict__ z, const T* __restrict__ w2, const float* __restrict__ w0,
+wkv_decay_kernel(float* out, const float* z, const T* __restrict__ w2, const float* __restrict__ w0,
                  int M, int N, int R) {
   pdl_launch_dependents();
   pdl_wait();
@@ -147,10 +150,8 @@ constexpr int WK_GROUP = 16, WK_COLS = 16, WK_ROWS = 8;
 
 template <typename T>
 __global__ void __launch_bounds__(512, 1)
-wkv_scan_kernel(float* __restrict__ out, const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v,
-                const float* __restrict__ w, const float* __restrict__ u, const T* __restrict__ h_in,
-                float* __restrict__ state, size_t state_stride, const int* __restrict__ q_start,
-                const int* __restrict__ slots, int H, int D, int V, int hidden, int parts, int fast) {
+wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, const float* __restrict__ u, const T* h_in,
+                float* state, size_t state_stride, const int* __restrict__ q_start, const int* __restrict__ slots, int H, int D, int V, int hidden, int parts, int fast) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float smem[];
@@ -303,8 +304,8 @@ constexpr int PJ_WARPS = 16, PJ_COLS = 64, PJ_UNROLL = 8, PJ_PAD = 32;
 
 template <int ROWS>
 __global__ void __launch_bounds__(PJ_WARPS * 32)
-wkv_project_kernel(bf16* __restrict__ out, float* __restrict__ z, const bf16* __restrict__ h, const bf16* __restrict__ mu,
-                   const bf16* __restrict__ w, const bf16* __restrict__ w1, const float* __restrict__ state,
+wkv_project_kernel(bf16* out, float* z, const bf16* h, const bf16* __restrict__ mu, const bf16* __restrict__ w,
+                   const bf16* __restrict__ w1, const float* state,
                    size_t state_stride, size_t prev_off, const int* __restrict__ slots, int M, int n, int N, int R, int K) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char pj_smem[];
@@ -412,10 +413,10 @@ constexpr int ST_ROWS = 16;
 
 template <typename T, int THREADS>
 __global__ void __launch_bounds__(THREADS, THREADS == 256 ? 3 : 1)
-wkv_step_kernel(T* __restrict__ out, const T* __restrict__ rkvg, const float* __restrict__ z, const T* __restrict__ w2,
+wkv_step_kernel(T* out, const T* rkvg, const float* z, const T* __restrict__ w2,
                 const float* __restrict__ w0, const float* __restrict__ u, const float* __restrict__ norm_w, float eps,
-                const T* __restrict__ h_in, float* __restrict__ state, size_t state_stride, const int* __restrict__ slots,
-                int M, int H, int D, int R, int hidden, int cols, int w2_in_smem) {
+                const T* h_in, float* state, size_t state_stride, const int* __restrict__ slots, int M, int H, int D, int R,
+                int hidden, int cols, int w2_in_smem) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float st_smem[];
   __shared__ float scratch[32];
