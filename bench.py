@@ -1322,6 +1322,190 @@ def suranex_kernels(ops, z: dict, pk: dict, T: int, B: int, ctx: int, page: int)
     return out
 
 
+# ---- Fetedra (a matrix state per head that fades channel by channel, latent attention with a window, sinks and head gates,
+# grouped routing with a gated shared expert, a stream in copies) beside Pizunex layers of the same width (latent attention, a
+# matrix state per head) and Gugezen layers (the stream in copies, routed feed-forwards with a shared expert) ---------------
+FETEDRA_SIZES = {
+    # width; time mixer: heads, head width, rank of the decay; latent attention: heads, plain / rotated / value widths, latent
+    # sizes, window; gated dense ff; experts, groups and groups kept, top, expert ff, shared expert ff; the sizes beside it
+    "1.5b": dict(width=1536, heads=24, dim=64, rank=64, lheads=12, nope=128, rope=64, lvdim=128, q_rank=768, kv_rank=512, window=1024,
+                 ff=8960, experts=8, groups=4, keep=2, top=2, eff=1536, shared=1536, streams=2, beside="1.5b"),
+    "7b": dict(width=3584, heads=56, dim=64, rank=128, lheads=28, nope=128, rope=64, lvdim=128, q_rank=1536, kv_rank=512, window=1024,
+               ff=18944, experts=8, groups=4, keep=2, top=2, eff=4096, shared=4096, streams=2, beside="7b"),
+}
+
+
+def fetedra_config(z: dict, groups: int, vocab: int):
+    """``groups`` times four layers: (time mixer, dense), (latent attention, routed), (time mixer, routed), (latent attention,
+    dense)."""
+    from turingserve_b200.models.fetedra import make_config
+    wkv = {"type": "wkv", "mixer": {"heads": z["heads"], "dim": z["dim"], "decay_rank": z["rank"]}}
+    lat = {"type": "latent_attention", "mixer": {
+        "heads": z["lheads"], "dim": z["nope"], "rot_dim": z["rope"], "vdim": z["lvdim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+        "scale": (z["nope"] + z["rope"]) ** -0.5, "mask": {"size": z["window"]}, "rot": {"base": 500000.0, "dims": z["rope"]}}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"], "limit": 7.0}, "shared": {"ff": z["shared"], "limit": 6.0},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": z["groups"], "keep": z["keep"]}}}
+    four = [{**wkv, "mlp": dense}, {**lat, "mlp": moe}, {**wkv, "mlp": moe}, {**lat, "mlp": dense}]
+    return make_config(width=z["width"], vocab=vocab, layers=four * groups, eps=1e-6, streams=z["streams"], logit_scale=0.5)
+
+
+def fetedra_kernels(ops, z: dict, pk: dict, T: int, B: int, ctx: int, page: int) -> dict:
+    """Each kernel of the new mechanisms alone, beside the like kernel of the closest designs: a portion of T tokens and B
+    single tokens at context ``ctx``."""
+    import torch
+    from types import SimpleNamespace
+    dev = torch.device("cuda", 0)
+    big = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    flush = lambda: big.fill_(1)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    out = {}
+    hbm = pk["hbm_gbs"] * 1e9
+    bf = torch.bfloat16
+    W = z["width"]
+    us = lambda ms: round(ms * 1e3, 1)
+    frac = lambda byts, ms: round(byts / (ms / 1e3) / hbm, 3)
+    tensor = lambda flops, ms: round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 3)
+    fp32 = lambda flops, ms: round(flops / (ms / 1e3) / FP32_PEAK, 3)
+    rn = lambda *s: torch.randn(*s, device=dev)
+
+    # the time mixer, beside the delta rule (Pizunex), the linear attention and the state-space mixer (Gugezen)
+    H, D, R = z["heads"], z["dim"], z["rank"]
+    n = H * D
+    p, g = PIZUNEX_SIZES[z["beside"]], GUGEZEN_SIZES[z["beside"]]
+    dH, dG, dD, dV, taps = p["dheads"], p["dkv"], p["ddim"], p["dvdim"], 4
+    dqk, dhv = dG * dD, dH * dV
+    LH, LD = g["lheads"], g["dim"]
+    SH, P, N, SG = g["sheads"], g["sdim"], g["state"], g["sgroups"]
+    inner, channels = SH * P, SH * P + 2 * SG * N
+    mu, w2 = rn(5, W).to(bf), (rn(n, R) * 0.05).to(bf)
+    wp, w1 = (rn(4, n, W) * 0.02).to(bf), (rn(R, W) * 0.02).to(bf)
+    w0, u, nw = rn(n) - 4.0, rn(H, D), torch.ones(n, device=dev)
+    for name, reqs, per in (("prefill", 1, T), ("decode", B, 1)):
+        rows = reqs * per
+        h = rn(rows, W).to(bf)
+        slot = -(-(n * D + W) // 4) * 4
+        state = torch.zeros(reqs + 1, slot, device=dev)
+        step = SimpleNamespace(q_start=i32([i * per for i in range(reqs + 1)]), state_slots=i32(list(range(reqs))), num_requests=reqs,
+                               token_request=i32([r for r in range(reqs) for _ in range(per)]), max_q_len=per)
+        mixes, rkvg = torch.empty(5, rows, W, dtype=bf, device=dev), rn(4, rows, n).to(bf)
+        zz, w = rn(rows, R), torch.empty(rows, n, device=dev)
+        o, y = torch.empty(rows, n, device=dev), torch.empty(rows, n, dtype=bf, device=dev)
+        ms_s = timed(lambda: ops.token_shift(mixes, h, mu, state, n * D, step), flush)
+        ms_d = timed(lambda: ops.wkv_decay(w, zz, w2, w0), flush)
+        ms_k = timed(lambda: ops.wkv_scan(o, rkvg[0], rkvg[1], rkvg[2], w, u, h, state, step, H, D), flush)
+        ms_n = timed(lambda: ops.head_gated_rmsnorm(y, o, rkvg[3], nw, 1e-6, H, D), flush)
+        # decay (multiply, add) and read (multiply, add) and the product k v: five operations a state value a token
+        fl = 5.0 * rows * n * D
+        entry = {"shift_us": us(ms_s), "shift_frac_of_hbm": frac(rows * W * 12.0, ms_s), "decay_us": us(ms_d),
+                 "decay_frac_of_hbm": frac(rows * (n + R) * 4.0 + n * R * 2.0, ms_d), "scan_us": us(ms_k),
+                 "scan_tflops_fp32": round(fl / ms_k / 1e9, 2), "scan_frac_of_fp32_nominal": fp32(fl, ms_k),
+                 "scan_frac_of_hbm": frac(reqs * n * D * 8.0 + rows * n * (6.0 + 8.0), ms_k), "head_norm_us": us(ms_n),
+                 "head_norm_frac_of_hbm": frac(rows * n * 8.0, ms_n)}
+        if per == 1:
+            ms_p = timed(lambda: ops.wkv_project(rkvg, zz, h, mu, wp, w1, state, n * D, step), flush)
+            ms_1 = timed(lambda: ops.wkv_step(y, rkvg, zz, w2, w0, u, nw, 1e-6, h, state, step, H, D), flush)
+            x4 = torch.empty(rows, 4 * n, dtype=bf, device=dev)
+            ms_l = timed(lambda: ops.linear(x4, h, wp.view(4 * n, W)), flush)
+            entry.update({"project_us": us(ms_p), "project_frac_of_hbm": frac((4 * n + R) * W * 2.0, ms_p),
+                          "beside_plain_product_us": us(ms_l), "beside_plain_product_frac_of_hbm": frac(4 * n * W * 2.0, ms_l),
+                          "step_us": us(ms_1), "step_frac_of_hbm": frac(reqs * n * D * 8.0 + n * R * 2.0 + rows * n * 10.0, ms_1)})
+        # beside: the delta rule
+        dC = 2 * dqk + dhv
+        dproj = rn(rows, dC + dhv + 2 * dH).to(bf)
+        dstate = torch.zeros(reqs + 1, dH * dD * dV + (taps - 1) * dC, device=dev)
+        ready, do = torch.empty(rows, dC + 2 * dH + dG, device=dev), torch.empty(rows, dhv, device=dev)
+        conv, zh = rn(dC, taps) * 0.3, torch.zeros(dH, device=dev)
+        ms = timed(lambda: ops.delta_prepare(ready, dproj, conv, zh, zh, dstate, step, dH, dG, dD, dV, taps, 1e-6), flush)
+        ms_b = timed(lambda: ops.delta_scan(do, ready, dproj, dstate, step, dH, dG, dD, dV, taps), flush)
+        dn = torch.empty(rows, dhv, dtype=bf, device=dev)
+        ms_h = timed(lambda: ops.head_gated_rmsnorm(dn, do, dproj[:, dC:dC + dhv], torch.ones(dV, device=dev), 1e-6, dH, dV), flush)
+        dfl = 8.0 * rows * dH * dD * dV
+        entry.update({"beside_delta_prepare_us": us(ms), "beside_delta_prepare_frac_of_hbm": frac(rows * (dC * 6.0), ms),
+                      "beside_delta_scan_us": us(ms_b), "beside_delta_scan_frac_of_fp32_nominal": fp32(dfl, ms_b),
+                      "beside_delta_scan_frac_of_hbm": frac(reqs * dH * dD * dV * 8.0 + rows * dC * 4.0, ms_b),
+                      "beside_head_norm_us": us(ms_h), "beside_head_norm_frac_of_hbm": frac(rows * dhv * 8.0, ms_h)})
+        # beside: the linear attention and the state-space mixer
+        lproj, lo = rn(rows, 4 * LH * LD).to(bf), torch.empty(rows, LH * LD, device=dev)
+        lstate, decay = torch.zeros(reqs + 1, LH, LD, LD, device=dev), torch.full((LH,), 0.99, device=dev)
+        ms = timed(lambda: ops.lightning(lo, lproj, lstate, decay, step, LH, LD, LD), flush)
+        sproj, sready = rn(rows, 2 * inner + 2 * SG * N + SH).to(bf), rn(rows, channels + 2 * SH)
+        sstate, so, hz = torch.zeros(reqs + 1, SH * N * P + (taps - 1) * channels, device=dev), torch.empty(rows, inner, device=dev), torch.zeros(SH, device=dev)
+        ms_q = timed(lambda: ops.ssm_scan(so, sready, sproj, inner, sstate, hz, step, SH, SG, N, P, taps), flush)
+        entry.update({"beside_linear_scan_us": us(ms), "beside_linear_scan_frac_of_fp32_nominal": fp32(5.0 * rows * LH * LD * LD, ms),
+                      "beside_linear_scan_frac_of_hbm": frac(reqs * LH * LD * LD * 8.0 + rows * LH * LD * 10.0, ms),
+                      "beside_ssm_scan_us": us(ms_q), "beside_ssm_scan_frac_of_fp32_nominal": fp32(5.0 * rows * SH * N * P, ms_q),
+                      "beside_ssm_scan_frac_of_hbm": frac(reqs * SH * N * P * 8.0 + rows * (channels + inner) * 4.0, ms_q)})
+        out[f"time_mixer_{name}"] = entry
+
+    # latent attention: the projection's parts, the queries' way into the latent space, the attention with window, sinks and
+    # gates; beside it without them (what Pizunex runs)
+    lH, dn, dr, dv, qr, rank, win = (z[k] for k in ("lheads", "nope", "rope", "lvdim", "q_rank", "kv_rank", "window"))
+    row = rank + dr
+    pages = B * (-(-(ctx + 1) // page)) + -(-T // page) + 2
+    width = -(-max(ctx + 1, T) // page)
+    kc = rn(pages, 1, page, row).to(bf)
+    freq = (500000.0 ** (-2.0 * torch.arange(dr // 2, dtype=torch.float64) / dr)).float().to(dev)
+    kw_, qw_ = torch.ones(rank, device=dev), torch.ones(qr, device=dev)
+    n_in = -(-(qr + row + lH) // 8) * 8
+    ukt, uv = (rn(lH, rank, dn) * 0.05).to(bf), (rn(lH, dv, rank) * 0.05).to(bf)
+    sinks = torch.zeros(lH, device=dev)
+    for name, reqs, per, seq in (("prefill", 1, T, T), ("decode", B, 1, ctx + 1)):
+        rows = reqs * per
+        proj, cq = rn(rows, n_in).to(bf), torch.empty(rows, qr, dtype=bf, device=dev)
+        pos, slots = i32(list(range(rows))), i32(list(range(page, page + rows)))
+        ms_w = timed(lambda: ops.latent_kv_write(proj, qr, kw_, 1e-6, pos, freq, 1.0, dr, kc, slots, rank, dr, page, "halves", cq, qw_), flush)
+        ms_w2 = timed(lambda: ops.latent_kv_write(proj, qr, kw_, 1e-6, pos, freq, 1.0, dr, kc, slots, rank, dr, page, "neighbours"), flush)
+        q, qa = rn(rows, lH * (dn + dr)).to(bf), torch.empty(rows, lH, row, dtype=bf, device=dev)
+        ms_q = timed(lambda: ops.latent_queries(qa, q, ukt, pos, freq, 1.0, dr, "halves"), flush)
+        mixed, heads = torch.empty(rows, lH, rank, dtype=bf, device=dev), torch.empty(rows, lH, dv, dtype=bf, device=dev)
+        ms_v = timed(lambda: ops.batched_linear(heads, mixed, uv), flush)
+        bt = torch.zeros(reqs, width, dtype=torch.int32, device=dev)
+        m = -(-seq // page)
+        for r in range(reqs):
+            bt[r, :m] = torch.arange(1 + r * m, 1 + (r + 1) * m, dtype=torch.int32, device=dev)
+        step = SimpleNamespace(q_start=i32([i * per for i in range(reqs + 1)]), seq_lens=i32([seq] * reqs), num_requests=reqs,
+                               num_decode=reqs if per == 1 else 0, max_q_len=per, max_seq_len=seq)
+        qa = rn(rows, lH, row).to(bf)
+        gate = proj[:, qr + row:qr + row + lH]
+        entry = {"rows_us": us(ms_w), "rows_frac_of_hbm": frac(rows * (qr + row) * 4.0, ms_w), "beside_cache_row_us": us(ms_w2),
+                 "beside_cache_row_frac_of_hbm": frac(rows * row * 4.0, ms_w2), "queries_us": us(ms_q),
+                 "queries_frac_of_hbm": frac(lH * rank * dn * 2.0 + rows * lH * (dn + dr + row) * 2.0, ms_q),
+                 "queries_frac_of_bf16": tensor(2.0 * rows * lH * rank * dn, ms_q), "values_us": us(ms_v),
+                 "values_frac_of_hbm": frac(lH * rank * dv * 2.0 + rows * lH * (rank + dv) * 2.0, ms_v)}
+        for tag, w, mine in (("", win, True), ("no_window_", None, True), ("beside_plain_", None, False)):
+            kw = dict(sinks=sinks, gate=gate) if mine else {}
+            ms = timed(lambda: ops.attention_biased(mixed, qa, kc, None, bt, step, 1, page, (dn + dr) ** -0.5, 0.0, None, w, **kw), flush)
+            seen = sum(min(i + 1, w) if w else i + 1 for i in range(seq - per, seq))
+            held = min(seq, w) if w and per == 1 else seq
+            fl = 2.0 * (row + rank) * lH * seen * reqs
+            entry.update({f"attention_{tag}us": us(ms), f"attention_{tag}tflops": round(fl / ms / 1e9, 1),
+                          f"attention_{tag}frac_of_bf16": tensor(fl, ms),
+                          f"attention_{tag}frac_of_hbm": frac(reqs * held * row * 2.0 + rows * lH * (row + rank) * 2.0, ms)})
+        out[f"latent_attention_{name}"] = entry
+
+    # the router with groups, correction and the shared expert's row, beside the plain one; the sum of a token's choices with
+    # and without the shared expert's weight
+    E, top, ff = z["experts"], z["top"], z["eff"]
+    wr, corr = rn(E + 1, W) * 0.05, rn(E) * 0.1
+    for name, rows in (("prefill", T), ("decode", B)):
+        x = rn(rows, W).to(bf)
+        idx, wts, share = torch.empty(rows, top, dtype=torch.int32, device=dev), torch.empty(rows, top, device=dev), torch.empty(rows, device=dev)
+        ms = timed(lambda: ops.router_topk(idx, wts, x, wr, False, True, corr, z["groups"], z["keep"], 2.5, share), flush)
+        ms_p = timed(lambda: ops.router_topk(idx, wts, x, wr[:E], True, True), flush)
+        ops.router_topk(idx, wts, x, wr, False, True, corr, z["groups"], z["keep"], 2.5, share)
+        offsets, order, place, tiles = ops.moe_align(idx, E)
+        y, add, o = rn(rows * top, W), rn(rows, W).to(bf), torch.empty(rows, W, dtype=bf, device=dev)
+        ms_c = timed(lambda: ops.moe_combine(o, y, place, wts, top, add=add, share=share), flush)
+        ms_d = timed(lambda: ops.moe_combine(o, y, place, wts, top, add=add), flush)
+        out[f"routed_ff_{name}"] = {
+            "router_us": us(ms), "router_frac_of_hbm": frac(rows * W * 2.0 + (E + 1) * W * 4.0, ms), "beside_plain_router_us": us(ms_p),
+            "beside_router_frac_of_hbm": frac(rows * W * 2.0 + E * W * 4.0, ms_p), "sum_us": us(ms_c),
+            "sum_frac_of_hbm": frac(rows * W * (4.0 + 4 * top), ms_c), "beside_plain_sum_us": us(ms_d),
+            "beside_sum_frac_of_hbm": frac(rows * W * (4.0 + 4 * top), ms_d)}
+    return out
+
+
 def run_design(a) -> dict:
     """``--design komirax``: prefill and decode throughput of Komirax layers beside Qwen2 layers of the same
     width and count (random weights, bfloat16, through the step function), and each new kernel alone."""
@@ -1439,6 +1623,26 @@ def run_design(a) -> dict:
                          decode_ratio=round(entry["suranex"]["decode_tok_s"] / entry["gugezen"]["decode_tok_s"], 3))
             if "kernels" in a.phases.split(","):
                 entry["kernels"] = suranex_kernels(ops, z, pk, T, B, ctx, page)
+            result["sizes"][name] = entry
+            continue
+        if a.design == "fetedra":
+            # beside Pizunex layers (latent attention, a matrix state per head) and Gugezen layers (the stream in copies, routed
+            # feed-forwards with a shared expert) of the same width
+            z = FETEDRA_SIZES[name]
+            made = (("fetedra", fetedra_config(z, groups, vocab)), ("pizunex", pizunex_config(PIZUNEX_SIZES[z["beside"]], groups, vocab)),
+                    ("gugezen", gugezen_config(GUGEZEN_SIZES[z["beside"]], groups, vocab)))
+            entry = {"layers": 4 * groups, "width": z["width"], "beside": [f"pizunex-{z['beside']}", f"gugezen-{z['beside']}"]}
+            for which, mcfg in made:
+                eng = build_engine_on_device(f"{which}-{name}", 4 * groups, ctx_len=ctx_len, page=page, max_seqs=B,
+                                             max_tokens=max(T, ctx), graph_sizes=(B,), mcfg=mcfg)
+                entry[which] = measure(eng)
+                del eng
+                torch.cuda.empty_cache()
+            for which in ("pizunex", "gugezen"):
+                entry.update({f"prefill_ratio_{which}": round(entry["fetedra"]["prefill_tok_s"] / entry[which]["prefill_tok_s"], 3),
+                              f"decode_ratio_{which}": round(entry["fetedra"]["decode_tok_s"] / entry[which]["decode_tok_s"], 3)})
+            if "kernels" in a.phases.split(","):
+                entry["kernels"] = fetedra_kernels(ops, z, pk, T, B, ctx, page)
             result["sizes"][name] = entry
             continue
         if a.design == "pizunex":
@@ -1570,9 +1774,10 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=2048)
     ap.add_argument("--phases", default="prefill,decode,points,e2e,kernels,mixed",
                     help="which measurements to run (decode always runs); fewer for a profiler capture")
-    ap.add_argument("--design", default="", choices=["", "komirax", "pizunex", "vofinex", "gugezen", "suranex"],
+    ap.add_argument("--design", default="", choices=["", "komirax", "pizunex", "vofinex", "gugezen", "suranex", "fetedra"],
                     help="instead of the default workload: layers of this design beside layers of the closest other one (Komirax "
-                         "beside Qwen2, Pizunex, Vofinex and Gugezen beside Komirax, Suranex beside Gugezen) at the same width "
+                         "beside Qwen2, Pizunex, Vofinex and Gugezen beside Komirax, Suranex beside Gugezen, Fetedra beside Pizunex "
+                         "and Gugezen) at the same width "
                          "(prefill and decode throughput, and each of the design's kernels alone)")
     ap.add_argument("--design-sizes", default="1.5b,7b", help="which of the design's layer sizes to run")
     a = ap.parse_args()

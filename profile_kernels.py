@@ -460,7 +460,7 @@ def main() -> int:
     s.add_argument("--layers", type=int, default=4)
     s.add_argument("--page", type=int, default=PAGE)
     s = sub.add_parser("design_step")
-    s.add_argument("--design", default="gugezen", choices=["komirax", "pizunex", "vofinex", "gugezen", "suranex"])
+    s.add_argument("--design", default="gugezen", choices=["komirax", "pizunex", "vofinex", "gugezen", "suranex", "fetedra"])
     s.add_argument("--size", default="1.5b")
     s.add_argument("--layers", type=int, default=4)
     s.add_argument("--prefill", type=int, default=0, help="a prompt of this many tokens (0: single tokens)")

@@ -151,7 +151,8 @@ constexpr int WK_GROUP = 16, WK_COLS = 16, WK_ROWS = 8;
 template <typename T>
 __global__ void __launch_bounds__(512, 1)
 wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, const float* __restrict__ u, const T* h_in,
-                float* state, size_t state_stride, const int* __restrict__ q_start, const int* __restrict__ slots, int H, int D, int V, int hidden, int parts, int fast) {
+                float* state, size_t state_stride, const int* __restrict__ q_start, const int* __restrict__ slots, int H, int D,
+                int V, int hidden, int parts, int fast) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float smem[];

@@ -46,13 +46,13 @@ def _mixer(kind: str, m: dict, eps: float, where: str):
         dims = int(rot.get("dims", rope_dim))
         if dims > rope_dim or dims % 2:
             raise ValueError(f"{where}: rot.dims {dims} must be even and at most rot_dim {rope_dim}")
-        mask = m.get("mask") or None
+        mask = m.get("mask")
         return LatentAttentionSpec(
             num_heads=heads, nope_dim=dim, rope_dim=rope_dim, value_dim=int(_require(m, "vdim", where)),
             q_rank=int(_require(m, "q_rank", where)), kv_rank=int(_require(m, "kv_rank", where)),
             scale=float(_require(m, "scale", where)), norm_eps=eps,
             position=HalfRotarySpec(base=float(_require(rot, "base", where)), dims=dims),
-            window=int(_require(mask, "size", where)) if mask else None, sinks=True, head_gate=True)
+            window=int(_require(mask, "size", where)) if mask is not None else None, sinks=True, head_gate=True)
     raise ValueError(f"{where}: unknown layer type {kind!r} (known: wkv, latent_attention)")
 
 
