@@ -1362,6 +1362,7 @@ def fetedra_kernels(ops, z: dict, pk: dict, T: int, B: int, ctx: int, page: int)
     out = {}
     hbm = pk["hbm_gbs"] * 1e9
     bf = torch.bfloat16
+    FP32_PEAK = 148 * 128 * 2 * 1.965e9                      # FFMA lanes x 2 x the highest SM clock: nominal
     W = z["width"]
     us = lambda ms: round(ms * 1e3, 1)
     frac = lambda byts, ms: round(byts / (ms / 1e3) / hbm, 3)
