@@ -135,3 +135,244 @@ class Unit:
 
 UNITS = pytest.mark.parametrize("H,D,hidden,R", [(3, 20, 60, 12), (2, 7, 33, 5), (4, 64, 128, 32), (2, 128, 96, 16), (1, 40, 48, 24),
                                                  (3, 48, 200, 16), (1, 256, 64, 8), (2, 33, 40, 1), (32, 64, 2048, 64)])
+
+
+@DTYPES
+@UNITS
+def test_time_mixer_whole_in_portions_and_token_by_token(ops, dtype, H, D, hidden, R):
+    """One sequence in four ways beside another request, slots that others left something in: the same outputs and the same
+    last state, and the outputs are the plain ones."""
+    g = torch.Generator(device=DEV).manual_seed(H * D)
+    u = Unit(g, H, D, hidden, R, dtype)
+    T = 37 if H * D <= 512 else 19
+    h = torch.randn(T, hidden, generator=g, device=DEV).to(dtype)
+    other = torch.randn(T + 8, hidden, generator=g, device=DEV).to(dtype)
+    want, S = u.plain(h)
+    slack = 4.0 if dtype == torch.bfloat16 else 60.0
+    states = []
+    for cuts in ([T], [2, 3, 16, T - 21] if T > 22 else [2, 3, T - 5], [1] * T, [T - 3, 1, 1, 1]):
+        state = torch.randn(4, u.slot, generator=g, device=DEV)
+        state[2].zero_()
+        got, at = [], 0
+        for n in cuts:
+            rows, _ = u.run(ops, torch.cat([other[:n + 1], h[at:at + n]]), batch([n + 1, n], [0, 2]), state)
+            got.append(rows[n + 1:])
+            at += n
+        out = torch.cat(got)
+        assert close(out, want, dtype, slack), (cuts, float((out.double().cpu() - want).abs().max()))
+        states.append(state[2].clone())
+    assert close(states[0][:u.off].view(H, D, D), S, torch.float32, 2e4 if dtype == torch.bfloat16 else 60.0)
+    lim = dict(rtol=1e-5, atol=1e-5) if dtype == torch.float32 else dict(rtol=2e-2, atol=2e-2)
+    for s in states:
+        assert torch.equal(s[u.off:u.off + hidden], h[-1].float())
+        assert torch.allclose(s[:u.off], states[0][:u.off], **lim)
+
+
+@DTYPES
+@UNITS
+@pytest.mark.parametrize("B", [1, 5, 8, 9, 16, 20])
+def test_single_tokens_in_one_kernel_steps(ops, dtype, H, D, hidden, R, B):
+    """Batches of single tokens against the kernels of portions: products of 8 and of 16 rows, heads whose state one block holds
+    and heads too wide for it; requests in slots of any order, other slots untouched."""
+    g = torch.Generator(device=DEV).manual_seed(B)
+    u = Unit(g, H, D, hidden, R, dtype)
+    state = torch.randn(B + 2, u.slot, generator=g, device=DEV) * 0.3
+    slots = torch.randperm(B + 2, generator=torch.Generator().manual_seed(B)).tolist()[:B]
+    a, b = state.clone(), state.clone()
+    for t in range(3):
+        h = torch.randn(B, hidden, generator=g, device=DEV).to(dtype)
+        step = batch([1] * B, slots)
+        y1, used = u.run(ops, h, step, a)
+        y2, _ = u.run(ops, h, step, b, one_kernel=False)
+        assert used[0] == (dtype == torch.bfloat16 and hidden % 8 == 0 and B <= 16 and u.off % 4 == 0)
+        assert used[1] == (-(-D // 32) * 32 * -(-D // 16) <= 1024)
+        assert close(y1, y2, dtype, 4.0 if dtype == torch.bfloat16 else 60.0), (t, float((y1.float() - y2.float()).abs().max()))
+    idle = [s for s in range(B + 2) if s not in slots]
+    assert torch.equal(a[idle], state[idle]) and torch.equal(b[idle], state[idle])
+    lim = dict(rtol=1e-5, atol=1e-5) if dtype == torch.float32 else dict(rtol=3e-2, atol=3e-2)
+    assert torch.allclose(a[slots], b[slots], **lim)
+
+
+@DTYPES
+@pytest.mark.parametrize("D", [16, 20, 64, 100])
+def test_a_slow_channel_keeps_a_value_for_a_thousand_tokens(ops, dtype, D):
+    """One loud key and value, then silence: the read-out a thousand tokens later is the product of the decays between, in one
+    portion, in portions and over single tokens; the bonus counts at the token itself only."""
+    H, T = 1, 1000
+    u = Unit(torch.Generator(device=DEV).manual_seed(3), H, D, 24, 4, dtype)
+    r, k, v = (torch.zeros(T, D, dtype=dtype, device=DEV) for _ in range(3))
+    k[0, 5], v[0, 9] = 2.0, 3.0
+    r[:, 5] = 1.0
+    w = torch.rand(T, D, generator=torch.Generator(device=DEV).manual_seed(4), device=DEV) * 1e-3 + 0.9985
+    bonus = torch.full((1, D), -0.5, device=DEV)
+    h = torch.randn(T, 24, device=DEV).to(dtype)
+    want = torch.zeros(T, dtype=torch.float64)
+    want[0] = -3.0
+    want[1:] = 6.0 * torch.cat([torch.ones(1, dtype=torch.float64), w[1:-1, 5].double().cpu().cumprod(0)])
+    for cuts in ([T], [7, 16, 2, 1, 300, T - 326], [500] + [1] * 500):
+        state, out, at = torch.zeros(1, u.slot, device=DEV), torch.empty(T, D, device=DEV), 0
+        for n in cuts:
+            s = slice(at, at + n)
+            ops.wkv_scan(out[s], r[s], k[s], v[s], w[s], bonus, h[s], state, batch([n], [0]), H, D)
+            at += n
+        assert float((out[:, 9].double().cpu() - want).abs().max()) < 2e-4
+        assert float(out[:, :9].abs().max()) == 0.0 and float(out[:, 10:].abs().max()) == 0.0
+
+
+@DTYPES
+@pytest.mark.parametrize("H,D", [(3, 24), (2, 64), (1, 128)])
+def test_unequal_requests_in_one_scan_are_bit_for_bit_those_alone(ops, dtype, H, D):
+    """Requests of 1 to 150 tokens in one launch, each alone, and each cut in two: the same bits of outputs and states."""
+    g = torch.Generator(device=DEV).manual_seed(8)
+    rn = lambda *s: torch.randn(*s, generator=g, device=DEV)
+    cuts, slots, n, hid = [1, 150, 16, 17, 2, 33], [5, 0, 3, 1, 6, 2], H * D, 40
+    T = sum(cuts)
+    r, k, v = (rn(T, n).to(dtype) for _ in range(3))
+    w, bonus, h = torch.rand(T, n, generator=g, device=DEV), rn(H, D), rn(T, hid).to(dtype)
+    state = rn(7, n * D + hid)
+    both, out = state.clone(), torch.empty(T, n, device=DEV)
+    ops.wkv_scan(out, r, k, v, w, bonus, h, both, batch(cuts, slots), H, D)
+    at = 0
+    for m, slot in zip(cuts, slots):
+        for parts in ([m], [m - m // 3, m // 3] if m > 2 else [m]):
+            one, got, p = state.clone(), torch.empty(m, n, device=DEV), 0
+            for q in parts:
+                s, d = slice(at + p, at + p + q), slice(p, p + q)
+                ops.wkv_scan(got[d], r[s], k[s], v[s], w[s], bonus, h[s], one, batch([q], [slot]), H, D)
+                p += q
+            assert torch.equal(got, out[at:at + m]) and torch.equal(one[slot], both[slot])
+        at += m
+
+
+@DTYPES
+def test_norm_of_heads_with_weights_of_their_own(ops, dtype):
+    g = torch.Generator(device=DEV).manual_seed(1)
+    for T, H, V in ((9, 4, 15), (600, 5, 64), (3, 24, 64), (520, 3, 128)):
+        x, gate = torch.randn(T, H * V, generator=g, device=DEV) * 3, torch.randn(T, H * V, generator=g, device=DEV).to(dtype)
+        w = torch.randn(H * V, generator=g, device=DEV)
+        out = torch.empty(T, H * V, dtype=dtype, device=DEV)
+        ops.head_gated_rmsnorm(out, x, gate, w, 0.2, H, V)
+        unit = plain.unit_rms(x.double().view(T, H, V), 0.2).reshape(T, H * V)
+        assert close(out, unit * w.double() * plain.silu(gate.double()), dtype, 6.0)
+        common = w[:V].contiguous()
+        ops.head_gated_rmsnorm(out, x, gate, common, 0.2, H, V)
+        assert close(out, unit * common.double().repeat(H) * plain.silu(gate.double()), dtype, 6.0)
+
+
+# -- latent attention ----------------------------------------------------------------------------------------------------------
+def freqs(base, dims):
+    return torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], device=DEV)
+
+
+def turn(x, pos, base, dims, pairing):
+    if pairing == "halves":
+        return plain.rotate_halves(x, pos, base, dims)
+    order = list(range(0, dims, 2)) + list(range(1, dims, 2)) + list(range(dims, x.shape[-1]))     # neighbours -> halves
+    y = plain.rotate_halves(x[..., order], pos, base, dims)
+    back = torch.empty_like(y)
+    back[..., order] = y
+    return back
+
+
+@DTYPES
+@pytest.mark.parametrize("pairing", ["halves", "neighbours"])
+@pytest.mark.parametrize("T,q_rank,rank,R,rot,extra", [(1, 20, 28, 6, 6, 3), (9, 14, 18, 10, 6, 5), (40, 768, 512, 64, 64, 12), (3, 8, 24, 4, 4, 0)])
+def test_rows_of_a_latent_projection(ops, dtype, pairing, T, q_rank, rank, R, rot, extra):
+    """The cached row and the query latent of every token; a slot of -1 caches nothing; other rows of the pool untouched."""
+    g = torch.Generator(device=DEV).manual_seed(T + rank)
+    n_in, page = q_rank + rank + R + extra, 8
+    proj = (torch.randn(T, n_in, generator=g, device=DEV) * 2).to(dtype)
+    kw, qw = 1 + 0.3 * torch.randn(rank, generator=g, device=DEV), 1 + 0.3 * torch.randn(q_rank, generator=g, device=DEV)
+    pos = torch.randint(0, 3000, (T,), generator=g, device=DEV, dtype=torch.int32)
+    slots = (torch.randperm(T + 16, generator=torch.Generator().manual_seed(T))[:T] + page).to(torch.int32).to(DEV)
+    if T > 2:
+        slots[1] = -1
+    pool = torch.full((-(-(T + 16) // page) + 2, 1, page, rank + R), 7.0, dtype=dtype, device=DEV)
+    cq = torch.empty(T, q_rank, dtype=dtype, device=DEV)
+    back = ops.latent_kv_write(proj, q_rank, kw, 0.1, pos, freqs(50.0, rot), 1.0, rot, pool, slots, rank, R, page, pairing, cq, qw)
+    assert back is proj
+    p = proj.double().cpu()
+    assert close(cq, plain.unit_rms(p[:, :q_rank], 0.1) * qw.double().cpu(), dtype, 4.0)
+    c = plain.unit_rms(p[:, q_rank:q_rank + rank], 0.1) * kw.double().cpu()
+    kr = turn(p[:, q_rank + rank:q_rank + rank + R], pos.cpu(), 50.0, rot, pairing)
+    flat, seen = pool.view(-1, rank + R), []
+    for t, s in enumerate(slots.tolist()):
+        if s >= 0:
+            seen.append(s)
+            assert close(flat[s, :rank], c[t], dtype, 4.0)
+            assert float((flat[s, rank:].double().cpu() - kr[t]).abs().max()) < (0.06 if dtype == torch.bfloat16 else 5e-3)
+    rest = [i for i in range(flat.shape[0]) if i not in seen]
+    assert bool((flat[rest] == 7.0).all())
+
+
+@pytest.mark.parametrize("T", [1, 8, 40])
+def test_rows_of_a_product_left_unreduced(ops, T):
+    """The projection's partial sums: the values from the finished product, gates finished in place."""
+    from turingserve_b200 import kernels
+    g = torch.Generator(device=DEV).manual_seed(T)
+    q_rank, rank, R, H, K, page = 96, 64, 16, 6, 1024, 16
+    n_in = q_rank + rank + R + 8
+    x = torch.randn(T, K, generator=g, device=DEV).to(torch.bfloat16)
+    w = (torch.randn(n_in, K, generator=g, device=DEV) * 0.05).to(torch.bfloat16)
+    kw, qw = torch.ones(rank, device=DEV), torch.ones(q_rank, device=DEV)
+    pos, slots = i32(list(range(T))), i32(list(range(page, page + T)))
+    results = []
+    for defer in (False, True):
+        proj = torch.empty(T, n_in, dtype=torch.bfloat16, device=DEV)
+        p = ops.linear(proj, x, w, may_defer=defer, lazy=False)
+        assert isinstance(p, kernels.Deferred) == defer
+        pool = torch.zeros(8, 1, page, rank + R, dtype=torch.bfloat16, device=DEV)
+        cq = torch.empty(T, q_rank, dtype=torch.bfloat16, device=DEV)
+        back = ops.latent_kv_write(p, q_rank, kw, 1e-6, pos, freqs(100.0, R), 1.0, R, pool, slots, rank, R, page, "halves", cq, qw,
+                                   (q_rank + rank + R, H))
+        results.append((pool, cq, back[:, q_rank + rank + R:q_rank + rank + R + H].clone()))
+    for a, b in zip(*results):
+        assert close(a, b, torch.bfloat16, 2.0) and float(a.abs().max()) > 0
+
+
+@DTYPES
+@pytest.mark.parametrize("pairing", ["halves", "neighbours"])
+@pytest.mark.parametrize("T", [1, 7, 8, 13, 16, 17, 70])
+@pytest.mark.parametrize("H,N,K,R,rot", [(3, 28, 10, 6, 6), (3, 256, 32, 64, 64), (12, 512, 128, 64, 64), (2, 96, 320, 8, 4), (5, 72, 24, 16, 16)])
+def test_queries_into_the_latent_space(ops, dtype, pairing, T, H, N, K, R, rot):
+    g = torch.Generator(device=DEV).manual_seed(T * H)
+    q = torch.randn(T, H * (K + R), generator=g, device=DEV).to(dtype)
+    w = (torch.randn(H, N, K, generator=g, device=DEV) * K ** -0.5).to(dtype)
+    pos = torch.randint(0, 2000, (T,), generator=g, device=DEV, dtype=torch.int32)
+    qa = torch.empty(T, H, N + R, dtype=dtype, device=DEV)
+    ops.latent_queries(qa, q, w, pos, freqs(80.0, rot), 1.0, rot, pairing)
+    heads = q.double().cpu().view(T, H, K + R)
+    assert close(qa[:, :, :N], torch.einsum("thk,hnk->thn", heads[:, :, :K], w.double().cpu()), dtype, 8.0)
+    want = turn(heads[:, :, K:], pos.cpu(), 80.0, rot, pairing)
+    assert float((qa[:, :, N:].double().cpu() - want).abs().max()) < (0.04 if dtype == torch.bfloat16 else 3e-3)
+
+
+@pytest.mark.parametrize("T", [1, 8, 9, 16, 24])
+def test_queries_of_a_product_left_unreduced(ops, T):
+    from turingserve_b200 import kernels
+    g = torch.Generator(device=DEV).manual_seed(T)
+    H, N, K, R, rank = 4, 128, 64, 32, 512
+    x = torch.randn(T, rank, generator=g, device=DEV).to(torch.bfloat16)
+    uq = (torch.randn(H * (K + R), rank, generator=g, device=DEV) * 0.05).to(torch.bfloat16)
+    w = (torch.randn(H, N, K, generator=g, device=DEV) * 0.1).to(torch.bfloat16)
+    pos, out = i32(list(range(5, 5 + T))), []
+    for defer in (False, True):
+        q = ops.linear(torch.empty(T, H * (K + R), dtype=torch.bfloat16, device=DEV), x, uq, may_defer=defer, lazy=False)
+        assert isinstance(q, kernels.Deferred) == defer
+        qa = torch.empty(T, H, N + R, dtype=torch.bfloat16, device=DEV)
+        ops.latent_queries(qa, q, w, pos, freqs(80.0, R), 1.0, R, "halves")
+        out.append(qa)
+    assert close(out[0], out[1], torch.bfloat16, 2.0) and float(out[0].abs().max()) > 0
+
+
+@pytest.mark.parametrize("T", [1, 8, 11, 16])
+@pytest.mark.parametrize("H,N,K", [(12, 128, 512), (3, 40, 256), (2, 9, 1032), (5, 33, 8)])
+def test_products_per_head_of_few_rows(ops, T, H, N, K):
+    """Strided rows in and out, the tensor-core instances with k whole and in four shares."""
+    g = torch.Generator(device=DEV).manual_seed(N)
+    x = torch.randn(T, H, K + 8, generator=g, device=DEV).to(torch.bfloat16)[:, :, :K]
+    w = (torch.randn(H, N, K, generator=g, device=DEV) * K ** -0.5).to(torch.bfloat16)
+    wide = torch.full((T, H, N + 2), 5.0, dtype=torch.bfloat16, device=DEV)
+    ops.batched_linear(wide[:, :, :N], x, w)
+    assert close(wide[:, :, :N], torch.einsum("thk,hnk->thn", x.double().cpu(), w.double().cpu()), torch.bfloat16, 8.0)
+    assert bool((wide[:, :, N:] == 5.0).all())
