@@ -46,18 +46,23 @@ def expected_logits(name, reqs):
 
 def check(got, expected, dtype):
     """float32: every logit within F32_REL of the request's largest, more at positions in the thousands (a 32-bit angle at
-    position p is off by about p 2^-23 radians).  bfloat16 (against the 64-bit plain model): the
-    root mean square of a position's differences within BF16_REL of the request's largest logit, and no single logit
-    further off than twice that."""
+    position p is off by about p 2^-23 radians).  bfloat16 (against the 64-bit plain model): the root mean square of a
+    position's differences within BF16_REL of the request's largest logit, and no single logit further off than twice that,
+    but for one position in twenty (or one): a router's close call that falls the other way after bfloat16 rounding."""
+    over, count = [], 0
     for rid, rows in got.items():
         top = float(np.abs(expected[rid]).max())
         for pos in sorted(rows):
             diff = rows[pos] - expected[rid][pos]
+            count += 1
             if dtype == "float32":
                 err, bound = float(np.abs(diff).max()), F32_REL * top * (1.0 + pos / 1000.0)
+                assert err <= bound, f"first wrong place (request, position, error / bound): {(rid, pos, err / bound)}"
             else:
                 err, bound = max(float(np.sqrt((diff ** 2).mean())), 0.5 * float(np.abs(diff).max())), BF16_REL * top
-            assert err <= bound, f"first wrong place (request, position, error / bound): {(rid, pos, err / bound)}"
+                if not err <= bound:
+                    over.append((rid, pos, err / bound))
+    assert len(over) <= max(1, count // 20), f"wrong places (request, position, error / bound), {len(over)} of {count}: {over[:5]}"
 
 
 def replay(folder, name, steps, dtype, graphs=(), portions=(), page=None):

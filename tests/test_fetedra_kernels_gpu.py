@@ -376,3 +376,167 @@ def test_products_per_head_of_few_rows(ops, T, H, N, K):
     ops.batched_linear(wide[:, :, :N], x, w)
     assert close(wide[:, :, :N], torch.einsum("thk,hnk->thn", x.double().cpu(), w.double().cpu()), torch.bfloat16, 8.0)
     assert bool((wide[:, :, N:] == 5.0).all())
+
+
+def run_attention(ops, q, rows, q_lens, page, rank, scale, window, sinks, gate):
+    """q [T, H, row]; rows: every request's cached rows up to its length; pages in a shuffled pool, those a window has passed
+    for every query given back (their entries name the null page)."""
+    rng = torch.Generator().manual_seed(len(rows))
+    n_pages = [-(-r.shape[0] // page) for r in rows]
+    order = (torch.randperm(sum(n_pages), generator=rng) + 1).tolist()
+    pool = torch.zeros(sum(n_pages) + 1, 1, page, q.shape[2], dtype=q.dtype, device=DEV)
+    bt = torch.zeros(len(rows), max(n_pages), dtype=torch.int32)
+    at, starts = 0, [0]
+    for r, (x, n) in enumerate(zip(rows, n_pages)):
+        mine = order[at:at + n]
+        at += n
+        bt[r, :n] = torch.tensor(mine)
+        for p, place in enumerate(mine):
+            part = x[p * page:(p + 1) * page]
+            pool[place, 0, :part.shape[0]] = part
+        if window:
+            bt[r, :max(0, x.shape[0] - q_lens[r] - window + 1) // page] = 0
+        starts.append(starts[-1] + q_lens[r])
+    lens = [x.shape[0] for x in rows]
+    step = SimpleNamespace(q_start=i32(starts), seq_lens=i32(lens), num_requests=len(rows), num_decode=sum(1 for n in q_lens if n == 1),
+                           max_q_len=max(q_lens), max_seq_len=max(lens))
+    out = torch.empty(q.shape[0], q.shape[1], rank, dtype=q.dtype, device=DEV)
+    ops.attention_biased(out, q, pool, None, bt.to(DEV), step, 1, page, scale, 0.0, None, window, sinks=sinks, gate=gate)
+    return out
+
+
+def plain_attention(q, rows, rank, scale, window, sinks, gate):
+    T, n, H = rows.shape[0], q.shape[0], q.shape[1]
+    ok = plain.visible(T, window)[T - n:]
+    k = rows.double().cpu()
+    out = []
+    for h in range(H):
+        p = plain.sink_softmax(q[:, h].double().cpu() @ k.T * scale, ok, sinks[h].double().cpu())
+        out.append(p @ k[:, :rank] * torch.sigmoid(gate[:, h].double().cpu())[:, None])
+    return torch.stack(out, 1)
+
+
+# (rank, rotated width): rows the tensor-core instances take (bfloat16) and others
+ROWS = pytest.mark.parametrize("dtype,H,rank,R,page", [
+    (torch.float32, 3, 28, 6, 16), (torch.bfloat16, 3, 28, 6, 16), (torch.bfloat16, 5, 96, 24, 64), (torch.bfloat16, 12, 256, 64, 64),
+    (torch.bfloat16, 28, 512, 64, 64), (torch.bfloat16, 40, 256, 64, 16), (torch.float32, 6, 256, 64, 64), (torch.bfloat16, 2, 512, 64, 8)])
+
+
+@ROWS
+@pytest.mark.parametrize("window", [None, 1, 30, 64, 100])
+@pytest.mark.parametrize("splits", [0, 3])
+def test_attention_in_batches_of_unequal_requests(ops, dtype, H, rank, R, page, window, splits):
+    """Single tokens and portions in one launch, windows that end inside, at and past tiles, sinks, gates in columns of a wider
+    tensor, pages that the window has passed given back."""
+    g = torch.Generator(device=DEV).manual_seed(H * rank + (window or 0))
+    q_lens, lens = [1, 1, 1, 1, 2, 40, 7], [1, 64, 333, 129, 71, 150, 7]
+    T, row = sum(q_lens), rank + R
+    q = (torch.randn(T, H, row, generator=g, device=DEV) * 1.5).to(dtype)
+    rows = [torch.randn(n, row, generator=g, device=DEV).to(dtype) for n in lens]
+    gate = torch.randn(T, H + 16, generator=g, device=DEV).to(dtype)[:, 8:8 + H]
+    sinks = torch.randn(H, generator=g, device=DEV) + 1.0
+    old = ops.biased_decode_splits
+    ops.biased_decode_splits = splits
+    try:
+        got = run_attention(ops, q, rows, q_lens, page, rank, row ** -0.5, window, sinks, gate)
+    finally:
+        ops.biased_decode_splits = old
+    at = 0
+    for r, n in enumerate(q_lens):
+        want = plain_attention(q[at:at + n], rows[r], rank, row ** -0.5, window, sinks, gate[at:at + n])
+        assert close(got[at:at + n], want, dtype, 4.0 if dtype == torch.bfloat16 else 30.0), (r, float((got[at:at + n].double().cpu() - want).abs().max()))
+        at += n
+
+
+@pytest.mark.parametrize("decode", [False, True])
+@ROWS
+def test_one_loud_key_at_every_edge(ops, decode, dtype, H, rank, R, page):
+    """Every key is silent but one, whose value is marked: the query finds it exactly where the window lets it, just inside and
+    just outside, at page borders, far away, and never ahead of itself; a sink takes half of what equals it."""
+    row, marked = rank + R, 3
+    sinks, gate_row = torch.full((H,), 20.0, device=DEV), 30.0
+    for T, window in ((330, 100), (150, 64), (321, 1), (90, 200), (700, None)):
+        n_q = 1 if decode else 24
+        i, w = T - 1, window or T
+        places = {i, i - 1, i - w + 1, i - w, i - w - 1, 0, 1, page - 1, page, (i // page) * page, (i // page) * page - 1, i // 2}
+        for j in sorted(p for p in places if 0 <= p <= i):
+            k = torch.zeros(T, row, dtype=dtype, device=DEV)
+            k[j, rank + 1] = 20.0
+            k[j, marked] = 1.0
+            q = torch.zeros(n_q, H, row, dtype=dtype, device=DEV)
+            q[:, :, rank + 1] = 1.0
+            gate = torch.full((n_q, H), gate_row, dtype=dtype, device=DEV)
+            out = run_attention(ops, q, [k], [n_q], page, rank, 1.0, window, sinks, gate)[:, H - 1, marked].tolist()
+            for at, value in enumerate(out):
+                p = T - n_q + at
+                seen = j <= p and p - j < w
+                assert abs(value - (0.5 if seen else 0.0)) < 1e-3, (T, window, j, p, value)
+
+
+# -- routing ------------------------------------------------------------------------------------------------------------------
+@DTYPES
+@pytest.mark.parametrize("E,top,groups,keep", [(16, 2, 2, 1), (12, 3, 4, 2), (6, 2, 6, 3), (9, 1, 3, 1), (5, 2, 1, 1), (64, 6, 8, 3), (8, 4, 2, 2),
+                                               (130, 5, 65, 7)])
+def test_grouped_routing(ops, dtype, E, top, groups, keep):
+    """Choices by scores with corrections (negative ones too), groups by their two largest; weights without the correction over
+    their sum, times a constant; the shared expert's weight beside them."""
+    g = torch.Generator(device=DEV).manual_seed(E + top)
+    T, K = 50, 72
+    x = torch.randn(T, K, generator=g, device=DEV).to(dtype)
+    w = torch.randn(E + 1, K, generator=g, device=DEV) * 0.2
+    corr = torch.randn(E, generator=g, device=DEV) * 0.3 - 0.6
+    idx, wts, share = torch.empty(T, top, dtype=torch.int32, device=DEV), torch.empty(T, top, device=DEV), torch.empty(T, device=DEV)
+    ops.router_topk(idx, wts, x, w, False, True, corr, groups, keep, 1.7, share)
+    s = torch.sigmoid(x.double().cpu() @ w.double().cpu().T)
+    assert float((share.double().cpu() - s[:, E]).abs().max()) < 1e-5
+    assert bool((s[:, :E] + corr.double().cpu() < 0).any())
+    right = 0
+    for t in range(T):
+        want = plain.choose(s[t, :E], corr.double().cpu(), top, groups, keep)
+        got = idx[t].tolist()
+        if got != want:                              # (two choice scores or two groups closer than 32-bit arithmetic tells apart)
+            continue
+        right += 1
+        picked = s[t, got]
+        assert float((wts[t].double().cpu() - picked / picked.sum() * 1.7).abs().max()) < 1e-5
+    assert right >= T - 1
+
+
+def test_a_kept_group_without_the_best_expert(ops):
+    """The single best expert lies in a group whose two largest add up to less: it must not be chosen; without a correction
+    vector the groups go by the scores."""
+    logit = lambda p: math.log(p / (1 - p))
+    scores = [0.95, 0.05, 0.1, 0.6, 0.7, 0.2]                      # groups of three: 0.95 + 0.1 against 0.7 + 0.6
+    w = torch.tensor([[logit(p)] for p in scores], device=DEV)
+    x = torch.ones(1, 1, device=DEV)
+    idx, wts = torch.empty(1, 2, dtype=torch.int32, device=DEV), torch.empty(1, 2, device=DEV)
+    ops.router_topk(idx, wts, x, w, False, True, None, 2, 1)
+    assert idx[0].tolist() == [4, 3] and torch.allclose(wts[0], torch.tensor([0.7, 0.6], device=DEV) / 1.3, atol=1e-6)
+    ops.router_topk(idx, wts, x, w, False, False, None, 2, 2, 3.0)
+    assert idx[0].tolist() == [0, 4] and torch.allclose(wts[0], torch.tensor([2.85, 2.1], device=DEV), atol=1e-5)
+
+
+@DTYPES
+@pytest.mark.parametrize("T", [1, 5, 30, 400])
+@pytest.mark.parametrize("W,E,top,ff,groups,shared", [(72, 12, 3, 24, (4, 2), (16, 0.5)), (64, 4, 4, 33, (1, 1), None), (128, 16, 2, 64, (8, 3), (96, 0.9))])
+def test_routed_feed_forward(ops, dtype, T, W, E, top, ff, groups, shared):
+    """The whole part against the plain one; many rows go to products of the experts' own."""
+    from turingserve_b200.config.model_config import RoutedMLPSpec
+    from turingserve_b200.parts.base import BuildContext, build
+    kw = dict(shared_intermediate_size=shared[0], shared_glu_limit=shared[1], shared_gate=True) if shared else {}
+    spec = RoutedMLPSpec(num_experts=E, top_k=top, intermediate_size=ff, activation="clamped_glu", gated=True, scoring="sigmoid", renormalize=True,
+                         weight_on="output", correction=True, groups=groups[0], groups_kept=groups[1], weight_scale=1.4, glu_limit=0.8, **kw)
+    part = build("feed_forward", spec, BuildContext(W, dtype, torch.device(DEV), 0))
+    g = torch.Generator(device=DEV).manual_seed(W)
+    t = {n: torch.randn(p.shape, generator=g, device=DEV) * (2.0 * p.shape[-1] ** -0.5) for n, p in part.parameters().items()}
+    t["correction"] = torch.randn(E, generator=g, device=DEV) * 0.2 - 0.5
+    t = {n: v.to(dtype) if part.parameters()[n].compute_dtype else v for n, v in t.items()}
+    part.load(t)
+    x = torch.randn(T, W, generator=g, device=DEV).to(dtype)
+    got = part.forward(x)
+    f = {"router": {"top": top, "scale": 1.4, "groups": {"count": groups[0], "keep": groups[1]}}, "expert": {"limit": 0.8},
+         "shared": {"limit": shared[1]} if shared else None}
+    want = plain.routed_ff(x.double().cpu(), {n: v.double().cpu() for n, v in t.items()}, "", f)
+    err = (got.double().cpu() - want).abs().amax(1)
+    bad = int((err > (0.03 if dtype == torch.bfloat16 else 1e-5) * float(want.abs().max())).sum())
+    assert bad <= T // 100, (bad, float(err.max()))                 # (two choice scores closer than 32-bit arithmetic tells apart)

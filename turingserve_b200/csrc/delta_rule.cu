@@ -365,8 +365,8 @@ TS_API int ts_head_gated_rmsnorm(void* out, const float* x, const void* gate, in
                                  float eps, int T, int H, int V, int dtype, void* stream) {
   if (T <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
-  // few tokens: the heads of a token spread over blocks of four warps; many: one block a token
-  const int heads_y = T >= 512 ? 1 : min(ceil_div(H, 4), 65535);
+  // the heads of a token spread over blocks of four warps; many tokens: two heads a warp
+  const int heads_y = min(ceil_div(H, T >= 512 ? 8 : 4), 65535);
   if (dtype == TS_F32)
     ts_launch(head_gated_rmsnorm_kernel<float>, dim3(T, heads_y), dim3(128), 0, s, (float*)out, x, (const float*)gate, gate_stride, w, w_stride, eps, H, V);
   else if (dtype == TS_BF16)

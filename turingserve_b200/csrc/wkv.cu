@@ -141,153 +141,224 @@ wkv_decay_kernel(float* out, const float* z, const T* __restrict__ w2, const flo
   }
 }
 
-// ---------------------------------------------------------------------------------------------------------------------
-// One block owns WK_COLS columns of one (head, request) state and keeps them in registers over the step's tokens: thread
-// (part, col) holds rows part * WK_ROWS .. of column col.  Tokens come in groups; a warp brings whole tokens (r, k, v as
-// stored, w in 32-bit) by cp.async while the group before is computed, turns its own tokens into 32-bit rows in shared memory
-// and sums r u k, the weight with which the token's own value enters its output.  Two block-wide barriers a group.
-constexpr int WK_GROUP = 16, WK_COLS = 16, WK_ROWS = 8;
+// The same on the tensor cores for bfloat16 weights: tanh(z) enters as two bfloat16 terms (hi + lo, two products a step), so it
+// carries 16 bits of mantissa; 32-bit accumulation.  Tiles of 64 tokens x 128 channels, 8 warps of 16 x 64; the whole rank sits
+// in shared memory.  The rank is a multiple of 8, at most DM_MAX_R.
+constexpr int DM_M = 64, DM_N = 128, DM_MAX_R = 256;
 
-template <typename T>
-__global__ void __launch_bounds__(512, 1)
+__global__ void __launch_bounds__(256)
+wkv_decay_mma_kernel(float* out, const float* z, const bf16* __restrict__ w2, const float* __restrict__ w0, int M, int N, int R) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) unsigned char dm_smem[];
+  const int Rp = (R + 15) / 16 * 16, stride = Rp + 8;
+  bf16* zh = reinterpret_cast<bf16*>(dm_smem);                        // [DM_M][stride]
+  bf16* zl = zh + DM_M * stride;
+  bf16* ws = zl + DM_M * stride;                                      // [DM_N][stride]
+  const int m0 = blockIdx.y * DM_M, n0 = blockIdx.x * DM_N;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int wm = (warp & 3) * 16, wn = (warp >> 2) * 64;
+  const int chunks = Rp / 8;
+  for (int i = threadIdx.x; i < DM_N * chunks; i += blockDim.x) {     // (weights: nobody's output)
+    const int row = i / chunks, c = (i % chunks) * 8;
+    const bool ok = n0 + row < N && c < R;
+    cp_async_16(ws + row * stride + c, ok ? w2 + (size_t)(n0 + row) * R + c : w2, ok);
+  }
+  cp_async_commit();
+  pdl_wait();
+  for (int i = threadIdx.x; i < DM_M * Rp; i += blockDim.x) {
+    const int row = i / Rp, c = i % Rp;
+    const float t = (m0 + row < M && c < R) ? tanhf(z[(size_t)(m0 + row) * R + c]) : 0.f;
+    const bf16 hi = __float2bfloat16_rn(t);
+    zh[row * stride + c] = hi;
+    zl[row * stride + c] = __float2bfloat16_rn(t - __bfloat162float(hi));
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  float acc[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  const int mat = lane >> 3, r8 = lane & 7;
+  for (int k0 = 0; k0 < Rp; k0 += 16) {
+    unsigned ah[4], al[4];
+    const int a_at = (wm + (mat & 1) * 8 + r8) * stride + k0 + (mat >> 1) * 8;
+    ldmatrix_x4(ah[0], ah[1], ah[2], ah[3], zh + a_at);
+    ldmatrix_x4(al[0], al[1], al[2], al[3], zl + a_at);
+#pragma unroll
+    for (int np = 0; np < 4; ++np) {
+      unsigned b0, b1, b2, b3;
+      ldmatrix_x4(b0, b1, b2, b3, ws + (wn + np * 16 + (mat >> 1) * 8 + r8) * stride + k0 + (mat & 1) * 8);
+      mma_bf16(acc[2 * np], ah, b0, b1);
+      mma_bf16(acc[2 * np], al, b0, b1);
+      mma_bf16(acc[2 * np + 1], ah, b2, b3);
+      mma_bf16(acc[2 * np + 1], al, b2, b3);
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int m = m0 + wm + (lane >> 2) + 8 * hh, c = n0 + wn + nt * 8 + (lane & 3) * 2;
+      if (m >= M) continue;
+      float* dst = out + (size_t)m * N + c;
+      if (c < N) dst[0] = expf(-expf(acc[nt][2 * hh] + w0[c]));
+      if (c + 1 < N) dst[1] = expf(-expf(acc[nt][2 * hh + 1] + w0[c + 1]));
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// A warp owns WK_COLS columns of one (head, request) state: lane l holds rows l * RPL .. of them in registers over the step's
+// tokens.  A block's WK_WARPS warps take neighbouring columns and share the staged rows: r, k and v as stored, w in 32-bit,
+// which a warp brings whole tokens of by cp.async, WK_STAGES - 1 groups of WK_GROUP tokens ahead; one block-wide barrier a
+// group.  Per token a lane adds its rows' share of (S + diag(u) k v^T)^T r and fades and writes its rows; the lanes' shares of
+// eight tokens are added through the warp's own piece of shared memory (lane l adds up the 32 shares of output l: token l / 4,
+// column l % 4, in lane order), so nothing crosses lanes inside a token.
+constexpr int WK_GROUP = 16, WK_COLS = 4, WK_WARPS = 4, WK_STAGES = 4, WK_BATCH = 8, WK_RED = 36;
+static_assert(WK_BATCH * WK_COLS == 32, "a lane adds up one output of a batch of tokens");
+
+template <typename T, int N>
+struct alignas(sizeof(T) * N) WkVec {
+  T v[N];
+};
+
+template <typename T, int RPL>
+__global__ void __launch_bounds__(WK_WARPS * 32, 1)
 wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, const float* __restrict__ u, const T* h_in,
                 float* state, size_t state_stride, const int* __restrict__ q_start, const int* __restrict__ slots, int H, int D,
-                int V, int hidden, int parts, int fast) {
+                int V, int hidden, int fast) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float smem[];
   const int h = blockIdx.y, b = blockIdx.z;
   const int t0 = q_start[b], n = q_start[b + 1] - t0;
   if (n <= 0) return;
-  const int Dp = parts * WK_ROWS;                          // D rounded up: rows beyond D hold zeros
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
-  const int col = threadIdx.x & (WK_COLS - 1), part = threadIdx.x / WK_COLS;
-  const int j = blockIdx.x * WK_COLS + col;
-  const int cols_here = min(WK_COLS, V - (int)blockIdx.x * WK_COLS);
-  const bool live = col < cols_here;
+  constexpr int Dp = 32 * RPL, BC = WK_COLS * WK_WARPS, PER = 16 / (int)sizeof(T);     // (rows beyond D hold zeros)
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int b0 = blockIdx.x * BC, c0 = b0 + warp * WK_COLS;            // the block's and this warp's first column
+  const int cols_here = min(BC, V - b0);
   float* base = state + (size_t)slots[b] * state_stride;
   float* S = base + (size_t)h * D * V;
-  float* r_s = smem;                                       // [WK_GROUP][Dp]
-  float* k_s = r_s + WK_GROUP * Dp;                        // [WK_GROUP][Dp]
-  float* w_s = k_s + WK_GROUP * Dp;                        // [2][WK_GROUP][Dp]
-  float* u_s = w_s + 2 * WK_GROUP * Dp;                    // [Dp]
-  float* v_s = u_s + Dp;                                   // [2][WK_GROUP][WK_COLS]
-  float* c_s = v_s + 2 * WK_GROUP * WK_COLS;               // [2][WK_GROUP]: the sum of r u k
-  float* o_s = c_s + 2 * WK_GROUP;                         // [WK_GROUP][parts][WK_COLS]
-  T* raw = reinterpret_cast<T*>(o_s + WK_GROUP * parts * WK_COLS);   // [2][WK_GROUP][D r | D k | WK_COLS v]
-  const int raw_row = 2 * D + WK_COLS;
+  float* w_s = smem;                                                   // [WK_STAGES][WK_GROUP][Dp]
+  float* red = w_s + WK_STAGES * WK_GROUP * Dp + warp * 32 * WK_RED;   // [32 outputs][WK_RED]: the lanes' shares
+  T* r_s = reinterpret_cast<T*>(w_s + WK_STAGES * WK_GROUP * Dp + WK_WARPS * 32 * WK_RED);   // [WK_STAGES][WK_GROUP][Dp]
+  T* k_s = r_s + WK_STAGES * WK_GROUP * Dp;
+  T* v_s = k_s + WK_STAGES * WK_GROUP * Dp;                            // [WK_STAGES][WK_GROUP][BC]
   const int HD = H * D, HV = H * V;
-  constexpr int PER = 16 / (int)sizeof(T);
 
-  float s[WK_ROWS];
+  float s[RPL][WK_COLS], uu[RPL];
 #pragma unroll
-  for (int i = 0; i < WK_ROWS; ++i) {
-    const int d = part * WK_ROWS + i;
-    s[i] = (live && d < D) ? S[(size_t)d * V + j] : 0.f;
+  for (int i = 0; i < RPL; ++i) {
+    const int d = lane * RPL + i;
+    uu[i] = d < D ? u[h * D + d] : 0.f;
+#pragma unroll
+    for (int j = 0; j < WK_COLS; ++j) s[i][j] = (d < D && c0 + j < V) ? S[(size_t)d * V + c0 + j] : 0.f;
   }
-  for (int i = threadIdx.x; i < 4 * WK_GROUP * Dp; i += blockDim.x) smem[i] = 0.f;
-  for (int i = threadIdx.x; i < Dp; i += blockDim.x) u_s[i] = i < D ? u[h * D + i] : 0.f;
+  for (int i = threadIdx.x; i < WK_STAGES * WK_GROUP * Dp; i += blockDim.x) {
+    w_s[i] = 0.f;
+    r_s[i] = from_f<T>(0.f);
+    k_s[i] = from_f<T>(0.f);
+  }
+  for (int i = threadIdx.x; i < WK_STAGES * WK_GROUP * BC; i += blockDim.x) v_s[i] = from_f<T>(0.f);
   __syncthreads();
 
-  auto fetch = [&](int g0, int buf) {
+  auto fetch = [&](int g0, int st) {
     const int gn = min(WK_GROUP, n - g0);
-    for (int q = warp; q < gn; q += nwarps) {
+    for (int q = warp; q < gn; q += WK_WARPS) {
       const size_t t = t0 + g0 + q;
       const T* rr = r + t * HD + h * D;
       const T* kr = k + t * HD + h * D;
-      const T* vr = v + t * HV + h * V + blockIdx.x * WK_COLS;
+      const T* vr = v + t * HV + h * V + b0;
       const float* wr = w + t * HD + h * D;
-      T* dst = raw + ((size_t)buf * WK_GROUP + q) * raw_row;
-      float* wd = w_s + ((size_t)buf * WK_GROUP + q) * Dp;
+      const int at = st * WK_GROUP + q;
       if (fast) {
         for (int c = lane * PER; c < D; c += 32 * PER) {
-          cp_async_16(dst + c, rr + c, true);
-          cp_async_16(dst + D + c, kr + c, true);
+          cp_async_16(r_s + at * Dp + c, rr + c, true);
+          cp_async_16(k_s + at * Dp + c, kr + c, true);
         }
-        for (int c = lane * 4; c < D; c += 128) cp_async_16(wd + c, wr + c, true);
-        if (lane * PER < cols_here) cp_async_16(dst + 2 * D + lane * PER, vr + lane * PER, true);
+        for (int c = lane * 4; c < D; c += 128) cp_async_16(w_s + at * Dp + c, wr + c, true);
+        if (lane * PER < cols_here) cp_async_16(v_s + at * BC + lane * PER, vr + lane * PER, true);
       } else {
         for (int c = lane; c < D; c += 32) {
-          dst[c] = rr[c];
-          dst[D + c] = kr[c];
-          wk_cp_async_4(wd + c, wr + c);
+          r_s[at * Dp + c] = rr[c];
+          k_s[at * Dp + c] = kr[c];
+          wk_cp_async_4(w_s + at * Dp + c, wr + c);
         }
-        for (int c = lane; c < cols_here; c += 32) dst[2 * D + c] = vr[c];
+        for (int c = lane; c < cols_here; c += 32) v_s[at * BC + c] = vr[c];
       }
     }
   };
-  fetch(0, 0);
-  cp_async_commit();
-  int buf = 0;
-  for (int g0 = 0; g0 < n; g0 += WK_GROUP, buf ^= 1) {
-    const int gn = min(WK_GROUP, n - g0);
-    if (g0 + WK_GROUP < n) fetch(g0 + WK_GROUP, buf ^ 1);
-    cp_async_commit();
-    cp_async_wait<1>();
-    __syncwarp();                                          // (a warp turns the tokens that it brought itself)
-    float* vg = v_s + buf * WK_GROUP * WK_COLS;
-    float* cg = c_s + buf * WK_GROUP;
-    for (int q = warp; q < gn; q += nwarps) {
-      const T* src = raw + ((size_t)buf * WK_GROUP + q) * raw_row;
-      float c = 0.f;
-      if (fast) {                                          // (D is even then)
-        for (int d = 2 * lane; d < D; d += 64) {
-          const float r0 = to_f(src[d]), r1 = to_f(src[d + 1]), k0 = to_f(src[D + d]), k1 = to_f(src[D + d + 1]);
-          *reinterpret_cast<float2*>(r_s + q * Dp + d) = make_float2(r0, r1);
-          *reinterpret_cast<float2*>(k_s + q * Dp + d) = make_float2(k0, k1);
-          const float2 uu = *reinterpret_cast<const float2*>(u_s + d);
-          c = fmaf(r0 * uu.x, k0, c);
-          c = fmaf(r1 * uu.y, k1, c);
-        }
-      } else {
-        for (int d = lane; d < D; d += 32) {
-          const float r0 = to_f(src[d]), k0 = to_f(src[D + d]);
-          r_s[q * Dp + d] = r0;
-          k_s[q * Dp + d] = k0;
-          c = fmaf(r0 * u_s[d], k0, c);
-        }
-      }
-      if (lane < WK_COLS) vg[q * WK_COLS + lane] = lane < cols_here ? to_f(src[2 * D + lane]) : 0.f;
-      c = warp_sum(c);
-      if (lane == 0) cg[q] = c;
-    }
-    __syncthreads();                                       // the group is ready; the sums of the one before are out
-    const float* wg = w_s + (size_t)buf * WK_GROUP * Dp;
-#pragma unroll 4
-    for (int q = 0; q < gn; ++q) {
-      const float vj = vg[q * WK_COLS + col];
-      const float4* rr = reinterpret_cast<const float4*>(r_s + q * Dp + part * WK_ROWS);
-      const float4* kr = reinterpret_cast<const float4*>(k_s + q * Dp + part * WK_ROWS);
-      const float4* wr = reinterpret_cast<const float4*>(wg + q * Dp + part * WK_ROWS);
-      float o = 0.f, o2 = 0.f;
 #pragma unroll
-      for (int i = 0; i < WK_ROWS / 4; ++i) {
-        const float4 r4 = rr[i], k4 = kr[i], w4 = wr[i];
-        o = fmaf(s[4 * i + 0], r4.x, o);
-        o2 = fmaf(s[4 * i + 1], r4.y, o2);
-        o = fmaf(s[4 * i + 2], r4.z, o);
-        o2 = fmaf(s[4 * i + 3], r4.w, o2);
-        s[4 * i + 0] = fmaf(w4.x, s[4 * i + 0], k4.x * vj);
-        s[4 * i + 1] = fmaf(w4.y, s[4 * i + 1], k4.y * vj);
-        s[4 * i + 2] = fmaf(w4.z, s[4 * i + 2], k4.z * vj);
-        s[4 * i + 3] = fmaf(w4.w, s[4 * i + 3], k4.w * vj);
+  for (int st = 0; st < WK_STAGES - 1; ++st) {
+    if (st * WK_GROUP < n) fetch(st * WK_GROUP, st);
+    cp_async_commit();
+  }
+  int st = 0;
+  for (int g0 = 0; g0 < n; g0 += WK_GROUP, st = (st + 1) % WK_STAGES) {
+    const int gn = min(WK_GROUP, n - g0);
+    cp_async_wait<WK_STAGES - 2>();
+    __syncthreads();                                       // this group is here for all; the one before it is used up
+    if (g0 + (WK_STAGES - 1) * WK_GROUP < n) fetch(g0 + (WK_STAGES - 1) * WK_GROUP, (st + WK_STAGES - 1) % WK_STAGES);
+    cp_async_commit();
+#pragma unroll 1
+    for (int q0 = 0; q0 < gn; q0 += WK_BATCH) {
+      float o[WK_BATCH][WK_COLS];
+#pragma unroll
+      for (int q = 0; q < WK_BATCH; ++q) {
+#pragma unroll
+        for (int j = 0; j < WK_COLS; ++j) o[q][j] = 0.f;
+        if (q0 + q < gn) {
+          const int at = st * WK_GROUP + q0 + q;
+          const WkVec<T, RPL> r4 = *reinterpret_cast<const WkVec<T, RPL>*>(r_s + at * Dp + lane * RPL);
+          const WkVec<T, RPL> k4 = *reinterpret_cast<const WkVec<T, RPL>*>(k_s + at * Dp + lane * RPL);
+          float w4[RPL], vf[WK_COLS];
+          if constexpr (RPL >= 4) {
+#pragma unroll
+            for (int i = 0; i < RPL; i += 4) *reinterpret_cast<float4*>(w4 + i) = *reinterpret_cast<const float4*>(w_s + at * Dp + lane * RPL + i);
+          } else if constexpr (RPL == 2) {
+            *reinterpret_cast<float2*>(w4) = *reinterpret_cast<const float2*>(w_s + at * Dp + lane * 2);
+          } else {
+            w4[0] = w_s[at * Dp + lane];
+          }
+          const WkVec<T, WK_COLS> v4 = *reinterpret_cast<const WkVec<T, WK_COLS>*>(v_s + at * BC + warp * WK_COLS);
+#pragma unroll
+          for (int j = 0; j < WK_COLS; ++j) vf[j] = to_f(v4.v[j]);
+          float c = 0.f;                                   // this lane's part of the sum of r u k
+#pragma unroll
+          for (int i = 0; i < RPL; ++i) {
+            const float rf = to_f(r4.v[i]), kf = to_f(k4.v[i]);
+            c = fmaf(rf, uu[i] * kf, c);
+#pragma unroll
+            for (int j = 0; j < WK_COLS; ++j) {
+              o[q][j] = fmaf(s[i][j], rf, o[q][j]);
+              s[i][j] = fmaf(w4[i], s[i][j], kf * vf[j]);
+            }
+          }
+#pragma unroll
+          for (int j = 0; j < WK_COLS; ++j) o[q][j] = fmaf(c, vf[j], o[q][j]);
+        }
       }
-      o_s[(q * parts + part) * WK_COLS + col] = o + o2;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < gn * WK_COLS; i += blockDim.x) {
-      const int q = i / WK_COLS, c = i % WK_COLS;
-      if (c >= cols_here) continue;
-      float o = cg[q] * vg[i];
-      for (int p = 0; p < parts; ++p) o += o_s[(q * parts + p) * WK_COLS + c];
-      out[(size_t)(t0 + g0 + q) * HV + h * V + blockIdx.x * WK_COLS + c] = o;
+      __syncwarp();                                        // (the batch before has been added up)
+#pragma unroll
+      for (int q = 0; q < WK_BATCH; ++q)
+#pragma unroll
+        for (int j = 0; j < WK_COLS; ++j) red[(q * WK_COLS + j) * WK_RED + lane] = o[q][j];
+      __syncwarp();
+      float total = 0.f;
+#pragma unroll
+      for (int i = 0; i < 32; i += 4) {
+        const float4 p = *reinterpret_cast<const float4*>(red + lane * WK_RED + i);
+        total += (p.x + p.y) + (p.z + p.w);
+      }
+      const int q = q0 + lane / WK_COLS, c = c0 + lane % WK_COLS;
+      if (q < gn && c < V) out[(size_t)(t0 + g0 + q) * HV + h * V + c] = total;
     }
   }
   cp_async_wait<0>();
 #pragma unroll
-  for (int i = 0; i < WK_ROWS; ++i) {
-    const int d = part * WK_ROWS + i;
-    if (live && d < D) S[(size_t)d * V + j] = s[i];
+  for (int i = 0; i < RPL; ++i) {
+    const int d = lane * RPL + i;
+#pragma unroll
+    for (int j = 0; j < WK_COLS; ++j)
+      if (d < D && c0 + j < V) S[(size_t)d * V + c0 + j] = s[i][j];
   }
   // the request's last input, for its next token; every block of the request takes a share of the channels
   float* prev = base + (size_t)H * D * V;
@@ -298,31 +369,33 @@ wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, 
 
 // ---------------------------------------------------------------------------------------------------------------------
 // Single tokens (bfloat16): out[s, m, :] = W[s] mix_s(m) for the s < n stacked matrices [n, N, K], and z[m, :] = w1 mix_n(m) in
-// 32-bit.  A block takes 64 columns of one matrix: it puts the first weights of its 16 warps on their way (they are nobody's
-// output), then makes its mix of all rows in shared memory and multiplies on the tensor cores; two warps share 8 columns,
-// each half of k.  (The products' k index is a permutation of the real one, the same for both operands.)
-constexpr int PJ_WARPS = 16, PJ_COLS = 64, PJ_UNROLL = 8, PJ_PAD = 32;
+// 32-bit.  A block takes 64 columns of one matrix: it puts the first weights of its warps on their way (they are nobody's
+// output), then makes its mix of all rows in shared memory and multiplies on the tensor cores.  KS = 2: two warps share 8 columns, each
+// half of k (launches of one wave); KS = 1: a warp takes the whole of k, two blocks an SM.  (The products' k index is a
+// permutation of the real one, the same for both operands.)
+constexpr int PJ_COLS = 64, PJ_UNROLL = 8, PJ_PAD = 32;
 
-template <int ROWS>
-__global__ void __launch_bounds__(PJ_WARPS * 32)
+template <int ROWS, int KS>
+__global__ void __launch_bounds__(PJ_COLS / 8 * KS * 32)
 wkv_project_kernel(bf16* out, float* z, const bf16* h, const bf16* __restrict__ mu, const bf16* __restrict__ w,
                    const bf16* __restrict__ w1, const float* state,
                    size_t state_stride, size_t prev_off, const int* __restrict__ slots, int M, int n, int N, int R, int K) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char pj_smem[];
   bf16* x_s = reinterpret_cast<bf16*>(pj_smem);                       // [ROWS][K + PJ_PAD]
-  __shared__ float red[PJ_WARPS / 2][ROWS][8];
+  constexpr int THREADS = PJ_COLS / 8 * KS * 32;
+  __shared__ float red[PJ_COLS / 8][ROWS][8];
   const int xs = K + PJ_PAD;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
   const int per = (N + PJ_COLS - 1) / PJ_COLS;
   const int s = min((int)blockIdx.x / per, n);                        // which mix; n: the decay's
   const int n_cols = s < n ? N : R;
-  const int n0 = ((int)blockIdx.x - s * per) * PJ_COLS + (warp >> 1) * 8;
+  const int n0 = ((int)blockIdx.x - s * per) * PJ_COLS + warp / KS * 8;
   const bool n_ok = n0 + g < n_cols;
   const bf16* mat = s < n ? w + (size_t)s * N * K : w1;
-  const int steps = (K + 31) / 32, half = (steps + 1) / 2;
-  const int st0 = (warp & 1) * half, st1 = min(st0 + half, steps);
+  const int steps = (K + 31) / 32, share = (steps + KS - 1) / KS;
+  const int st0 = warp % KS * share, st1 = min(st0 + share, steps);
   const bf16* wrow = mat + (size_t)(n_ok ? n0 + g : 0) * K + t * 8;
   uint4 wv[2][PJ_UNROLL];
   auto fetch = [&](int st, int bf) {
@@ -335,7 +408,7 @@ wkv_project_kernel(bf16* out, float* z, const bf16* h, const bf16* __restrict__ 
   fetch(st0, 0);
   if constexpr (ROWS == 8) fetch(st0 + PJ_UNROLL, 1);
   pdl_wait();
-  for (int i = threadIdx.x * 8; i < ROWS * K; i += PJ_WARPS * 32 * 8) {
+  for (int i = threadIdx.x * 8; i < ROWS * K; i += THREADS * 8) {
     const int m = i / K, c = i - m * K;
     uint4 o = make_uint4(0u, 0u, 0u, 0u);
     if (m < M) {
@@ -387,22 +460,24 @@ wkv_project_kernel(bf16* out, float* z, const bf16* h, const bf16* __restrict__ 
     }
   }
   // (lane (g, t) holds rows g and g + 8 of columns 2 t and 2 t + 1)
-  if (warp & 1) {
+  if constexpr (KS == 2) {
+    if (warp & 1) {
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      red[warp >> 1][g][2 * t + e] = acc[e];
-      if constexpr (ROWS == 16) red[warp >> 1][g + 8][2 * t + e] = acc[2 + e];
+      for (int e = 0; e < 2; ++e) {
+        red[warp >> 1][g][2 * t + e] = acc[e];
+        if constexpr (ROWS == 16) red[warp >> 1][g + 8][2 * t + e] = acc[2 + e];
+      }
     }
+    __syncthreads();
+    if (warp & 1) return;
   }
-  __syncthreads();
-  if (warp & 1) return;
 #pragma unroll
   for (int hh = 0; hh < ROWS / 8; ++hh)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int m = g + 8 * hh, c = n0 + 2 * t + e;
       if (m >= M || c >= n_cols) continue;
-      const float val = acc[2 * hh + e] + red[warp >> 1][m][2 * t + e];
+      const float val = KS == 2 ? acc[2 * hh + e] + red[warp >> 1][m][2 * t + e] : acc[2 * hh + e];
       if (s < n) out[((size_t)s * M + m) * N + c] = from_f<bf16>(val);
       else z[(size_t)m * R + c] = val;
     }
@@ -544,6 +619,17 @@ TS_API int ts_wkv_decay(float* out, const float* z, const void* w2, const float*
   const dim3 grid(ceil_div(N, DC_N), ceil_div(T, DC_M));
   if (grid.y > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_decay: %d tokens", T);
   cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == TS_BF16 && R % 8 == 0 && R <= DM_MAX_R && !((uintptr_t)w2 & 15)) {
+    const size_t smem = (size_t)(2 * DM_M + DM_N) * ((R + 15) / 16 * 16 + 8) * 2;
+    static size_t configured = 0;
+    if (smem > 48 * 1024 && smem > configured) {
+      cudaError_t e = cudaFuncSetAttribute(wkv_decay_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_decay: shared memory %zu: %s", smem, cudaGetErrorString(e));
+      configured = smem;
+    }
+    ts_launch(wkv_decay_mma_kernel, dim3(ceil_div(N, DM_N), ceil_div(T, DM_M)), dim3(256), smem, s, out, z, (const bf16*)w2, w0, T, N, R);
+    TS_LAUNCH_CHECK();
+  }
   if (dtype == TS_F32) ts_launch(wkv_decay_kernel<float>, grid, dim3(256), 0, s, out, z, (const float*)w2, w0, T, N, R);
   else if (dtype == TS_BF16) ts_launch(wkv_decay_kernel<bf16>, grid, dim3(256), 0, s, out, z, (const bf16*)w2, w0, T, N, R);
   else TS_REFUSE(TS_ERR_DTYPE, "ts_wkv_decay: dtype %d", dtype);
@@ -560,36 +646,42 @@ TS_API int ts_wkv_scan(float* out, const void* r, const void* k, const void* v, 
                        int hidden, int longest, int dtype, void* stream) {
   if (B <= 0) return 0;
   if (H <= 0 || D <= 0 || V <= 0) TS_REFUSE(TS_ERR_SHAPE, "ts_wkv_scan: %d heads of %d x %d", H, D, V);
-  const int parts = ceil_div(ceil_div(D, WK_ROWS), 2) * 2;            // (whole warps)
-  if (parts * WK_COLS > 512) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_scan: keys of %d (limit %d)", D, 512 / WK_COLS * WK_ROWS);
+  if (D > 256) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_scan: keys of %d (limit 256)", D);
   if (B > 65535 || H > 65535) TS_REFUSE(TS_ERR_LIMIT, "ts_wkv_scan: %d requests / %d heads per launch", B, H);
   cudaStream_t s = (cudaStream_t)stream;
   const int elem = dtype == TS_F32 ? 4 : 2, per = 16 / elem;
   const int fast = D % per == 0 && V % per == 0 && D % 4 == 0 &&
                    !(((uintptr_t)r | (uintptr_t)k | (uintptr_t)v | (uintptr_t)w) & 15);
-  const int Dp = parts * WK_ROWS;
-  const size_t smem = sizeof(float) * ((size_t)4 * WK_GROUP * Dp + Dp + 2 * WK_GROUP * (WK_COLS + 1) + (size_t)WK_GROUP * parts * WK_COLS) +
-                      (size_t)2 * WK_GROUP * (2 * D + WK_COLS) * elem;
-  const dim3 grid(ceil_div(V, WK_COLS), H, B);
-#define TS_WK(TT)                                                                                                       \
-  do {                                                                                                                  \
-    static size_t configured = 0;                                                                                       \
-    if (smem > 48 * 1024 && smem > configured) {                                                                        \
-      cudaError_t e = cudaFuncSetAttribute(wkv_scan_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-      if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_scan: shared memory %zu: %s", smem, cudaGetErrorString(e));       \
-      configured = smem;                                                                                                \
-    }                                                                                                                   \
-    if (longest >= WK_LATE_TOKENS)                                                                                      \
-      ts_launch_late(wkv_scan_kernel<TT>, grid, dim3(parts * WK_COLS), smem, s, out, (const TT*)r, (const TT*)k, (const TT*)v, w, u, \
-                     (const TT*)h_in, state, (size_t)state_stride, q_start, slots, H, D, V, hidden, parts, fast);       \
-    else                                                                                                                \
-      ts_launch(wkv_scan_kernel<TT>, grid, dim3(parts * WK_COLS), smem, s, out, (const TT*)r, (const TT*)k, (const TT*)v, w, u, \
-                (const TT*)h_in, state, (size_t)state_stride, q_start, slots, H, D, V, hidden, parts, fast);            \
+  const dim3 grid(ceil_div(V, WK_COLS * WK_WARPS), H, B);
+#define TS_WKR(TT, RPL)                                                                                                  \
+  do {                                                                                                                   \
+    const size_t smem = (size_t)WK_STAGES * WK_GROUP * (32 * RPL * (sizeof(float) + 2 * sizeof(TT)) + WK_COLS * WK_WARPS * sizeof(TT)) + \
+                        sizeof(float) * WK_WARPS * 32 * WK_RED;                                                          \
+    static bool configured = false;                                                                                      \
+    if (!configured) {                                                                                                   \
+      cudaError_t e = cudaFuncSetAttribute(wkv_scan_kernel<TT, RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_scan: shared memory %zu: %s", smem, cudaGetErrorString(e));        \
+      configured = true;                                                                                                 \
+    }                                                                                                                    \
+    if (longest >= WK_LATE_TOKENS)                                                                                       \
+      ts_launch_late(wkv_scan_kernel<TT, RPL>, grid, dim3(WK_WARPS * 32), smem, s, out, (const TT*)r, (const TT*)k, (const TT*)v, w, u, \
+                     (const TT*)h_in, state, (size_t)state_stride, q_start, slots, H, D, V, hidden, fast);               \
+    else                                                                                                                 \
+      ts_launch(wkv_scan_kernel<TT, RPL>, grid, dim3(WK_WARPS * 32), smem, s, out, (const TT*)r, (const TT*)k, (const TT*)v, w, u, \
+                (const TT*)h_in, state, (size_t)state_stride, q_start, slots, H, D, V, hidden, fast);                    \
+  } while (0)
+#define TS_WK(TT)                  \
+  do {                             \
+    if (D <= 32) TS_WKR(TT, 1);    \
+    else if (D <= 64) TS_WKR(TT, 2);  \
+    else if (D <= 128) TS_WKR(TT, 4); \
+    else TS_WKR(TT, 8);            \
   } while (0)
   if (dtype == TS_F32) TS_WK(float);
   else if (dtype == TS_BF16) TS_WK(bf16);
   else TS_REFUSE(TS_ERR_DTYPE, "ts_wkv_scan: dtype %d", dtype);
 #undef TS_WK
+#undef TS_WKR
   TS_LAUNCH_CHECK();
 }
 
@@ -606,20 +698,21 @@ TS_API int ts_wkv_project(void* out, float* z, const void* h, const void* mu, co
     TS_REFUSE(TS_ERR_UNSUPPORTED, "ts_wkv_project: %d tokens, rows of %d", M, K);
   const dim3 grid(n * ceil_div(N, PJ_COLS) + ceil_div(R, PJ_COLS));
   cudaStream_t s = (cudaStream_t)stream;
-#define TS_PJ(ROWS)                                                                                                      \
+#define TS_PJ(ROWS, KS)                                                                                                  \
   do {                                                                                                                   \
-    const size_t smem = (size_t)ROWS * (K + PJ_PAD) * 2;                                                                      \
+    const size_t smem = (size_t)ROWS * (K + PJ_PAD) * 2;                                                                 \
     static size_t configured = 0;                                                                                        \
     if (smem > 40 * 1024 && smem > configured) {                                                                         \
-      cudaError_t e = cudaFuncSetAttribute(wkv_project_kernel<ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      cudaError_t e = cudaFuncSetAttribute(wkv_project_kernel<ROWS, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_project: shared memory %zu: %s", smem, cudaGetErrorString(e));     \
       configured = smem;                                                                                                 \
     }                                                                                                                    \
-    ts_launch(wkv_project_kernel<ROWS>, grid, dim3(PJ_WARPS * 32), smem, s, (bf16*)out, z, (const bf16*)h, (const bf16*)mu, \
+    ts_launch(wkv_project_kernel<ROWS, KS>, grid, dim3(PJ_COLS / 8 * KS * 32), smem, s, (bf16*)out, z, (const bf16*)h, (const bf16*)mu, \
               (const bf16*)w, (const bf16*)w1, state, (size_t)state_stride, (size_t)prev_off, slots, M, n, N, R, K);     \
   } while (0)
-  if (M <= 8) TS_PJ(8);
-  else TS_PJ(16);
+  const bool one_wave = grid.x <= 148;
+  if (M <= 8) { if (one_wave) TS_PJ(8, 2); else TS_PJ(8, 1); }
+  else { if (one_wave) TS_PJ(16, 2); else TS_PJ(16, 1); }
 #undef TS_PJ
   TS_LAUNCH_CHECK();
 }
