@@ -24,7 +24,7 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 # (windows are passed in prompts and by decoded tokens: A 7 and 21, B 40, C 70, D 1)
 LENGTHS = {"A": [5, 18, 34, 70, 41, 64], "B": [1, 9, 41, 70, 97, 33], "C": [2, 129, 201, 70, 257, 64], "D": [4, 40, 22, 70, 33, 8]}
 F32_REL = 3e-5          # of the largest expected logit of the request
-BF16_REL = 3e-2
+BF16_REL, BF16_MEDIAN = 5e-2, 1e-2
 
 
 def requests_for(name, folder):
@@ -48,8 +48,9 @@ def check(got, expected, dtype):
     """float32: every logit within F32_REL of the request's largest, more at positions in the thousands (a 32-bit angle at
     position p is off by about p 2^-23 radians).  bfloat16 (against the 64-bit plain model): the root mean square of a
     position's differences within BF16_REL of the request's largest logit, and no single logit further off than twice that,
-    but for one position in twenty (or one): a router's close call that falls the other way after bfloat16 rounding."""
-    over, count = [], 0
+    but for one position in twenty (or one): a router's close call that falls the other way after bfloat16 rounding; half the
+    positions within BF16_MEDIAN."""
+    over, count, ratios = [], 0, []
     for rid, rows in got.items():
         top = float(np.abs(expected[rid]).max())
         for pos in sorted(rows):
@@ -60,9 +61,11 @@ def check(got, expected, dtype):
                 assert err <= bound, f"first wrong place (request, position, error / bound): {(rid, pos, err / bound)}"
             else:
                 err, bound = max(float(np.sqrt((diff ** 2).mean())), 0.5 * float(np.abs(diff).max())), BF16_REL * top
+                ratios.append(err / top)
                 if not err <= bound:
                     over.append((rid, pos, err / bound))
     assert len(over) <= max(1, count // 20), f"wrong places (request, position, error / bound), {len(over)} of {count}: {over[:5]}"
+    assert count < 40 or dtype == "float32" or float(np.median(ratios)) <= BF16_MEDIAN
 
 
 def replay(folder, name, steps, dtype, graphs=(), portions=(), page=None):

@@ -208,12 +208,13 @@ wkv_decay_mma_kernel(float* out, const float* z, const bf16* __restrict__ w2, co
 // ---------------------------------------------------------------------------------------------------------------------
 // A warp owns WK_COLS columns of one (head, request) state: lane l holds rows l * RPL .. of them in registers over the step's
 // tokens.  A block's WK_WARPS warps take neighbouring columns and share the staged rows: r, k and v as stored, w in 32-bit,
-// which a warp brings whole tokens of by cp.async, WK_STAGES - 1 groups of WK_GROUP tokens ahead; one block-wide barrier a
-// group.  Per token a lane adds its rows' share of (S + diag(u) k v^T)^T r and fades and writes its rows; the lanes' shares of
-// eight tokens are added through the warp's own piece of shared memory (lane l adds up the 32 shares of output l: token l / 4,
-// column l % 4, in lane order), so nothing crosses lanes inside a token.
-constexpr int WK_GROUP = 16, WK_COLS = 4, WK_WARPS = 4, WK_STAGES = 4, WK_BATCH = 8, WK_RED = 36;
-static_assert(WK_BATCH * WK_COLS == 32, "a lane adds up one output of a batch of tokens");
+// which a warp brings whole tokens of by cp.async, two or three groups of WK_GROUP tokens ahead; one block-wide barrier a group.  Per token a lane adds its rows' share of (S + diag(u) k v^T)^T r and fades and writes its rows; the lanes' shares of
+// a group are added through the warp's own piece of shared memory (lane l adds up the 32 shares of output l: token l / 2,
+// column l % 2, in lane order), so nothing crosses lanes inside a token.  Few columns a warp mean many warps a scheduler: one
+// warp alone issues an instruction every three or four cycles.
+constexpr int WK_GROUP = 16, WK_COLS = 2, WK_WARPS = 8, WK_RED = 36;
+static_assert(WK_GROUP * WK_COLS == 32, "a lane adds up one output of a group of tokens");
+template <typename T, int RPL> constexpr int wk_stages() { return RPL * (int)sizeof(T) >= 32 ? 3 : 4; }
 
 template <typename T, int N>
 struct alignas(sizeof(T) * N) WkVec {
@@ -231,7 +232,7 @@ wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, 
   const int h = blockIdx.y, b = blockIdx.z;
   const int t0 = q_start[b], n = q_start[b + 1] - t0;
   if (n <= 0) return;
-  constexpr int Dp = 32 * RPL, BC = WK_COLS * WK_WARPS, PER = 16 / (int)sizeof(T);     // (rows beyond D hold zeros)
+  constexpr int WK_STAGES = wk_stages<T, RPL>(), Dp = 32 * RPL, BC = WK_COLS * WK_WARPS, PER = 16 / (int)sizeof(T);     // (rows beyond D hold zeros)
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int b0 = blockIdx.x * BC, c0 = b0 + warp * WK_COLS;            // the block's and this warp's first column
   const int cols_here = min(BC, V - b0);
@@ -298,59 +299,60 @@ wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, 
     __syncthreads();                                       // this group is here for all; the one before it is used up
     if (g0 + (WK_STAGES - 1) * WK_GROUP < n) fetch(g0 + (WK_STAGES - 1) * WK_GROUP, (st + WK_STAGES - 1) % WK_STAGES);
     cp_async_commit();
-#pragma unroll 1
-    for (int q0 = 0; q0 < gn; q0 += WK_BATCH) {
-      float o[WK_BATCH][WK_COLS];
+    float o[WK_GROUP][WK_COLS];
+    const T* r_l = r_s + st * WK_GROUP * Dp + lane * RPL;
+    const T* k_l = k_s + st * WK_GROUP * Dp + lane * RPL;
+    const float* w_l = w_s + st * WK_GROUP * Dp + lane * RPL;
+    const T* v_l = v_s + st * WK_GROUP * BC + warp * WK_COLS;
+    auto token = [&](int q, float (&oq)[WK_COLS]) {
+      const WkVec<T, RPL> rq = *reinterpret_cast<const WkVec<T, RPL>*>(r_l + q * Dp);
+      const WkVec<T, RPL> kq = *reinterpret_cast<const WkVec<T, RPL>*>(k_l + q * Dp);
+      const WkVec<float, RPL> wq = *reinterpret_cast<const WkVec<float, RPL>*>(w_l + q * Dp);
+      const WkVec<T, WK_COLS> vq = *reinterpret_cast<const WkVec<T, WK_COLS>*>(v_l + q * BC);
+      float c = 0.f, vf[WK_COLS];                          // c: this lane's part of the sum of r u k
 #pragma unroll
-      for (int q = 0; q < WK_BATCH; ++q) {
+      for (int j = 0; j < WK_COLS; ++j) {
+        vf[j] = to_f(vq.v[j]);
+        oq[j] = 0.f;
+      }
 #pragma unroll
-        for (int j = 0; j < WK_COLS; ++j) o[q][j] = 0.f;
-        if (q0 + q < gn) {
-          const int at = st * WK_GROUP + q0 + q;
-          const WkVec<T, RPL> r4 = *reinterpret_cast<const WkVec<T, RPL>*>(r_s + at * Dp + lane * RPL);
-          const WkVec<T, RPL> k4 = *reinterpret_cast<const WkVec<T, RPL>*>(k_s + at * Dp + lane * RPL);
-          float w4[RPL], vf[WK_COLS];
-          if constexpr (RPL >= 4) {
+      for (int i = 0; i < RPL; ++i) {
+        const float rf = to_f(rq.v[i]), kf = to_f(kq.v[i]);
+        c = fmaf(rf, uu[i] * kf, c);
 #pragma unroll
-            for (int i = 0; i < RPL; i += 4) *reinterpret_cast<float4*>(w4 + i) = *reinterpret_cast<const float4*>(w_s + at * Dp + lane * RPL + i);
-          } else if constexpr (RPL == 2) {
-            *reinterpret_cast<float2*>(w4) = *reinterpret_cast<const float2*>(w_s + at * Dp + lane * 2);
-          } else {
-            w4[0] = w_s[at * Dp + lane];
-          }
-          const WkVec<T, WK_COLS> v4 = *reinterpret_cast<const WkVec<T, WK_COLS>*>(v_s + at * BC + warp * WK_COLS);
-#pragma unroll
-          for (int j = 0; j < WK_COLS; ++j) vf[j] = to_f(v4.v[j]);
-          float c = 0.f;                                   // this lane's part of the sum of r u k
-#pragma unroll
-          for (int i = 0; i < RPL; ++i) {
-            const float rf = to_f(r4.v[i]), kf = to_f(k4.v[i]);
-            c = fmaf(rf, uu[i] * kf, c);
-#pragma unroll
-            for (int j = 0; j < WK_COLS; ++j) {
-              o[q][j] = fmaf(s[i][j], rf, o[q][j]);
-              s[i][j] = fmaf(w4[i], s[i][j], kf * vf[j]);
-            }
-          }
-#pragma unroll
-          for (int j = 0; j < WK_COLS; ++j) o[q][j] = fmaf(c, vf[j], o[q][j]);
+        for (int j = 0; j < WK_COLS; ++j) {
+          oq[j] = fmaf(s[i][j], rf, oq[j]);
+          s[i][j] = fmaf(wq.v[i], s[i][j], kf * vf[j]);
         }
       }
-      __syncwarp();                                        // (the batch before has been added up)
 #pragma unroll
-      for (int q = 0; q < WK_BATCH; ++q)
+      for (int j = 0; j < WK_COLS; ++j) oq[j] = fmaf(c, vf[j], oq[j]);
+    };
+    if (gn == WK_GROUP) {
 #pragma unroll
-        for (int j = 0; j < WK_COLS; ++j) red[(q * WK_COLS + j) * WK_RED + lane] = o[q][j];
-      __syncwarp();
-      float total = 0.f;
+      for (int q = 0; q < WK_GROUP; ++q) token(q, o[q]);
+    } else {
 #pragma unroll
-      for (int i = 0; i < 32; i += 4) {
-        const float4 p = *reinterpret_cast<const float4*>(red + lane * WK_RED + i);
-        total += (p.x + p.y) + (p.z + p.w);
+      for (int q = 0; q < WK_GROUP; ++q) {
+#pragma unroll
+        for (int j = 0; j < WK_COLS; ++j) o[q][j] = 0.f;
+        if (q < gn) token(q, o[q]);
       }
-      const int q = q0 + lane / WK_COLS, c = c0 + lane % WK_COLS;
-      if (q < gn && c < V) out[(size_t)(t0 + g0 + q) * HV + h * V + c] = total;
     }
+#pragma unroll
+    for (int q = 0; q < WK_GROUP; ++q)
+#pragma unroll
+      for (int j = 0; j < WK_COLS; ++j) red[(q * WK_COLS + j) * WK_RED + lane] = o[q][j];
+    __syncwarp();
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < 32; i += 4) {
+      const float4 p = *reinterpret_cast<const float4*>(red + lane * WK_RED + i);
+      total += (p.x + p.y) + (p.z + p.w);
+    }
+    const int q = lane / WK_COLS, c = c0 + lane % WK_COLS;
+    if (q < gn && c < V) out[(size_t)(t0 + g0 + q) * HV + h * V + c] = total;
+    // (the next group's shares are written past the next block-wide barrier)
   }
   cp_async_wait<0>();
 #pragma unroll
@@ -655,7 +657,7 @@ TS_API int ts_wkv_scan(float* out, const void* r, const void* k, const void* v, 
   const dim3 grid(ceil_div(V, WK_COLS * WK_WARPS), H, B);
 #define TS_WKR(TT, RPL)                                                                                                  \
   do {                                                                                                                   \
-    const size_t smem = (size_t)WK_STAGES * WK_GROUP * (32 * RPL * (sizeof(float) + 2 * sizeof(TT)) + WK_COLS * WK_WARPS * sizeof(TT)) + \
+    const size_t smem = (size_t)wk_stages<TT, RPL>() * WK_GROUP * (32 * RPL * (sizeof(float) + 2 * sizeof(TT)) + WK_COLS * WK_WARPS * sizeof(TT)) + \
                         sizeof(float) * WK_WARPS * 32 * WK_RED;                                                          \
     static bool configured = false;                                                                                      \
     if (!configured) {                                                                                                   \
