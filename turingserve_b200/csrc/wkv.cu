@@ -216,10 +216,36 @@ constexpr int WK_GROUP = 16, WK_COLS = 2, WK_WARPS = 8, WK_RED = 36;
 static_assert(WK_GROUP * WK_COLS == 32, "a lane adds up one output of a group of tokens");
 template <typename T, int RPL> constexpr int wk_stages() { return RPL * (int)sizeof(T) >= 32 ? 3 : 4; }
 
-template <typename T, int N>
-struct alignas(sizeof(T) * N) WkVec {
-  T v[N];
-};
+// N neighbouring values as 32-bit numbers, in loads of up to 16 bytes
+template <int N> __device__ __forceinline__ void wk_load(float (&f)[N], const float* p) {
+  if constexpr (N >= 4) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      const float4 x = *reinterpret_cast<const float4*>(p + i);
+      f[i] = x.x; f[i + 1] = x.y; f[i + 2] = x.z; f[i + 3] = x.w;
+    }
+  } else if constexpr (N == 2) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    f[0] = x.x; f[1] = x.y;
+  } else {
+    f[0] = p[0];
+  }
+}
+template <int N> __device__ __forceinline__ void wk_load(float (&f)[N], const bf16* p) {
+  if constexpr (N == 1) {
+    f[0] = to_f(p[0]);
+  } else {
+    unsigned x[N / 2];
+    if constexpr (N == 8) *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(p);
+    else if constexpr (N == 4) *reinterpret_cast<uint2*>(x) = *reinterpret_cast<const uint2*>(p);
+    else x[0] = *reinterpret_cast<const unsigned*>(p);
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      f[2 * i] = __uint_as_float(x[i] << 16);
+      f[2 * i + 1] = __uint_as_float(x[i] & 0xffff0000u);
+    }
+  }
+}
 
 template <typename T, int RPL>
 __global__ void __launch_bounds__(WK_WARPS * 32, 1)
@@ -253,37 +279,67 @@ wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, 
 #pragma unroll
     for (int j = 0; j < WK_COLS; ++j) s[i][j] = (d < D && c0 + j < V) ? S[(size_t)d * V + c0 + j] : 0.f;
   }
-  for (int i = threadIdx.x; i < WK_STAGES * WK_GROUP * Dp; i += blockDim.x) {
-    w_s[i] = 0.f;
-    r_s[i] = from_f<T>(0.f);
-    k_s[i] = from_f<T>(0.f);
-  }
-  for (int i = threadIdx.x; i < WK_STAGES * WK_GROUP * BC; i += blockDim.x) v_s[i] = from_f<T>(0.f);
+  if (D < Dp)
+    for (int i = threadIdx.x; i < WK_STAGES * WK_GROUP * Dp; i += blockDim.x) {
+      w_s[i] = 0.f;
+      r_s[i] = from_f<T>(0.f);
+      k_s[i] = from_f<T>(0.f);
+    }
+  if (cols_here < BC)
+    for (int i = threadIdx.x; i < WK_STAGES * WK_GROUP * BC; i += blockDim.x) v_s[i] = from_f<T>(0.f);
   __syncthreads();
 
+  // Which 16-byte pieces of a token's rows [r | k | w | v] a lane brings is the same for every token: where they come from, how
+  // far apart two tokens' are there and here, and where they go is worked out once.  (`fast`: every piece starts on a 16-byte
+  // boundary on both sides; else single values.)
+  constexpr int PIECES = (RPL * (2 * (int)sizeof(T) + 4) + 15) / 16 + 1;
+  const char* src[PIECES];
+  unsigned src_step[PIECES], dst[PIECES], dst_step[PIECES];
+  const unsigned smem0 = (unsigned)__cvta_generic_to_shared(smem);
+  const int pr = D / PER, pw = D / 4, pv = (cols_here + PER - 1) / PER;
+#pragma unroll
+  for (int i = 0; i < PIECES; ++i) {
+    int at = lane + 32 * i;
+    src[i] = nullptr;
+    src_step[i] = dst[i] = dst_step[i] = 0u;
+    if (!fast) continue;
+    if (at < 2 * pr) {
+      const bool is_k = at >= pr;
+      const int c = (is_k ? at - pr : at) * PER;
+      src[i] = reinterpret_cast<const char*>((is_k ? k : r) + (size_t)t0 * HD + h * D + c);
+      src_step[i] = HD * (unsigned)sizeof(T);
+      dst[i] = smem0 + (unsigned)((const char*)((is_k ? k_s : r_s) + c) - (const char*)smem);
+      dst_step[i] = Dp * (unsigned)sizeof(T);
+    } else if ((at -= 2 * pr) < pw) {
+      src[i] = reinterpret_cast<const char*>(w + (size_t)t0 * HD + h * D + at * 4);
+      src_step[i] = HD * 4u;
+      dst[i] = smem0 + (unsigned)((const char*)(w_s + at * 4) - (const char*)smem);
+      dst_step[i] = Dp * 4u;
+    } else if ((at -= pw) < pv) {
+      src[i] = reinterpret_cast<const char*>(v + (size_t)t0 * HV + h * V + b0 + at * PER);
+      src_step[i] = HV * (unsigned)sizeof(T);
+      dst[i] = smem0 + (unsigned)((const char*)(v_s + at * PER) - (const char*)smem);
+      dst_step[i] = BC * (unsigned)sizeof(T);
+    }
+  }
   auto fetch = [&](int g0, int st) {
     const int gn = min(WK_GROUP, n - g0);
     for (int q = warp; q < gn; q += WK_WARPS) {
-      const size_t t = t0 + g0 + q;
-      const T* rr = r + t * HD + h * D;
-      const T* kr = k + t * HD + h * D;
-      const T* vr = v + t * HV + h * V + b0;
-      const float* wr = w + t * HD + h * D;
       const int at = st * WK_GROUP + q;
       if (fast) {
-        for (int c = lane * PER; c < D; c += 32 * PER) {
-          cp_async_16(r_s + at * Dp + c, rr + c, true);
-          cp_async_16(k_s + at * Dp + c, kr + c, true);
-        }
-        for (int c = lane * 4; c < D; c += 128) cp_async_16(w_s + at * Dp + c, wr + c, true);
-        if (lane * PER < cols_here) cp_async_16(v_s + at * BC + lane * PER, vr + lane * PER, true);
+#pragma unroll
+        for (int i = 0; i < PIECES; ++i)
+          if (src[i] != nullptr)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst[i] + (unsigned)at * dst_step[i]),
+                         "l"(src[i] + (size_t)(unsigned)(g0 + q) * src_step[i]));
       } else {
+        const size_t t = t0 + g0 + q;
         for (int c = lane; c < D; c += 32) {
-          r_s[at * Dp + c] = rr[c];
-          k_s[at * Dp + c] = kr[c];
-          wk_cp_async_4(w_s + at * Dp + c, wr + c);
+          r_s[at * Dp + c] = r[t * HD + h * D + c];
+          k_s[at * Dp + c] = k[t * HD + h * D + c];
+          wk_cp_async_4(w_s + at * Dp + c, w + t * HD + h * D + c);
         }
-        for (int c = lane; c < cols_here; c += 32) v_s[at * BC + c] = vr[c];
+        for (int c = lane; c < cols_here; c += 32) v_s[at * BC + c] = v[t * HV + h * V + b0 + c];
       }
     }
   };
@@ -305,24 +361,20 @@ wkv_scan_kernel(float* out, const T* r, const T* k, const T* v, const float* w, 
     const float* w_l = w_s + st * WK_GROUP * Dp + lane * RPL;
     const T* v_l = v_s + st * WK_GROUP * BC + warp * WK_COLS;
     auto token = [&](int q, float (&oq)[WK_COLS]) {
-      const WkVec<T, RPL> rq = *reinterpret_cast<const WkVec<T, RPL>*>(r_l + q * Dp);
-      const WkVec<T, RPL> kq = *reinterpret_cast<const WkVec<T, RPL>*>(k_l + q * Dp);
-      const WkVec<float, RPL> wq = *reinterpret_cast<const WkVec<float, RPL>*>(w_l + q * Dp);
-      const WkVec<T, WK_COLS> vq = *reinterpret_cast<const WkVec<T, WK_COLS>*>(v_l + q * BC);
-      float c = 0.f, vf[WK_COLS];                          // c: this lane's part of the sum of r u k
+      float rq[RPL], kq[RPL], wq[RPL], vf[WK_COLS], c = 0.f;   // c: this lane's part of the sum of r u k
+      wk_load(rq, r_l + q * Dp);
+      wk_load(kq, k_l + q * Dp);
+      wk_load(wq, w_l + q * Dp);
+      wk_load(vf, v_l + q * BC);
 #pragma unroll
-      for (int j = 0; j < WK_COLS; ++j) {
-        vf[j] = to_f(vq.v[j]);
-        oq[j] = 0.f;
-      }
+      for (int j = 0; j < WK_COLS; ++j) oq[j] = 0.f;
 #pragma unroll
       for (int i = 0; i < RPL; ++i) {
-        const float rf = to_f(rq.v[i]), kf = to_f(kq.v[i]);
-        c = fmaf(rf, uu[i] * kf, c);
+        c = fmaf(rq[i], uu[i] * kq[i], c);
 #pragma unroll
         for (int j = 0; j < WK_COLS; ++j) {
-          oq[j] = fmaf(s[i][j], rf, oq[j]);
-          s[i][j] = fmaf(wq.v[i], s[i][j], kf * vf[j]);
+          oq[j] = fmaf(s[i][j], rq[i], oq[j]);
+          s[i][j] = fmaf(wq[i], s[i][j], kq[i] * vf[j]);
         }
       }
 #pragma unroll
@@ -642,6 +694,9 @@ TS_API int ts_wkv_decay(float* out, const float* z, const void* w2, const float*
 // input; state [slots, state_stride]: [H D V | hidden].  longest: the most tokens a request brings (0: not known); long
 // portions are launched late (see ts_launch_late).
 constexpr int WK_LATE_TOKENS = 64;
+// Long portions whose blocks are at most one an SM ask for so much shared memory that no SM takes two of them (left to itself the
+// hardware puts two on some SMs while others stay empty, and the scan is as slow as those).
+constexpr size_t WK_ALONE_BYTES = 116 * 1024;
 
 TS_API int ts_wkv_scan(float* out, const void* r, const void* k, const void* v, const float* w, const float* u, const void* h_in,
                        float* state, long long state_stride, const int* q_start, const int* slots, int B, int H, int D, int V,
@@ -655,13 +710,15 @@ TS_API int ts_wkv_scan(float* out, const void* r, const void* k, const void* v, 
   const int fast = D % per == 0 && V % per == 0 && D % 4 == 0 &&
                    !(((uintptr_t)r | (uintptr_t)k | (uintptr_t)v | (uintptr_t)w) & 15);
   const dim3 grid(ceil_div(V, WK_COLS * WK_WARPS), H, B);
+  const bool alone = longest >= WK_LATE_TOKENS && (long long)grid.x * grid.y * grid.z <= 148;
 #define TS_WKR(TT, RPL)                                                                                                  \
   do {                                                                                                                   \
-    const size_t smem = (size_t)wk_stages<TT, RPL>() * WK_GROUP * (32 * RPL * (sizeof(float) + 2 * sizeof(TT)) + WK_COLS * WK_WARPS * sizeof(TT)) + \
+    size_t smem = (size_t)wk_stages<TT, RPL>() * WK_GROUP * (32 * RPL * (sizeof(float) + 2 * sizeof(TT)) + WK_COLS * WK_WARPS * sizeof(TT)) + \
                         sizeof(float) * WK_WARPS * 32 * WK_RED;                                                          \
+    if (alone && smem < WK_ALONE_BYTES) smem = WK_ALONE_BYTES;                                                           \
     static bool configured = false;                                                                                      \
     if (!configured) {                                                                                                   \
-      cudaError_t e = cudaFuncSetAttribute(wkv_scan_kernel<TT, RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      cudaError_t e = cudaFuncSetAttribute(wkv_scan_kernel<TT, RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(smem < WK_ALONE_BYTES ? WK_ALONE_BYTES : smem)); \
       if (e != cudaSuccess) TS_REFUSE((int)e, "ts_wkv_scan: shared memory %zu: %s", smem, cudaGetErrorString(e));        \
       configured = true;                                                                                                 \
     }                                                                                                                    \
