@@ -71,7 +71,7 @@ def test_mixes_of_a_token_and_the_one_before(ops, dtype, hidden):
 
 
 @DTYPES
-@pytest.mark.parametrize("T,N,R", [(1, 14, 5), (3, 192, 16), (70, 100, 33), (130, 256, 64), (2, 64, 1), (300, 320, 128), (65, 72, 24)])
+@pytest.mark.parametrize("T,N,R", [(1, 14, 5), (3, 200, 16), (70, 100, 33), (130, 256, 64), (2, 64, 1), (300, 320, 128), (65, 72, 24)])
 def test_decays(ops, dtype, T, N, R):
     """From decays that keep everything to decays that keep nothing, all in 32-bit in both engine types."""
     g = torch.Generator(device=DEV).manual_seed(T + N)
@@ -475,7 +475,7 @@ def test_one_loud_key_at_every_edge(ops, decode, dtype, H, rank, R, page):
 
 # -- routing ------------------------------------------------------------------------------------------------------------------
 @DTYPES
-@pytest.mark.parametrize("E,top,groups,keep", [(16, 2, 2, 1), (12, 3, 4, 2), (6, 2, 6, 3), (9, 1, 3, 1), (5, 2, 1, 1), (64, 6, 8, 3), (8, 4, 2, 2),
+@pytest.mark.parametrize("E,top,groups,keep", [(20, 2, 2, 1), (12, 3, 4, 2), (6, 2, 6, 3), (9, 1, 3, 1), (5, 2, 1, 1), (64, 6, 8, 3), (8, 4, 2, 2),
                                                (130, 5, 65, 7)])
 def test_grouped_routing(ops, dtype, E, top, groups, keep):
     """Choices by scores with corrections (negative ones too), groups by their two largest; weights without the correction over
